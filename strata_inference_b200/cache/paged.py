@@ -20,7 +20,12 @@ and fixed-size per-sequence state.
   are still there when its last one arrives.
 * *State* is a fixed-size tensor per slot and schedule entry for mixers
   that carry a recurrent state instead of keys; it is zeroed when the slot
-  is acquired.  (The attention mixer needs none.)
+  is acquired.  (The attention mixer needs none.)  A part at a mixer's input (a short
+  convolution) has a second one beside the mixer's, ``CacheNeed.inputs``.
+* A group whose need names ``keep_first`` = K (with a window) keeps the sequence's first K
+  positions for good: they lie in whole pages of their own ahead of the ring
+  (``fixed_tokens`` positions, K rounded up to pages), which nothing overwrites; position
+  p >= fixed_tokens lives in cell fixed_tokens + (p - fixed_tokens) % ring_tokens.
 
 The reference keeps one dense [max_seq_len, kv_dim] buffer per layer and a
 single position counter (src/model/cache.rs:23-43,77-112); its errors for
@@ -74,6 +79,8 @@ class KVNeed:
     # of chunks); every position is kept all the same, since a run that reads this cache may
     # cut its chunks elsewhere
     chunk: int = 0
+    # K > 0 (with a window): the sequence's first K positions stay visible for good
+    keep_first: int = 0
 
     @property
     def v_dim(self) -> int:
@@ -92,6 +99,8 @@ class StateNeed:
 class CacheNeed:
     kv: Optional[KVNeed] = None
     state: Optional[StateNeed] = None
+    # state of the part at the mixer's input, apart from the mixer's own
+    inputs: Optional[StateNeed] = None
 
 
 class PagePool:
@@ -165,6 +174,10 @@ class KVGroup:
         full_pages = -(-max_seq_len // page_tokens)
         # what a ring keeps behind a position: the window, and a whole block where blocks are pooled
         self.keep = max(need.window, need.pool) if need.window > 0 else 0
+        if need.keep_first > 0 and (need.window <= 0 or need.pool > 0 or need.values_in_keys):
+            raise CacheError("kept first positions go with a window, and without pooled blocks or shared cells")
+        # whole pages ahead of the ring for the positions that are kept for good
+        fixed_pages = -(-need.keep_first // page_tokens)
         if need.window <= 0:
             ring_pages = full_pages
         elif max_continuation is None:
@@ -172,12 +185,13 @@ class KVGroup:
         else:
             # a step of c positions writes c - 1 cells ahead of what its first row still sees
             ring_pages = -(-(self.keep + max(1, max_continuation) - 1) // page_tokens)
-        if ring_pages >= full_pages:
-            self.ring_tokens = 0          # never wraps
+        if fixed_pages + ring_pages >= full_pages:
+            self.ring_tokens = self.fixed_tokens = 0          # never wraps
             self.pages_per_seq = full_pages
         else:
             self.ring_tokens = ring_pages * page_tokens
-            self.pages_per_seq = ring_pages
+            self.fixed_tokens = fixed_pages * page_tokens
+            self.pages_per_seq = fixed_pages + ring_pages
         self.n_pages = min(n_pages, max_slots * self.pages_per_seq)
         self.pool = PagePool(self.n_pages)
         shape = (len(entries), self.n_pages, need.n_kv_heads, page_tokens)
@@ -209,7 +223,7 @@ class KVGroup:
         if self.ring_tokens == 0:
             return 1 << 30
         room = self.ring_tokens - self.keep + 1
-        return room if start is None else max(self.ring_tokens - start, room)
+        return room if start is None else max(self.fixed_tokens + self.ring_tokens - start, room)
 
     def bytes(self) -> int:
         held = self.k.numel() + (0 if self.v is self.k else self.v.numel())
@@ -235,8 +249,9 @@ class SequenceCache:
         if max_slots is None:
             # (state is held for every slot, live or not: where the caller names no number of
             # slots, no more of them than keep the state within STATE_BUDGET bytes)
-            per_slot = sum(_count(need.state.shape) * torch.empty((), dtype=need.state.dtype).element_size()
-                           for need in needs if need is not None and need.state is not None)
+            per_slot = sum(_count(st.shape) * torch.empty((), dtype=st.dtype).element_size()
+                           for need in needs if need is not None
+                           for st in (need.state, need.inputs) if st is not None)
             if per_slot * self.max_slots > STATE_BUDGET:
                 self.max_slots = max(MIN_SLOTS, min(self.max_slots, STATE_BUDGET // per_slot))
         # groups of schedule entries with the same need
@@ -253,11 +268,15 @@ class SequenceCache:
         for gi, g in enumerate(self.groups):
             for li, entry in enumerate(g.entries):
                 self._where[entry] = (gi, li)
+        def per_slot_state(st: StateNeed) -> torch.Tensor:
+            return torch.zeros((self.max_slots,) + tuple(st.shape), dtype=st.dtype, device=device)
         self.state: Dict[int, torch.Tensor] = {}
+        self.inputs: Dict[int, torch.Tensor] = {}
         for entry, need in enumerate(needs):
             if need is not None and need.state is not None:
-                self.state[entry] = torch.zeros((self.max_slots,) + tuple(need.state.shape),
-                                                dtype=need.state.dtype, device=device)
+                self.state[entry] = per_slot_state(need.state)
+            if need is not None and need.inputs is not None:
+                self.inputs[entry] = per_slot_state(need.inputs)
         self.named: Dict[str, torch.Tensor] = {
             name: torch.zeros((self.max_slots,) + tuple(need.shape), dtype=need.dtype, device=device)
             for name, need in (named_state or {}).items()}
@@ -278,7 +297,7 @@ class SequenceCache:
             raise CacheError(f"slot {s} handed out twice")
         self._live[s] = True
         self.lengths[s] = 0
-        for t in list(self.state.values()) + list(self.named.values()):
+        for t in list(self.state.values()) + list(self.inputs.values()) + list(self.named.values()):
             t[s].zero_()
         return s
 
@@ -365,7 +384,8 @@ class SequenceCache:
         g = self.groups[gi]
         c = g.cells
         if c is None:
-            return KVView(g.k[li], g.v[li], g.table, g.page_tokens, g.ring_tokens, g.need)
+            return KVView(g.k[li], g.v[li], g.table, g.page_tokens, g.ring_tokens, g.need,
+                          fixed_tokens=g.fixed_tokens)
         return KVView(g.k[li], g.v[li], g.table, g.page_tokens, g.ring_tokens, g.need,
                       c.k[li], c.v[li], c.table, c.page_tokens)
 
@@ -374,6 +394,9 @@ class SequenceCache:
 
     def state_view(self, entry: int) -> torch.Tensor:
         return self.state[entry]
+
+    def input_state_view(self, entry: int) -> torch.Tensor:
+        return self.inputs[entry]
 
     def named_state(self, name: str) -> torch.Tensor:
         return self.named[name]
@@ -401,3 +424,4 @@ class KVView:
     cell_v: Optional[torch.Tensor] = None
     cell_table: Optional[torch.Tensor] = None
     cell_page_tokens: int = 0
+    fixed_tokens: int = 0      # positions below it lie in cells of their own, ahead of the ring

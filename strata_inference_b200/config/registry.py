@@ -93,6 +93,8 @@ def _register_builtin() -> None:
     register_architecture(("Gegorax", "gegorax"), GegoraxConfig.from_dict, gegorax_spec, gegorax_sizes)
     from .besorax import BesoraxConfig, besorax_sizes, besorax_spec
     register_architecture(("Besorax", "besorax"), BesoraxConfig.from_dict, besorax_spec, besorax_sizes)
+    from .kerolorn import KerolornConfig, kerolorn_sizes, kerolorn_spec
+    register_architecture(("Kerolorn", "kerolorn"), KerolornConfig.from_dict, kerolorn_spec, kerolorn_sizes)
 
 
 _register_builtin()

@@ -51,6 +51,9 @@ struct AttnDecodeArgs {
     int fresh;
     // > 0: a row sees the positions of its own chunk of that many (first_visible)
     int chunk;
+    // > 0 (with a window): the sequence's first `keep` positions stay visible; they lie in the
+    // `fixed_tokens` cells ahead of the ring (common.cuh cell_of)
+    int keep, fixed_tokens;
     // one value per query head whose exponential joins the softmax's denominator; null: none
     const float* sink;
 };
@@ -179,14 +182,21 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) attention_decode_kernel(Attn
     const int pos = p.row_pos[r];
     const int slot = p.seq_slot[p.row_seq[r]];
     const int lo = first_visible(pos, p.window, p.chunk);
-    const int tile_lo = lo >> 4, tile_hi = pos >> 4;             // inclusive
-    const int n_tiles = tile_hi - tile_lo + 1;
+    // Tiles of kept first positions (n_kept of them), then the window's from the first that is
+    // not one of those; a tile's number `v` in that order is position tile v, or v + skip from
+    // the window on.
+    const int n_kept = kept_before(lo, p.keep);
+    const int kept_tiles = (n_kept + 15) >> 4;
+    const int tile_lo = max(lo >> 4, kept_tiles), tile_hi = pos >> 4;             // inclusive
+    const int skip = tile_lo - kept_tiles;
+    const int n_tiles = kept_tiles + max(0, tile_hi - tile_lo + 1);
     const int per = (n_tiles + nw * p.splits - 1) / (nw * p.splits);
-    const int t0 = tile_lo + (split * nw + warp) * per;
-    const int t1 = min(t0 + per, tile_hi + 1);
+    const int t0 = (split * nw + warp) * per;
+    const int t1 = min(t0 + per, n_tiles);
+    auto tile_at = [&](int v) { return v < kept_tiles ? v : v + skip; };
     const int* table = p.page_table + (size_t)slot * p.max_pages;
     if (t0 < t1) {
-        const int cell0 = p.ring_tokens > 0 ? (t0 << 4) % p.ring_tokens : (t0 << 4);
+        const int cell0 = cell_of(tile_at(t0) << 4, p.fixed_tokens, p.ring_tokens);
         asm volatile("prefetch.global.L1 [%0];\n" ::"l"(table + cell0 / p.page_tokens));
     }
     // One tile of keys and values: every load is issued before anything waits on one.
@@ -195,7 +205,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) attention_decode_kernel(Attn
     const int dim0 = (lane % LPK) * 8;   // its 8 dimensions
     auto load_tile = [&](int tile) {
         const int base = tile << 4;
-        const int cell = p.ring_tokens > 0 ? base % p.ring_tokens : base;
+        const int cell = cell_of(base, p.fixed_tokens, p.ring_tokens);
         const int page = table[cell / p.page_tokens];
         const size_t tile_off =
             (((size_t)page * p.n_kv + kvh) * p.page_tokens + cell % p.page_tokens) * HD;
@@ -213,8 +223,8 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) attention_decode_kernel(Attn
             v_r[i] = ld_stream16(vt + (size_t)min(i * KPP + sub, last) * HD + dim0);
     };
     // the first tile's keys and values, if the kernel before this one cannot have written them
-    const bool early = EARLY && p.fresh > 0 && t0 < t1 && (t0 << 4) + 15 < pos - p.fresh + 1;
-    if (early) load_tile(t0);
+    const bool early = EARLY && p.fresh > 0 && t0 < t1 && (tile_at(t0) << 4) + 15 < pos - p.fresh + 1;
+    if (early) load_tile(tile_at(t0));
     pdl_wait();
 
     // query heads of this kv head as the B operand: lane (g, t) holds head g
@@ -237,8 +247,8 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) attention_decode_kernel(Attn
     }
 
     for (int tile = t0; tile < t1; ++tile) {
-        const int base = tile << 4;                               // first position of the tile
-        if (!(early && tile == t0)) load_tile(tile);
+        const int base = tile_at(tile) << 4;                      // first position of the tile
+        if (!(early && tile == t0)) load_tile(tile_at(tile));
         // ---- scores: 16 keys x G heads ----
         float c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -254,7 +264,7 @@ __global__ void __launch_bounds__(WIDE ? 256 : 128) attention_decode_kernel(Attn
                 float s = c[i] * p.scale;
                 if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
                 const int kpos = base + key;
-                s_sm[key][head] = (kpos >= lo && kpos <= pos) ? s : -INFINITY;
+                s_sm[key][head] = ((kpos >= lo || kpos < n_kept) && kpos <= pos) ? s : -INFINITY;
             }
         }
         __syncwarp();
@@ -506,10 +516,14 @@ static int attention_decode(
     int max_pages, int page_tokens, int ring_tokens, const int* row_pos, const int* row_seq,
     const int* seq_slot, void* out, float* partial, int* tickets, int rows, int n_heads, int n_kv,
     int head_dim, float scale, float softcap, int window, int splits, int warps, int fresh,
-    void* stream, int chunk = 0, const float* sink = nullptr) {
+    void* stream, int chunk = 0, const float* sink = nullptr, int keep = 0, int fixed_tokens = 0) {
     if (rows == 0) return 0;
     SIB_REQUIRE(chunk >= 0 && (chunk == 0 || window == 0), "attention_decode: chunk=%d window=%d (a chunk "
                 "goes without a window)", chunk, window);
+    SIB_REQUIRE(keep >= 0 && fixed_tokens >= 0 && fixed_tokens % 16 == 0 && (keep == 0 || window > 0) &&
+                    (ring_tokens == 0 || fixed_tokens >= keep),
+                "attention_decode: keep=%d with window=%d (kept positions go with a window and lie in the "
+                "%d fixed cells)", keep, window, fixed_tokens);
     SIB_REQUIRE(sib_attention_decode_supports(n_heads, n_kv, head_dim, page_tokens),
                 "attention_decode: heads=%d kv_heads=%d head_dim=%d page_tokens=%d is not a shape "
                 "this kernel takes (groups of 1, 2, 4 or 8 heads; head_dim 64, 128 or 256; pages "
@@ -532,7 +546,7 @@ static int attention_decode(
     AttnDecodeArgs p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
                      (const __nv_bfloat16*)v_pool, (__nv_bfloat16*)out, partial, tickets, row_pos, row_seq,
                      seq_slot, page_table, q_stride, rows, n_heads, n_kv, max_pages, page_tokens,
-                     ring_tokens, window, splits, scale, softcap, fresh, chunk, sink};
+                     ring_tokens, window, splits, scale, softcap, fresh, chunk, keep, fixed_tokens, sink};
     const long long blocks = (long long)rows * n_kv * splits;
     SIB_REQUIRE(blocks < (1ll << 31), "attention_decode: too many rows (%d)", rows);
     cudaStream_t s = (cudaStream_t)stream;
@@ -603,18 +617,19 @@ SIB_EXPORT int sib_attention_decode_fresh(
                             stream);
 }
 
-// The same with a mask of chunks and a sink per query head (`chunk` 0 and `sink` null: neither).
+// The same with a mask of chunks, a sink per query head and first positions that a window keeps
+// (`chunk` 0, `sink` null, `keep` 0: none of them).
 SIB_EXPORT int sib_attention_decode_masked(
     const void* q, int q_stride, const void* k_pool, const void* v_pool, const int* page_table,
     int max_pages, int page_tokens, int ring_tokens, const int* row_pos, const int* row_seq,
     const int* seq_slot, void* out, float* partial, int* tickets, int rows, int n_heads, int n_kv,
     int head_dim, float scale, float softcap, int window, int splits, int warps, int fresh,
-    int chunk, const float* sink, void* stream) {
+    int chunk, const float* sink, int keep, int fixed_tokens, void* stream) {
     SIB_REQUIRE(fresh >= 0, "attention_decode: %d fresh positions", fresh);
     return attention_decode(q, q_stride, k_pool, v_pool, page_table, max_pages, page_tokens,
                             ring_tokens, row_pos, row_seq, seq_slot, out, partial, tickets, rows,
                             n_heads, n_kv, head_dim, scale, softcap, window, splits, warps, fresh,
-                            stream, chunk, sink);
+                            stream, chunk, sink, keep, fixed_tokens);
 }
 
 // ---------------------------------------------------------------------------

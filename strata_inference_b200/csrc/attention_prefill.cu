@@ -6,7 +6,8 @@
 // A block of 4 warps takes 64 query rows of one (sequence, kv head): the G
 // query heads that share the kv head times 64 / G consecutive positions, so a
 // key/value tile is loaded once for all of them.  Keys are walked in tiles of
-// 64, from the first tile any of its rows can see (window) to the diagonal
+// 64, from the first tile any of its rows can see (window; ahead of it the tiles of the
+// sequence's first positions where the window keeps some) to the diagonal
 // (causal); tiles are copied into shared memory with cp.async, two tiles in
 // flight, 16-byte chunks XOR-swizzled by row so that ldmatrix reads are free
 // of bank conflicts.  Scores and the weighted sum run on mma.m16n8k16 with the
@@ -24,7 +25,7 @@ struct AttnPrefillArgs {
     const int* seq_len;         // [seqs] rows (= positions, the step starts at position 0)
     int width;                  // elements per packed row
     int n_heads, n_kv;
-    int window;
+    int window, keep;           // keep > 0 (with a window): the first `keep` positions stay visible
     float scale, softcap;
 };
 
@@ -125,12 +126,16 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
     }
     const int k_hi = min(n, p0 + MP);                                    // keys < k_hi
     const int k_lo = p.window > 0 ? max(0, p0 - p.window + 1) : 0;
-    const int kt0 = k_lo >> 6, kt1 = (k_hi + 63) >> 6;
+    // tile number `v`: a tile of kept first positions, or v + skip from the window's first tile on
+    const int kept_tiles = (kept_before(k_lo, p.keep) + 63) >> 6;
+    const int skip = max(k_lo >> 6, kept_tiles) - kept_tiles;
+    const int nt = max((k_hi + 63) >> 6, kept_tiles + skip) - skip;
+    auto tile_at_number = [&](int v) { return v < kept_tiles ? v : v + skip; };
     const __nv_bfloat16* kbase = p.qkv + (size_t)row0 * p.width + (size_t)(p.n_heads + kvh) * HD;
     const __nv_bfloat16* vbase = kbase + (size_t)p.n_kv * HD;
-    load_rows<HD>(Ks, kbase, p.width, kt0 * 64, n - kt0 * 64);
+    load_rows<HD>(Ks, kbase, p.width, tile_at_number(0) * 64, n - tile_at_number(0) * 64);
     if (!DOUBLE) cp_async_commit();              // queries and keys first, values as a second group
-    load_rows<HD>(Vs, vbase, p.width, kt0 * 64, n - kt0 * 64);
+    load_rows<HD>(Vs, vbase, p.width, tile_at_number(0) * 64, n - tile_at_number(0) * 64);
     cp_async_commit();
 
     float o[DN][4];
@@ -140,19 +145,21 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
     // positions of this lane's two rows (g and g + 8 of the warp's 16)
     const int qpos0 = p0 + (16 * warp + g) % MP, qpos1 = p0 + (16 * warp + g + 8) % MP;
 
-    for (int kt = kt0; kt < kt1; ++kt) {
-        const int buf = DOUBLE ? (kt - kt0) & 1 : 0;
+    for (int v = 0; v < nt; ++v) {
+        const int kt = tile_at_number(v);
+        const int buf = DOUBLE ? v & 1 : 0;
         if (DOUBLE) {
-            if (kt + 1 < kt1) {
-                load_rows<HD>(Ks + (buf ^ 1) * 64 * HD, kbase, p.width, (kt + 1) * 64, n - (kt + 1) * 64);
-                load_rows<HD>(Vs + (buf ^ 1) * 64 * HD, vbase, p.width, (kt + 1) * 64, n - (kt + 1) * 64);
+            if (v + 1 < nt) {
+                const int after = tile_at_number(v + 1) * 64;
+                load_rows<HD>(Ks + (buf ^ 1) * 64 * HD, kbase, p.width, after, n - after);
+                load_rows<HD>(Vs + (buf ^ 1) * 64 * HD, vbase, p.width, after, n - after);
                 cp_async_commit();
                 cp_async_wait<1>();
             } else {
                 cp_async_wait<0>();
             }
         } else {
-            if (kt > kt0) {
+            if (v > 0) {
                 load_rows<HD>(Ks, kbase, p.width, kt * 64, n - kt * 64);
                 cp_async_commit();
                 load_rows<HD>(Vs, vbase, p.width, kt * 64, n - kt * 64);
@@ -186,7 +193,7 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
         // of the warp (consecutive positions of one head): no per-element mask there.
         const int wq_lo = p0 + (16 * warp) % MP;
         const bool inside = kt * 64 + 63 <= wq_lo && kt * 64 + 63 < n &&
-                            (p.window <= 0 || wq_lo + 15 - kt * 64 < p.window);
+                            (p.window <= 0 || wq_lo + 15 - kt * 64 < p.window || kt * 64 + 63 < p.keep);
         const float inv_cap = p.softcap > 0.f ? 1.0f / p.softcap : 0.f;
         float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
@@ -198,7 +205,8 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
                 if (!inside) {
                     const int key = kt * 64 + 8 * j + 2 * t + (i & 1);
                     const int qp = (i < 2) ? qpos0 : qpos1;
-                    const bool seen = key <= qp && key < n && (p.window <= 0 || qp - key < p.window);
+                    const bool seen = key <= qp && key < n &&
+                                      (p.window <= 0 || qp - key < p.window || key < p.keep);
                     v = seen ? v : -INFINITY;
                 }
                 s[j][i] = v;
@@ -307,7 +315,7 @@ static int launch_prefill(const AttnPrefillArgs& p, int n_seqs, int max_len, cud
 SIB_EXPORT int sib_attention_prefill(const void* qkv, int width, void* out, const int* seq_row0,
                                      const int* seq_len, int n_seqs, int max_len, int n_heads,
                                      int n_kv, int head_dim, float scale, float softcap,
-                                     int window, void* stream) {
+                                     int window, int keep, void* stream) {
     if (n_seqs == 0 || max_len == 0) return 0;
     SIB_REQUIRE(sib_attention_prefill_supports(n_heads, n_kv, head_dim),
                 "attention_prefill: heads=%d kv_heads=%d head_dim=%d is not a shape this kernel "
@@ -316,10 +324,11 @@ SIB_EXPORT int sib_attention_prefill(const void* qkv, int width, void* out, cons
     SIB_REQUIRE(width == (n_heads + 2 * n_kv) * head_dim && ((uintptr_t)qkv % 16) == 0 &&
                     ((uintptr_t)out % 16) == 0,
                 "attention_prefill: packed rows of %d elements do not fit the head counts", width);
-    SIB_REQUIRE(n_seqs > 0 && n_seqs < 65536 && n_kv < 65536 && max_len > 0 && window >= 0,
-                "attention_prefill: seqs=%d max_len=%d", n_seqs, max_len);
+    SIB_REQUIRE(n_seqs > 0 && n_seqs < 65536 && n_kv < 65536 && max_len > 0 && window >= 0 &&
+                    keep >= 0 && (keep == 0 || window > 0),
+                "attention_prefill: seqs=%d max_len=%d window=%d keep=%d", n_seqs, max_len, window, keep);
     AttnPrefillArgs p{(const __nv_bfloat16*)qkv, (__nv_bfloat16*)out, seq_row0, seq_len, width,
-                      n_heads, n_kv, window, scale, softcap};
+                      n_heads, n_kv, window, keep, scale, softcap};
     cudaStream_t s = (cudaStream_t)stream;
     const int G = n_heads / n_kv;
 #define BY_G(HD)                                                              \

@@ -231,17 +231,22 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-// Whether key j of the thread's 64 keys is one the row sees.
-__device__ __forceinline__ bool sees(int j, int j_lo, int j_hi) { return j >= j_lo && j <= j_hi; }
+// Whether key j of the thread's 64 keys is one the row sees (MASK 1: a range; MASK 2: the
+// range, and the keys below j_keep, the sequence's first positions that a window keeps).
+template <int MASK>
+__device__ __forceinline__ bool sees(int j, int j_lo, int j_hi, int j_keep) {
+    if (MASK == 2) return j <= j_hi && (j >= j_lo || j < j_keep);
+    return j >= j_lo && j <= j_hi;
+}
 
 // The largest of 64 raw products (of those the row sees, with MASK).
-template <bool MASK>
-__device__ __forceinline__ float row_max(const uint32_t (&raw)[64], int j_lo, int j_hi) {
+template <int MASK>
+__device__ __forceinline__ float row_max(const uint32_t (&raw)[64], int j_lo, int j_hi, int j_keep = 0) {
     float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < 64; ++j) {
         float v = __uint_as_float(raw[j]);
-        if (MASK) v = sees(j, j_lo, j_hi) ? v : -INFINITY;
+        if (MASK) v = sees<MASK>(j, j_lo, j_hi, j_keep) ? v : -INFINITY;
         m[j & 3] = fmaxf(m[j & 3], v);
     }
     return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
@@ -249,9 +254,9 @@ __device__ __forceinline__ float row_max(const uint32_t (&raw)[64], int j_lo, in
 
 // 64 probabilities 2^(score - ref) as 32 packed bfloat16 pairs (in place of the raw
 // products); returns their sum.  CAP: score = c2 * tanh(product * c1), else product * c1.
-template <bool CAP, bool MASK>
+template <bool CAP, int MASK>
 __device__ __forceinline__ float probabilities(uint32_t (&raw)[64], float c1, float c2, float ref,
-                                               int j_lo, int j_hi) {
+                                               int j_lo, int j_hi, int j_keep = 0) {
     float sum[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int k = 0; k < 32; ++k) {
@@ -262,7 +267,7 @@ __device__ __forceinline__ float probabilities(uint32_t (&raw)[64], float c1, fl
             float x = __uint_as_float(raw[j]);
             if (CAP) x = fmaf(c2, tanh_fast(x * c1), -ref);
             else x = fmaf(x, c1, -ref);
-            if (MASK) x = sees(j, j_lo, j_hi) ? x : -INFINITY;
+            if (MASK) x = sees<MASK>(j, j_lo, j_hi, j_keep) ? x : -INFINITY;
             e[h] = exp2_fast(x);
         }
         sum[k & 3] += e[0] + e[1];
@@ -282,6 +287,7 @@ struct TcArgs {
     int split_tiles;         // blocks with at least this many key tiles are split (0: none)
     int n_heads, n_kv;
     int window;
+    int keep;                // > 0 (with a window, no cap): the first `keep` positions stay visible
     float scale, softcap;
     const float* sink;       // [n_heads] or null: e^{sink_h} joins each row's denominator
     // [rows, n_heads, head_dim + 2] or null: per (row, head) the (max, sum, accumulator) of keys
@@ -379,7 +385,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
     const int row0 = p.seq_row0[b];
     const int k_hi = min(n, first0 + NB * MP);
     const int k_lo = p.window > 0 ? max(0, first0 - p.window + 1) : 0;
-    int kt0 = k_lo / BN, nt = (k_hi + BN - 1) / BN - kt0;
+    // Key tile number `v`: one of the tiles of kept first positions, or v + skip from the
+    // window's first tile on.
+    const int kept_tiles = (kept_before(k_lo, p.keep) + BN - 1) / BN;
+    const int skip = max(k_lo / BN, kept_tiles) - kept_tiles;
+    int kt0 = 0, nt = max((k_hi + BN - 1) / BN - skip, kept_tiles);
+    auto tile_at = [&](int v) { return v < kept_tiles ? v : v + skip; };
     // a long run of key tiles is shared with the block that has the other part
     // (the other blockIdx.z / n_kv of a grid, the other item of a list)
     const bool is_split = items.n > 0 ? listed_split : (p.split_tiles > 0 && nt >= p.split_tiles);
@@ -464,7 +475,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
                 for (int c = 0; c < CH; ++c)
                     for (int r64 = 0; r64 < K_ROWS / 64; ++r64)
                         load(Ks + s * KV_BYTES + c * K_CHUNK + r64 * (64 * 128), &bars->k_full[s],
-                             k_col + 64 * c, row0 + (kt0 + t) * BN + K_ROWS * rank + 64 * r64);
+                             k_col + 64 * c, row0 + tile_at(kt0 + t) * BN + K_ROWS * rank + 64 * r64);
                 return true;
             };
             auto load_v = [&](int t) -> bool {
@@ -474,7 +485,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
                 for (int c = 0; c < V_CH; ++c)
                     for (int r64 = 0; r64 < BN / 64; ++r64)
                         load(Vs + s * KV_BYTES + c * V_CHUNK + r64 * (64 * 128), &bars->v_full[s],
-                             v_col + (HD / NB) * rank + 64 * c, row0 + (kt0 + t) * BN + 64 * r64);
+                             v_col + (HD / NB) * rank + 64 * c, row0 + tile_at(kt0 + t) * BN + 64 * r64);
                 return true;
             };
             bool fed = nt == 0 || load_k(0);
@@ -581,15 +592,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
             tmem_ld_wait();
             // Which of the thread's 64 keys the row sees: j in [j_lo, j_hi].  A warp whose
             // rows all see all of them takes the path without the mask.
-            const int key0 = (kt0 + t) * BN + 64 * half;
+            const int key0 = tile_at(kt0 + t) * BN + 64 * half;
             const int j_hi = min(pos, n - 1) - key0;
             const int j_lo = p.window > 0 ? pos - p.window + 1 - key0 : -(1 << 30);
-            const bool whole = __all_sync(0xffffffffu, j_lo <= 0 && j_hi >= 63);
+            const int j_keep = p.keep - key0;          // (the same for a whole warp)
+            const bool whole = __all_sync(0xffffffffu, (j_lo <= 0 || j_keep >= 64) && j_hi >= 63);
             // The row's maximum, taken on the raw products: scaling by a positive factor and
             // the cap are both increasing, so the largest product gives the largest score.
             float mx_raw, other;
-            if (whole) mx_raw = row_max<false>(raw, j_lo, j_hi);
-            else mx_raw = row_max<true>(raw, j_lo, j_hi);
+            if (whole) mx_raw = row_max<0>(raw, j_lo, j_hi);
+            else if (j_keep > 0) mx_raw = row_max<2>(raw, j_lo, j_hi, j_keep);
+            else mx_raw = row_max<1>(raw, j_lo, j_hi);
             if (!swap_with_partner(t, mx_raw, other)) { if (lane == 0) *failed = 9; ok = false; break; }
             mx_raw = fmaxf(mx_raw, other);
             float mx = mx_raw * c1;
@@ -623,11 +636,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
             }
             const float ref = m_ref == -INFINITY ? 0.f : m_ref;
             if (capped) {
-                if (whole) l += probabilities<true, false>(raw, c1, c2, ref, j_lo, j_hi);
-                else l += probabilities<true, true>(raw, c1, c2, ref, j_lo, j_hi);
+                if (whole) l += probabilities<true, 0>(raw, c1, c2, ref, j_lo, j_hi);
+                else l += probabilities<true, 1>(raw, c1, c2, ref, j_lo, j_hi);
             } else {
-                if (whole) l += probabilities<false, false>(raw, c1, c2, ref, j_lo, j_hi);
-                else l += probabilities<false, true>(raw, c1, c2, ref, j_lo, j_hi);
+                if (whole) l += probabilities<false, 0>(raw, c1, c2, ref, j_lo, j_hi);
+                else if (j_keep > 0) l += probabilities<false, 2>(raw, c1, c2, ref, j_lo, j_hi, j_keep);
+                else l += probabilities<false, 1>(raw, c1, c2, ref, j_lo, j_hi);
             }
             // P over the first 64 columns of the score tile (both threads have read theirs)
             tmem_st32(s_addr + 32 * half, reinterpret_cast<uint32_t(&)[32]>(raw));
@@ -893,12 +907,12 @@ float plan_for(const std::vector<PlanBlock>& blocks, int n_kv, int split_from, i
 }
 
 bool plan_items_now(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, int head_dim,
-                    int window, int sms, TcItems* out, int* n_units);
+                    int window, int keep, int sms, TcItems* out, int* n_units);
 
 // Fills `out` for prompts of `lens` (host memory); false if a list does not fit or pay.
 // (Every layer of a step asks for the same few plans: the last ones are kept.)
 bool plan_items(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, int head_dim,
-                int window, int sms, TcItems* out, int* n_units) {
+                int window, int keep, int sms, TcItems* out, int* n_units) {
     struct Kept {
         std::vector<int> key;
         TcItems items;
@@ -910,8 +924,8 @@ bool plan_items(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, in
     if (!lens || n_seqs <= 0) return false;
     std::vector<int> key(lens, lens + n_seqs);
     for (int b = 0; b < n_seqs; ++b) key.push_back(q0s ? q0s[b] : 0);
-    const int tail[6] = {n_kv, G, head_dim, window, sms, tc_pairs_allowed() ? 1 : 0};
-    key.insert(key.end(), tail, tail + 6);
+    const int tail[7] = {n_kv, G, head_dim, window, keep, sms, tc_pairs_allowed() ? 1 : 0};
+    key.insert(key.end(), tail, tail + 7);
     for (Kept& k : kept)
         if (k.key == key) {
             if (k.ok) {
@@ -924,7 +938,7 @@ bool plan_items(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, in
     next = (next + 1) % 4;
     k.key = key;
     k.units = 0;
-    k.ok = plan_items_now(lens, q0s, n_seqs, n_kv, G, head_dim, window, sms, &k.items, &k.units);
+    k.ok = plan_items_now(lens, q0s, n_seqs, n_kv, G, head_dim, window, keep, sms, &k.items, &k.units);
     if (k.ok) {
         *out = k.items;
         if (n_units) *n_units = k.units;
@@ -933,7 +947,7 @@ bool plan_items(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, in
 }
 
 bool plan_items_now(const int* lens, const int* q0s, int n_seqs, int n_kv, int G, int head_dim,
-                    int window, int sms, TcItems* out, int* n_units) {
+                    int window, int keep, int sms, TcItems* out, int* n_units) {
     static const bool allowed = [] {
         const char* v = getenv("SIB_PREFILL_BALANCE");
         return !(v && v[0] == '0');
@@ -951,7 +965,10 @@ bool plan_items_now(const int* lens, const int* q0s, int n_seqs, int n_kv, int G
             if (q >= 4096 || (long long)(blocks.size() + 1) * n_kv > MAX_ITEMS) return false;
             const int first0 = q * span, k_hi = std::min(n, first0 + span);
             const int k_lo = window > 0 ? std::max(0, first0 - window + 1) : 0;
-            const int nt = (k_hi + BN - 1) / BN - k_lo / BN;
+            // (as the kernel counts them: the tiles of kept first positions, then the window's)
+            const int kept_tiles = (kept_before(k_lo, keep) + BN - 1) / BN;
+            const int skip = std::max(k_lo / BN, kept_tiles) - kept_tiles;
+            const int nt = std::max((k_hi + BN - 1) / BN - skip, kept_tiles);
             blocks.push_back({b, q, nt});
             nt_max = std::max(nt_max, nt);
         }
@@ -995,14 +1012,14 @@ int device_sms() {
 // of work items: bytes of scratch memory and ticket counters (int, zero between launches)
 // for the blocks it splits.  Returns the number of items, 0 if such a launch is a grid.
 SIB_EXPORT int sib_attention_prefill_tc_plan(const int* host_lens, const int* host_q0, int n_seqs,
-                                             int n_heads, int n_kv, int head_dim, int window,
+                                             int n_heads, int n_kv, int head_dim, int window, int keep,
                                              long long* scratch_bytes, int* n_tickets) {
     if (scratch_bytes) *scratch_bytes = 0;
     if (n_tickets) *n_tickets = 0;
     if (n_kv <= 0 || n_heads % n_kv) return 0;
     TcItems items;
     int units = 0;
-    if (!plan_items(host_lens, host_q0, n_seqs, n_kv, n_heads / n_kv, head_dim, window, device_sms(),
+    if (!plan_items(host_lens, host_q0, n_seqs, n_kv, n_heads / n_kv, head_dim, window, keep, device_sms(),
                     &items, &units))
         return 0;
     const int nb = (head_dim >= 128 && tc_pairs_allowed()) ? 2 : 1;
@@ -1055,11 +1072,14 @@ SIB_EXPORT int sib_attention_prefill_tc(const void* qkv, int width, int total_ro
                                         float scale, float softcap, int window, void* scratch,
                                         long long scratch_bytes, int* tickets, int n_tickets,
                                         const int* host_lens, const int* seq_q0, const int* host_q0,
-                                        const float* sink, const float* extra, void* stream) {
+                                        const float* sink, const float* extra, int keep, void* stream) {
     if (n_seqs == 0 || max_len == 0) return 0;
     SIB_REQUIRE(sink == nullptr || softcap == 0.f, "attention_prefill_tc: a sink together with a cap is not built");
     SIB_REQUIRE(extra == nullptr || (softcap == 0.f && sink == nullptr && ((uintptr_t)extra % 4) == 0),
                 "attention_prefill_tc: another kernel's partial results go with no cap and no sink");
+    SIB_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && softcap == 0.f)),
+                "attention_prefill_tc: keep=%d with window=%d and cap=%g (kept first positions go with a "
+                "window and without a cap)", keep, window, (double)softcap);
     SIB_REQUIRE(sib_attention_prefill_tc_supports(n_heads, n_kv, head_dim, width),
                 "attention_prefill_tc: heads=%d kv_heads=%d head_dim=%d is not a shape this kernel "
                 "takes (1 or 2 heads per kv head; head_dim 64, 128 or 256)", n_heads, n_kv, head_dim);
@@ -1103,8 +1123,8 @@ SIB_EXPORT int sib_attention_prefill_tc(const void* qkv, int width, int total_ro
     items.n = 0;
     if (host_lens) {
         int units = 0;
-        if (plan_items(host_lens, host_q0, n_seqs, n_kv, G, head_dim, window, device_sms(), &items,
-                       &units)) {
+        if (plan_items(host_lens, host_q0, n_seqs, n_kv, G, head_dim, window, keep, device_sms(),
+                       &items, &units)) {
             const int nb = (head_dim >= 128 && tc_pairs_allowed()) ? 2 : 1;
             const long long bytes = (long long)units * nb * 2 * (long long)BM * (head_dim + 2) * sizeof(float);
             if (units > 0 && (scratch == nullptr || tickets == nullptr || scratch_bytes < bytes ||
@@ -1116,7 +1136,7 @@ SIB_EXPORT int sib_attention_prefill_tc(const void* qkv, int width, int total_ro
     }
     if (items.n > 0) split_tiles = 0;
     TcArgs p{(__nv_bfloat16*)out, seq_row0, seq_len, seq_q0, error_flag, (float*)scratch, tickets,
-             split_tiles, n_heads, n_kv, window, scale, softcap, sink, extra};
+             split_tiles, n_heads, n_kv, window, keep, scale, softcap, sink, extra};
     cudaStream_t s = (cudaStream_t)stream;
 #define BY_G(HD, PAIR)                                                         \
     do {                                                                       \

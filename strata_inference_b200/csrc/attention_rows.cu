@@ -6,6 +6,7 @@
 // (key/value head g = h / (n_heads / n_kv)):
 //     s_j = scale * <q_h, k_{g,j}>;  if cap > 0: s_j = cap * tanh(s_j / cap)
 //     visible j: max(0, p - window + 1) <= j <= p   (window 0: all j <= p)
+//     and, with `keep` > 0 (and a window), every j < keep: the sequence's first tokens, kept for good
 //     with `chunk` > 0 instead: p - p % chunk <= j <= p   (the row's own chunk of positions)
 //     o = sum_j softmax(s)_j v_{g,j}
 // With a sink (one number per query head) the softmax's denominator has one more term,
@@ -47,7 +48,9 @@ struct AttnRowsArgs {
     int q_stride, kv_stride;
     int rows, n_heads, n_kv, head_dim;
     int max_pages, page_tokens, ring_tokens;
+    int fixed_tokens;       // positions ahead of the ring (common.cuh cell_of)
     int window, splits;
+    int keep;               // > 0 (with a window): the first `keep` positions stay visible
     int chunk;              // > 0: a row sees its own chunk of positions (first_visible)
     float scale, softcap;
     const float* sink;      // [n_heads] or null
@@ -89,7 +92,7 @@ __device__ __forceinline__ const T* key_ptr(const AttnRowsArgs& p, const T* fres
                                             int j, int start, int row0, int slot, int g) {
     if (fresh && j >= start)
         return fresh + (size_t)(row0 + (j - start)) * p.kv_stride + (size_t)g * p.head_dim;
-    const int cell = p.ring_tokens > 0 ? j % p.ring_tokens : j;
+    const int cell = cell_of(j, p.fixed_tokens, p.ring_tokens);
     const int page = p.page_table[(size_t)slot * p.max_pages + cell / p.page_tokens];
     return pool + (((size_t)page * p.n_kv + g) * p.page_tokens + cell % p.page_tokens) * p.head_dim;
 }
@@ -124,9 +127,11 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttnRowsArgs p) {
     const int start = p.seq_start[b];
     const int row0 = p.seq_row0[b];
     const int lo = first_visible(pos, p.window, p.chunk);
-    const int nb = p.pk_pool && p.window > 0 && slot >= 0 ? max(0, pos - p.window + 1) / p.pool : 0;
+    const int nb = p.keep > 0 ? kept_before(lo, p.keep)
+                   : p.pk_pool && p.window > 0 && slot >= 0 ? max(0, pos - p.window + 1) / p.pool : 0;
     const int last = p.cells_only ? lo - 1 : pos;
-    const int n = nb + last - lo + 1;          // keys are numbered lo - nb .. pos: blocks first
+    // keys are numbered lo - nb .. pos: blocks (or the kept first positions) first
+    const int n = nb + last - lo + 1;
     const int chunk = (n + p.splits - 1) / p.splits;
     const int j0 = lo - nb + split * chunk;
     const int j1 = min(j0 + chunk, last + 1);
@@ -156,8 +161,10 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttnRowsArgs p) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (j + u < j1) {
-                const T* kp = j + u < lo ? cell_ptr<T>(p, (const T*)p.pk_pool, j + u - (lo - nb), slot, g)
-                                         : key_ptr<T>(p, kf, kpool, j + u, start, row0, slot, g);
+                const int at = j + u < lo && p.keep > 0 ? j + u - (lo - nb) : j + u;
+                const T* kp = j + u < lo && p.keep <= 0
+                                  ? cell_ptr<T>(p, (const T*)p.pk_pool, j + u - (lo - nb), slot, g)
+                                  : key_ptr<T>(p, kf, kpool, at, start, row0, slot, g);
 #pragma unroll
                 for (int i = 0; i < NI; ++i)
                     if (live[i]) Vec16<T>::load(kp + (lane + 32 * i) * V, kv[u][i]);
@@ -203,8 +210,10 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttnRowsArgs p) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (j + u < j1 && !p.values_in_keys) {
-                const T* vp = j + u < lo ? cell_ptr<T>(p, (const T*)p.pv_pool, j + u - (lo - nb), slot, g)
-                                         : key_ptr<T>(p, vf, vpool, j + u, start, row0, slot, g);
+                const int at = j + u < lo && p.keep > 0 ? j + u - (lo - nb) : j + u;
+                const T* vp = j + u < lo && p.keep <= 0
+                                  ? cell_ptr<T>(p, (const T*)p.pv_pool, j + u - (lo - nb), slot, g)
+                                  : key_ptr<T>(p, vf, vpool, at, start, row0, slot, g);
 #pragma unroll
                 for (int i = 0; i < NI; ++i)
                     if (live[i]) Vec16<T>::load(vp + (lane + 32 * i) * V, kv[u][i]);
@@ -364,7 +373,7 @@ SIB_EXPORT int sib_attention_rows(
     int n_heads, int n_kv, int head_dim, float scale, float softcap, int window, int chunk,
     int splits, const float* sink, int values_in_keys, const void* pk_pool, const void* pv_pool,
     const int* pool_table, int pool, int pool_max_pages, int pool_page_tokens, int cells_only,
-    void* stream) {
+    int keep, int fixed_tokens, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(!cells_only || (pk_pool != nullptr && partial != nullptr && splits == 1 && sink == nullptr),
                 "attention_rows: the blocks alone need their cache, room for the results and one split");
@@ -386,6 +395,10 @@ SIB_EXPORT int sib_attention_rows(
     SIB_REQUIRE(window >= 0 && ring_tokens >= 0 && chunk >= 0 && (chunk == 0 || (window == 0 && !pk_pool)),
                 "attention_rows: window=%d ring=%d chunk=%d (a chunk goes without a window)", window,
                 ring_tokens, chunk);
+    SIB_REQUIRE(keep >= 0 && fixed_tokens >= 0 && (keep == 0 || (window > 0 && !pk_pool)) &&
+                    (ring_tokens == 0 || fixed_tokens >= keep),
+                "attention_rows: keep=%d with window=%d (kept positions go with a window and without "
+                "pooled blocks, and lie in the %d fixed cells)", keep, window, fixed_tokens);
     const int esz = dtype == SIB_F32 ? 4 : 2;
     SIB_REQUIRE(((size_t)q_stride * esz) % 16 == 0 && ((size_t)kv_stride * esz) % 16 == 0 &&
                     ((uintptr_t)q % 16) == 0 && ((uintptr_t)k_new % 16) == 0 &&
@@ -394,7 +407,8 @@ SIB_EXPORT int sib_attention_rows(
                 "attention_rows: rows must start on 16-byte boundaries");
     AttnRowsArgs p{q, k_new, v_new, k_pool, v_pool, out, partial, row_pos, row_seq, seq_slot,
                    seq_start, seq_row0, page_table, q_stride, kv_stride, rows, n_heads, n_kv,
-                   head_dim, max_pages, page_tokens, ring_tokens, window, splits, chunk, scale, softcap,
+                   head_dim, max_pages, page_tokens, ring_tokens, fixed_tokens, window, splits, keep, chunk, scale,
+                   softcap,
                    sink, values_in_keys, pk_pool, pv_pool, pool_table, pool, pool_max_pages,
                    pool_page_tokens, cells_only};
     const long long units = (long long)rows * n_heads * splits;

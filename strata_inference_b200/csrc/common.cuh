@@ -105,6 +105,22 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int window, int c
     return window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
 }
 
+// A window that also keeps the sequence's first `keep` positions: how many of them lie ahead of
+// the window's first position `lo` (the ones at `lo` and later are the window's own).
+__host__ __device__ __forceinline__ int kept_before(int lo, int keep) { return keep < lo ? keep : lo; }
+
+// The cache cell of a position.  A ring of `ring` positions (> 0) begins behind `fixed` cells that
+// are never overwritten: positions below `fixed` lie there, later ones wrap around in the ring.
+// ring 0: position p lies in cell p.
+__host__ __device__ __forceinline__ int cell_of(int pos, int fixed, int ring) {
+    return ring > 0 && pos >= fixed ? fixed + (pos - fixed) % ring : pos;
+}
+// Whether a step that leaves its sequence `end` long writes the position (a later row of the same
+// step owns the cell otherwise).
+__host__ __device__ __forceinline__ bool cell_written(int pos, int end, int fixed, int ring) {
+    return ring <= 0 || pos < fixed || pos >= end - ring;
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.
 // `scratch` holds 33 floats of shared memory and may be reused after return.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {

@@ -3,9 +3,12 @@
 //
 //   head_prepare   per row and head, in 32-bit:
 //       x  = proj + bias                                   (bias optional)
-//       q, k: x <- x / sqrt(mean(x^2) + eps) * w           (w optional: no norm without it)
+//       q, k: x <- x / sqrt(mean(x^2) + eps) * w           (with weights; NORM_BEFORE)
 //       q, k: the first `rot` dimensions rotated in half-split pairs (i, i + rot/2), or in
-//             neighbouring pairs (2i, 2i + 1), by the angle pos * inv_freq[i]; the rest pass
+//             neighbouring pairs (2i, 2i + 1), by the angle pos * inv_freq[i], cosine and sine
+//             both times `magnitude`; the rest pass
+//       q, k: x <- x / sqrt(mean(x^2) + eps)               (without weights; NORM_AFTER)
+//       q:    x <- x * temp[head]                          (temp optional)
 //       v:    v <- (1 - lambda) v + lambda v_first         (v_first optional)
 //     q, k and v go to a packed buffer whose heads are all `pad` wide (key width and value
 //     width may differ: the narrower one is filled up with zeros, which changes neither a
@@ -16,6 +19,8 @@
 //
 // Plain counterpart: tests/plain_karupel.py attention_mixer().
 #include "common.cuh"
+
+enum { NORM_NONE = 0, NORM_BEFORE = 1, NORM_AFTER = 2 };   // where q and k are normed: the rotation's side
 
 struct HeadPrepareArgs {
     const void* proj;          // [rows, proj_stride]: q heads | k heads | v heads | ...
@@ -37,6 +42,10 @@ struct HeadPrepareArgs {
     int n_heads, n_kv, kd, vd, pad, rot, v_first_pad;
     int max_pages, page_tokens, ring_tokens;
     float eps;
+    int norm;                  // NORM_NONE, NORM_BEFORE or NORM_AFTER
+    const float* temp;         // [n_heads] or null: a factor on each query head
+    float magnitude;           // of the rotation
+    int fixed_tokens;          // positions ahead of the ring (common.cuh cell_of)
     int neighbours;            // 1: the rotated pairs are (2i, 2i + 1) instead of (i, i + rot/2)
 };
 
@@ -65,9 +74,9 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(HeadPrepareArgs p) {
         const int slot = p.seq_slot[b];
         bool keep = slot >= 0;               // (a filling row's sequence holds no slot)
         int cell = pos;
-        if (keep && p.ring_tokens > 0) {
-            keep = pos >= p.seq_end[b] - p.ring_tokens;
-            cell = pos % p.ring_tokens;
+        if (keep) {
+            keep = cell_written(pos, p.seq_end[b], p.fixed_tokens, p.ring_tokens);
+            cell = cell_of(pos, p.fixed_tokens, p.ring_tokens);
         }
         if (keep) {
             const int page = p.page_table[(size_t)slot * p.max_pages + cell / p.page_tokens];
@@ -103,30 +112,37 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(HeadPrepareArgs p) {
         }
         return;
     }
-    const float* gain = is_q ? p.q_gain : p.k_gain;
-    float inv = 1.f;
-    if (gain) inv = 1.0f / sqrtf(warp_sum(ss) / (float)width + p.eps);
-    __syncwarp();
-    if (gain)
+    if (p.norm == NORM_BEFORE) {
+        const float* gain = is_q ? p.q_gain : p.k_gain;
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)width + p.eps);
+        __syncwarp();
         for (int d = lane; d < width; d += 32) mine[d] = mine[d] * inv * gain[d];
+    }
     __syncwarp();
+    float factor = p.temp && is_q ? p.temp[unit] : 1.f;
     const int half = p.inv_freq ? p.rot / 2 : 0;
-    for (int d = lane; d < p.pad; d += 32) {
-        float x = 0.f;
-        if (d < width) {
-            x = mine[d];
-            if (d < 2 * half && p.neighbours) {
-                const float ang = (float)pos * p.inv_freq[d >> 1];
-                const float c = cosf(ang), s = sinf(ang);
-                x = (d & 1) ? x * c + mine[d - 1] * s : x * c - mine[d + 1] * s;
-            } else if (d < 2 * half) {
-                const int i = d < half ? d : d - half;
-                const float ang = (float)pos * p.inv_freq[i];
-                const float c = cosf(ang), s = sinf(ang);
-                x = d < half ? x * c - mine[d + half] * s : x * c + mine[d - half] * s;
-            }
+    auto rotated = [&](int d) {
+        float x = mine[d];
+        if (d < 2 * half) {
+            const int i = p.neighbours ? d >> 1 : (d < half ? d : d - half);
+            const bool first = p.neighbours ? !(d & 1) : d < half;
+            const int other = p.neighbours ? d ^ 1 : (d < half ? d + half : d - half);
+            const float ang = (float)pos * p.inv_freq[i];
+            const float c = cosf(ang) * p.magnitude, s = sinf(ang) * p.magnitude;
+            x = first ? x * c - mine[other] * s : x * c + mine[other] * s;
         }
-        const T y = from_f32<T>(x);
+        return x;
+    };
+    if (p.norm == NORM_AFTER) {
+        float sr = 0.f;
+        for (int d = lane; d < width; d += 32) {
+            const float x = rotated(d);
+            sr += x * x;
+        }
+        factor *= 1.0f / sqrtf(warp_sum(sr) / (float)width + p.eps);
+    }
+    for (int d = lane; d < p.pad; d += 32) {
+        const T y = from_f32<T>(d < width ? rotated(d) * factor : 0.f);
         out[d] = y;
         if (dst) dst[d] = y;
     }
@@ -138,7 +154,8 @@ SIB_EXPORT int sib_head_prepare(
     const void* v_first, long long v_first_stride, int v_first_pad, const float* lambda, const int* row_pos,
     const int* row_seq, const int* seq_slot, const int* seq_end, void* k_pool, void* v_pool,
     const int* page_table, int max_pages, int page_tokens, int ring_tokens, int rows, int n_heads,
-    int n_kv, int kd, int vd, int pad, int neighbours, void* stream) {
+    int n_kv, int kd, int vd, int pad, int neighbours, int norm_after, const float* temp, float magnitude,
+    int fixed_tokens, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && n_heads > 0 && n_kv >= 0 && kd > 0 && vd > 0,
                 "head_prepare: rows=%d heads=%d kv_heads=%d key width=%d value width=%d", rows,
@@ -153,10 +170,14 @@ SIB_EXPORT int sib_head_prepare(
                 "head_prepare: incomplete cache description");
     SIB_REQUIRE(v_first == nullptr || (lambda != nullptr && v_first_pad >= vd),
                 "head_prepare: mixing values needs lambda and heads of at least %d", vd);
+    SIB_REQUIRE((q_gain != nullptr) == (k_gain != nullptr) && !(norm_after && q_gain) && fixed_tokens >= 0,
+                "head_prepare: q and k are normed together, with weights before the rotation or without "
+                "them behind it");
     HeadPrepareArgs p{proj, qkv, bias, q_gain, k_gain, rot ? inv_freq : nullptr, v_first, lambda,
                       row_pos, row_seq, seq_slot, seq_end, k_pool, v_pool, page_table, proj_stride,
                       v_first_stride, n_heads, n_kv, kd, vd, pad, rot, v_first_pad, max_pages, page_tokens,
-                      ring_tokens, eps, neighbours};
+                      ring_tokens, eps, norm_after ? NORM_AFTER : (q_gain ? NORM_BEFORE : NORM_NONE), temp,
+                      magnitude, fixed_tokens, neighbours};
     const int units = n_heads + 2 * n_kv;
     const size_t smem = (size_t)4 * pad * sizeof(float);
     SIB_REQUIRE(smem <= 48 * 1024, "head_prepare: heads of %d are too wide", pad);

@@ -235,7 +235,7 @@ struct GatherArgs {
     const int* seq_upto;       // [seqs] one past the last
     const int* seq_row0;       // [seqs] packed row of the sequence's position 0
     int n_heads, n_kv, head_dim;
-    int max_pages, page_tokens, ring_tokens;
+    int max_pages, page_tokens, ring_tokens, fixed_tokens;
 };
 
 __global__ void __launch_bounds__(128) gather_kv_rows_kernel(GatherArgs p) {
@@ -246,7 +246,7 @@ __global__ void __launch_bounds__(128) gather_kv_rows_kernel(GatherArgs p) {
     if (pos >= p.seq_upto[b]) return;
     const int hd = p.head_dim;
     const int width = (p.n_heads + 2 * p.n_kv) * hd;
-    const int cell = p.ring_tokens > 0 ? pos % p.ring_tokens : pos;
+    const int cell = cell_of(pos, p.fixed_tokens, p.ring_tokens);
     const int page = p.page_table[(size_t)p.seq_slot[b] * p.max_pages + cell / p.page_tokens];
     __nv_bfloat16* row = p.packed + (size_t)(p.seq_row0[b] + pos) * width;
     const int per_head = hd / 8;                 // 16-byte pieces of a head
@@ -269,21 +269,21 @@ SIB_EXPORT int sib_gather_kv_rows(void* packed, const void* k_pool, const void* 
                                   const int* page_table, const int* seq_slot, const int* seq_from,
                                   const int* seq_upto, const int* seq_row0, int n_seqs, int most,
                                   int n_heads, int n_kv, int head_dim, int max_pages,
-                                  int page_tokens, int ring_tokens, void* stream) {
+                                  int page_tokens, int ring_tokens, int fixed_tokens, void* stream) {
     if (n_seqs == 0 || most <= 0) return 0;
     SIB_REQUIRE(n_seqs > 0 && n_seqs < 65536 && n_heads > 0 && n_kv > 0 && head_dim > 0 &&
                     head_dim % 8 == 0,
                 "gather_kv_rows: seqs=%d heads=%d kv=%d head_dim=%d (a multiple of 8)", n_seqs, n_heads,
                 n_kv, head_dim);
     SIB_REQUIRE(packed && k_pool && v_pool && page_table && seq_slot && seq_from && seq_upto && seq_row0 &&
-                    page_tokens > 0 && max_pages > 0 && ring_tokens >= 0,
+                    page_tokens > 0 && max_pages > 0 && ring_tokens >= 0 && fixed_tokens >= 0,
                 "gather_kv_rows: incomplete description");
     SIB_REQUIRE(((uintptr_t)packed % 16) == 0 && ((uintptr_t)k_pool % 16) == 0 &&
                     ((uintptr_t)v_pool % 16) == 0,
                 "gather_kv_rows: buffers must be 16-byte aligned");
     GatherArgs p{(__nv_bfloat16*)packed, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
                  page_table, seq_slot, seq_from, seq_upto, seq_row0, n_heads, n_kv, head_dim,
-                 max_pages, page_tokens, ring_tokens};
+                 max_pages, page_tokens, ring_tokens, fixed_tokens};
     sib_launch_chained(gather_kv_rows_kernel, dim3(most, n_seqs), dim3(128), 0, (cudaStream_t)stream, p);
     return sib_check_launch("gather_kv_rows");
 }

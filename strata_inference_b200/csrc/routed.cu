@@ -16,13 +16,20 @@
 //                    from the pairs' outputs, found through the sort's inverse.
 //
 // Two things are parameters of every entry.  `score`: what a chosen expert's weight is,
-// SCORE_SOFTMAX_TOP (the softmax over the chosen logits alone) or SCORE_SIGMOID (the sigmoid of
-// the expert's own logit, not normalized).  `form`: what an expert computes, FORM_CLIPPED_GATED
-// (above; matrices [2 ff, width]) or FORM_PLAIN_GELU, down(gelu(w * up x)) with the exact gelu,
+// SCORE_SOFTMAX_TOP (the softmax over the chosen logits alone), SCORE_SIGMOID (the sigmoid of
+// the expert's own logit, not normalized) or SCORE_SOFTMAX_ALL (the softmax over ALL experts'
+// logits; the bias is then added to these scores for the choice only, and the weight is the
+// score without it times `scale`, not normalized).  `form`: what an expert computes,
+// FORM_CLIPPED_GATED (above; matrices [2 ff, width]), FORM_GATED_SILU, down(silu(gate) * up) with
+// matrices of the same layout, or FORM_PLAIN_GELU, down(gelu(w * up x)) with the exact gelu,
 // matrices [ff, width], where the pair's weight w multiplies what ENTERS the expert (it has no
 // bias, so w * (up x) = up (w x)) and the pairs' outputs are summed as they are.
+// The router's matrix may hold one row more than there are experts: its product with a row is
+// the logit of a gate, sigmoid(z[experts]), written to `gate` [rows], and the base row (a shared
+// expert's output) is multiplied by it where the pairs are summed (`base_weight`), in 32-bit.
 //
-// Plain counterpart: tests/plain_gegorax.py routed_ff(), expert().
+// Plain counterparts: tests/plain_gegorax.py routed_ff(), expert(); tests/plain_kerolorn.py
+// router_choice(), routed_ff().
 #include "common.cuh"
 
 namespace {
@@ -34,22 +41,36 @@ __device__ __forceinline__ float expert_act(float g, float u, float limit, float
     return g * sigmoid_r(alpha * g) * (u + 1.0f);
 }
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
-constexpr int SCORE_SOFTMAX_TOP = 0, SCORE_SIGMOID = 1;
-constexpr int FORM_CLIPPED_GATED = 0, FORM_PLAIN_GELU = 1;
+constexpr int SCORE_SOFTMAX_TOP = 0, SCORE_SIGMOID = 1, SCORE_SOFTMAX_ALL = 2;
+constexpr int FORM_CLIPPED_GATED = 0, FORM_PLAIN_GELU = 1, FORM_GATED_SILU = 2;
+__device__ __forceinline__ float gated_act(float g, float u, float limit, float alpha, int form) {
+    return form == FORM_GATED_SILU ? g * sigmoid_r(g) * u : expert_act(g, u, limit, alpha);
+}
 
 // One warp: the `top` largest of z[e] + bias[e] in order (ties: the lower index) and their
-// weights: the softmax over them alone, or each one's own sigmoid.
+// weights: the softmax over them alone, each one's own sigmoid, or (SCORE_SOFTMAX_ALL, where the
+// softmax over all experts stands in z's place) the score without the bias, times `scale`.
 __device__ __forceinline__ void choose_top(const float* z, const float* __restrict__ bias,
                                            int* __restrict__ ids, float* __restrict__ weights,
-                                           int experts, int top, int lane, int score) {
+                                           int experts, int top, int lane, int score, float scale) {
     float first = 0.f, sum = 0.f;
+    float z_max = 0.f, z_sum = 1.f;
+    if (score == SCORE_SOFTMAX_ALL) {
+        z_max = -INFINITY;
+        for (int e = lane; e < experts; e += 32) z_max = fmaxf(z_max, z[e]);
+        z_max = warp_max(z_max);
+        z_sum = 0.f;
+        for (int e = lane; e < experts; e += 32) z_sum += expf(z[e] - z_max);
+        z_sum = warp_sum(z_sum);
+    }
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;
         for (int e = lane; e < experts; e += 32) {
             bool taken = false;
             for (int j = 0; j < k; ++j) taken |= ids[j] == e;
-            const float v = z[e] + (bias ? bias[e] : 0.f);
+            const float s = score == SCORE_SOFTMAX_ALL ? expf(z[e] - z_max) / z_sum : z[e];
+            const float v = s + (bias ? bias[e] : 0.f);
             if (!taken && (v > best || (v == best && e < at))) { best = v; at = e; }
         }
 #pragma unroll
@@ -60,7 +81,9 @@ __device__ __forceinline__ void choose_top(const float* z, const float* __restri
         }
         if (k == 0) first = best;
         // (the first chosen logit is the largest)
-        const float w = score == SCORE_SIGMOID ? sigmoid_r(best) : expf(best - first);
+        const float w = score == SCORE_SOFTMAX_ALL ? scale * (expf(z[at] - z_max) / z_sum)
+                        : score == SCORE_SIGMOID   ? sigmoid_r(best)
+                                                   : expf(best - first);
         sum += w;
         if (lane == 0) {
             ids[k] = at;
@@ -73,16 +96,17 @@ __device__ __forceinline__ void choose_top(const float* z, const float* __restri
 
 // One warp per row.
 __global__ void __launch_bounds__(128)
-router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
-                   int* __restrict__ ids, float* __restrict__ weights, int rows, int experts, int top,
-                   int score) {
+router_topk_kernel(const float* __restrict__ logits, int stride, const float* __restrict__ bias,
+                   int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ gate, int rows,
+                   int experts, int top, int score, float scale) {
     pdl_trigger();
     pdl_wait();
     const int lane = threadIdx.x & 31;
     const int r = blockIdx.x * 4 + (threadIdx.x >> 5);
     if (r >= rows) return;
-    choose_top(logits + (size_t)r * experts, bias, ids + (size_t)r * top, weights + (size_t)r * top,
-               experts, top, lane, score);
+    const float* z = logits + (size_t)r * stride;
+    if (gate && lane == 0) gate[r] = sigmoid_r(z[experts]);
+    choose_top(z, bias, ids + (size_t)r * top, weights + (size_t)r * top, experts, top, lane, score, scale);
 }
 
 // Few rows: the router's product and the choice in one launch.  One block per row: the row in
@@ -92,8 +116,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 router_rows_kernel(const T* __restrict__ x, long long x_stride, const float* __restrict__ w,
                    const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights,
-                   int width, int experts, int top, int score) {
-    extern __shared__ __align__(16) float sh[];      // [width] the row, [experts] its logits
+                   float* __restrict__ gate, int width, int experts, int top, int score, float scale) {
+    extern __shared__ __align__(16) float sh[];      // [width] the row, [experts (+ the gate's)] its logits
     float* xs = sh;
     float* z = sh + ((width + 3) & ~3);
     pdl_trigger();
@@ -103,7 +127,7 @@ router_rows_kernel(const T* __restrict__ x, long long x_stride, const float* __r
     for (int c = threadIdx.x; c < width; c += blockDim.x) xs[c] = to_f32(x[(size_t)r * x_stride + c]);
     __syncthreads();
     const bool wide = width % 4 == 0 && ((uintptr_t)w % 16) == 0;
-    for (int e = warp; e < experts; e += blockDim.x >> 5) {
+    for (int e = warp; e < experts + (gate ? 1 : 0); e += blockDim.x >> 5) {
         const float* row = w + (size_t)e * width;
         float acc = 0.f;
         if (wide) {
@@ -118,8 +142,9 @@ router_rows_kernel(const T* __restrict__ x, long long x_stride, const float* __r
         if (lane == 0) z[e] = acc;
     }
     __syncthreads();
+    if (gate && threadIdx.x == 0) gate[r] = sigmoid_r(z[experts]);
     if (warp == 0)
-        choose_top(z, bias, ids + (size_t)r * top, weights + (size_t)r * top, experts, top, lane, score);
+        choose_top(z, bias, ids + (size_t)r * top, weights + (size_t)r * top, experts, top, lane, score, scale);
 }
 
 // `group` 8: gate and up columns lie interleaved in eights (8 gates, then their 8 ups), as the
@@ -168,7 +193,7 @@ __global__ void expert_activate_kernel(const T* __restrict__ gu, long long strid
             v = gelu_erf(to_f32(gu[r * stride + j]) * (row_weight ? row_weight[r] : 1.0f));
         } else {
             const size_t g = group ? (size_t)(j / group) * 2 * group + j % group : (size_t)j;
-            v = expert_act(to_f32(gu[r * stride + g]), to_f32(gu[r * stride + g + (group ? group : ff)]), limit, alpha);
+            v = gated_act(to_f32(gu[r * stride + g]), to_f32(gu[r * stride + g + (group ? group : ff)]), limit, alpha, form);
             if (row_weight) v *= row_weight[r];
         }
         y[i] = from_f32<T>(v);
@@ -204,9 +229,9 @@ __global__ void expert_activate8_kernel(const __nv_bfloat16* __restrict__ gu, lo
             const uint32_t wa[4] = {a.x, a.y, a.z, a.w}, wb[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                o[2 * e] = expert_act(__uint_as_float(wa[e] << 16), __uint_as_float(wb[e] << 16), limit, alpha) * rw;
-                o[2 * e + 1] = expert_act(__uint_as_float(wa[e] & 0xffff0000u), __uint_as_float(wb[e] & 0xffff0000u),
-                                          limit, alpha) * rw;
+                o[2 * e] = gated_act(__uint_as_float(wa[e] << 16), __uint_as_float(wb[e] << 16), limit, alpha, form) * rw;
+                o[2 * e + 1] = gated_act(__uint_as_float(wa[e] & 0xffff0000u), __uint_as_float(wb[e] & 0xffff0000u),
+                                         limit, alpha, form) * rw;
             }
         }
         uint4 out;
@@ -285,7 +310,7 @@ template <typename T, bool PLAIN>
 __global__ void __launch_bounds__(128)
 routed_rows_gate_up_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ w_gu,
                            const int* __restrict__ ids, const float* __restrict__ pair_weight,
-                           T* __restrict__ mid, int width, int ff, int top, float limit, float alpha) {
+                           T* __restrict__ mid, int width, int ff, int top, float limit, float alpha, int form) {
     extern __shared__ __align__(16) float xs[];
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -321,8 +346,8 @@ routed_rows_gate_up_kernel(const T* __restrict__ x, long long x_stride, const T*
         float d[4];
         rows_dot<T, 4>(rows, xv, width, lane, wide, d);
         if (lane == 0) {
-            mid[(size_t)pair * ff + j] = from_f32<T>(expert_act(d[0], d[1], limit, alpha));
-            if (j1 != j) mid[(size_t)pair * ff + j1] = from_f32<T>(expert_act(d[2], d[3], limit, alpha));
+            mid[(size_t)pair * ff + j] = from_f32<T>(gated_act(d[0], d[1], limit, alpha, form));
+            if (j1 != j) mid[(size_t)pair * ff + j1] = from_f32<T>(gated_act(d[2], d[3], limit, alpha, form));
         }
     }
 }
@@ -333,7 +358,8 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 routed_rows_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_down,
                         const int* __restrict__ ids, const float* __restrict__ weights,
-                        const T* __restrict__ base, T* __restrict__ out, int width, int ff, int top) {
+                        const T* __restrict__ base, const float* __restrict__ base_weight,
+                        T* __restrict__ out, int width, int ff, int top) {
     extern __shared__ __align__(16) float ms[];      // [top][ff]
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -343,7 +369,7 @@ routed_rows_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_down,
     __syncthreads();
     const bool wide = reads_wide(w_down, ff) && ff % 4 == 0;
     for (int n = blockIdx.x * 4 + warp; n < width; n += gridDim.x * 4) {
-        float acc = base ? to_f32(base[(size_t)r * width + n]) : 0.f;
+        float acc = base ? to_f32(base[(size_t)r * width + n]) * (base_weight ? base_weight[r] : 1.0f) : 0.f;
         for (int k0 = 0; k0 < top; k0 += 4) {
             const T* rows[4];
             const float* mv[4];
@@ -383,7 +409,7 @@ __global__ void __launch_bounds__(128)
 routed_expert_gate_up_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ w_gu,
                              const int* __restrict__ ids, const float* __restrict__ pair_weight,
                              T* __restrict__ mid, int width, int ff, int top, int pairs, float limit,
-                             float alpha) {
+                             float alpha, int form) {
     extern __shared__ __align__(16) float sh[];      // [width] a row, then the list of pairs
     __shared__ int count;
     float* xs = sh;
@@ -424,8 +450,8 @@ routed_expert_gate_up_kernel(const T* __restrict__ x, long long x_stride, const 
             float d[4];
             rows_dot<T, 4, true>(rows, xv, width, lane, wide, d);
             if (lane == 0) {
-                mid[(size_t)pair * ff + j] = from_f32<T>(expert_act(d[0], d[1], limit, alpha));
-                if (j1 != j) mid[(size_t)pair * ff + j1] = from_f32<T>(expert_act(d[2], d[3], limit, alpha));
+                mid[(size_t)pair * ff + j] = from_f32<T>(gated_act(d[0], d[1], limit, alpha, form));
+                if (j1 != j) mid[(size_t)pair * ff + j1] = from_f32<T>(gated_act(d[2], d[3], limit, alpha, form));
             }
         }
     }
@@ -472,14 +498,15 @@ routed_expert_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_dow
 template <typename T>
 __global__ void routed_combine_kernel(const T* __restrict__ ys, const int* __restrict__ where,
                                       const float* __restrict__ weights, const T* __restrict__ base,
-                                      T* __restrict__ out, int width, int top, size_t total) {
+                                      const float* __restrict__ base_weight, T* __restrict__ out,
+                                      int width, int top, size_t total) {
     pdl_trigger();
     pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total;
          i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / width;
         const int n = (int)(i - r * width);
-        float acc = base ? to_f32(base[i]) : 0.f;
+        float acc = base ? to_f32(base[i]) * (base_weight ? base_weight[r] : 1.0f) : 0.f;
         for (int k = 0; k < top; ++k)
             acc += (weights ? weights[r * top + k] : 1.0f) * to_f32(ys[(size_t)where[r * top + k] * width + n]);
         out[i] = from_f32<T>(acc);
@@ -493,41 +520,49 @@ int grid_for(size_t total) {
 
 }  // namespace
 
-SIB_EXPORT int sib_router_topk(const float* logits, const float* bias, int* ids, float* weights,
-                               int rows, int experts, int top, int score, void* stream) {
+// `stride`: floats between rows of `logits` (experts, or one more with a gate's logit behind them).
+SIB_EXPORT int sib_router_topk(const float* logits, int stride, const float* bias, int* ids,
+                               float* weights, float* gate, int rows, int experts, int top, int score,
+                               float scale, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && experts > 0 && top > 0 && top <= experts && top <= 32,
                 "router_topk: rows=%d experts=%d top=%d (at most 32 and the number of experts)",
                 rows, experts, top);
+    SIB_REQUIRE(stride >= experts + (gate ? 1 : 0), "router_topk: rows of %d logits for %d experts%s", stride,
+                experts, gate ? " and a gate" : "");
     sib_launch_chained(router_topk_kernel, dim3((rows + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
-                       logits, bias, ids, weights, rows, experts, top, score);
+                       logits, stride, bias, ids, weights, gate, rows, experts, top, score, scale);
     return sib_check_launch("router_topk");
 }
 
+// With `gate` the matrix has experts + 1 rows, the last of them the gate's.
 SIB_EXPORT int sib_router_rows(const void* x, long long x_stride, int dtype, const float* w,
-                               const float* bias, int* ids, float* weights, int rows, int width,
-                               int experts, int top, int score, float* logits, void* stream) {
+                               const float* bias, int* ids, float* weights, float* gate, int rows,
+                               int width, int experts, int top, int score, float scale, float* logits,
+                               void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && width > 0 && experts > 0 && top > 0 && top <= experts && top <= 32,
                 "router_rows: rows=%d width=%d experts=%d top=%d", rows, width, experts, top);
     if (logits != nullptr && experts >= 16 && rows < 65536 && (size_t)width * 4 <= 48 * 1024) {
         // (one block a row walked 32 experts' rows of 2 048 in 23 us; spread over the device the
         // product and the choice are two launches of a few us)
-        SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(router_logits_kernel<T>, dim3((experts + 3) / 4, rows),
+        const int n = experts + (gate ? 1 : 0);
+        SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(router_logits_kernel<T>, dim3((n + 3) / 4, rows),
                                                      dim3(128), (size_t)width * 4, (cudaStream_t)stream,
-                                                     (const T*)x, x_stride, w, logits, width, experts));
+                                                     (const T*)x, x_stride, w, logits, width, n));
         int rc = sib_check_launch("router_logits");
         if (rc) return rc;
         sib_launch_chained(router_topk_kernel, dim3((rows + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
-                           (const float*)logits, bias, ids, weights, rows, experts, top, score);
+                           (const float*)logits, n, bias, ids, weights, gate, rows, experts, top, score,
+                           scale);
         return sib_check_launch("router_topk");
     }
-    const size_t shared = ((size_t)((width + 3) & ~3) + experts) * 4;
+    const size_t shared = ((size_t)((width + 3) & ~3) + experts + 1) * 4;
     SIB_REQUIRE(shared <= 48 * 1024, "router_rows: a row of %d and %d logits do not fit shared memory",
                 width, experts);
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(router_rows_kernel<T>, dim3(rows), dim3(256), shared,
                                                  (cudaStream_t)stream, (const T*)x, x_stride, w, bias,
-                                                 ids, weights, width, experts, top, score));
+                                                 ids, weights, gate, width, experts, top, score, scale));
     return sib_check_launch("router_rows");
 }
 
@@ -554,9 +589,10 @@ SIB_EXPORT int sib_expert_activate(const void* gu, long long stride, void* y, co
 }
 
 SIB_EXPORT int sib_routed_rows(const void* x, long long x_stride, const void* w_gu, const void* w_down,
-                               const int* ids, const float* weights, const void* base, void* mid,
-                               void* out, int dtype, int rows, int width, int ff, int top,
-                               float limit, float alpha, int form, void* stream) {
+                               const int* ids, const float* weights, const void* base,
+                               const float* base_weight, void* mid, void* out, int dtype, int rows,
+                               int width, int ff, int top, float limit, float alpha, int form,
+                               void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && rows * (long long)top < 65536 && width > 0 && ff > 0 && top > 0,
                 "routed_rows: rows=%d top=%d width=%d ff=%d", rows, top, width, ff);
@@ -572,13 +608,13 @@ SIB_EXPORT int sib_routed_rows(const void* x, long long x_stride, const void* w_
                                                      dim3(min((ff + 15) / 16, 64), pairs), dim3(128),
                                                      (size_t)width * 4, s, (const T*)x, x_stride,
                                                      (const T*)w_gu, ids, weights, (T*)mid, width, ff,
-                                                     top, limit, alpha));
+                                                     top, limit, alpha, form));
     } else {
         SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(routed_rows_gate_up_kernel<T, false>,
                                                      dim3(min((ff + 7) / 8, 64), pairs), dim3(128),
                                                      (size_t)width * 4, s, (const T*)x, x_stride,
                                                      (const T*)w_gu, ids, weights, (T*)mid, width, ff,
-                                                     top, limit, alpha));
+                                                     top, limit, alpha, form));
     }
     int rc = sib_check_launch("routed_rows_gate_up");
     if (rc) return rc;
@@ -589,7 +625,7 @@ SIB_EXPORT int sib_routed_rows(const void* x, long long x_stride, const void* w_
                                                  dim3(down_tiles, rows), dim3(128),
                                                  (size_t)top * ff * 4, s, (const T*)mid,
                                                  (const T*)w_down, ids, out_weights, (const T*)base,
-                                                 (T*)out, width, ff, top));
+                                                 base_weight, (T*)out, width, ff, top));
     return sib_check_launch("routed_rows_down");
 }
 
@@ -597,8 +633,8 @@ SIB_EXPORT int sib_routed_rows(const void* x, long long x_stride, const void* w_
 // `order` the numbers 0 .. rows * top - 1 (where pair (r, k)'s output lies: r * top + k).
 SIB_EXPORT int sib_routed_by_expert(const void* x, long long x_stride, const void* w_gu,
                                     const void* w_down, const int* ids, const float* weights,
-                                    const void* base, void* mid, void* ys, const int* order, void* out,
-                                    int dtype, int rows, int width, int ff, int top, int experts,
+                                    const void* base, const float* base_weight, void* mid, void* ys,
+                                    const int* order, void* out, int dtype, int rows, int width, int ff, int top, int experts,
                                     float limit, float alpha, int form, void* stream) {
     if (rows == 0) return 0;
     const long long pairs = (long long)rows * top;
@@ -613,13 +649,13 @@ SIB_EXPORT int sib_routed_by_expert(const void* x, long long x_stride, const voi
                                                      dim3((ff + 15) / 16, experts), dim3(128),
                                                      ((size_t)((width + 3) & ~3) + pairs) * 4, s,
                                                      (const T*)x, x_stride, (const T*)w_gu, ids, weights,
-                                                     (T*)mid, width, ff, top, (int)pairs, limit, alpha));
+                                                     (T*)mid, width, ff, top, (int)pairs, limit, alpha, form));
     } else {
         SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(routed_expert_gate_up_kernel<T, false>,
                                                      dim3((ff + 7) / 8, experts), dim3(128),
                                                      ((size_t)((width + 3) & ~3) + pairs) * 4, s,
                                                      (const T*)x, x_stride, (const T*)w_gu, ids, weights,
-                                                     (T*)mid, width, ff, top, (int)pairs, limit, alpha));
+                                                     (T*)mid, width, ff, top, (int)pairs, limit, alpha, form));
     }
     int rc = sib_check_launch("routed_expert_gate_up");
     if (rc) return rc;
@@ -633,12 +669,12 @@ SIB_EXPORT int sib_routed_by_expert(const void* x, long long x_stride, const voi
     const size_t total = (size_t)rows * width;
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(routed_combine_kernel<T>, dim3(grid_for(total)),
                                                  dim3(256), 0, s, (const T*)ys, order, out_weights,
-                                                 (const T*)base, (T*)out, width, top, total));
+                                                 (const T*)base, base_weight, (T*)out, width, top, total));
     return sib_check_launch("routed_combine");
 }
 
 SIB_EXPORT int sib_routed_combine(const void* ys, const int* where, const float* weights,
-                                  const void* base, void* out, int dtype, int rows, int width,
+                                  const void* base, const float* base_weight, void* out, int dtype, int rows, int width,
                                   int top, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && width > 0 && top > 0, "routed_combine: rows=%d width=%d top=%d", rows,
@@ -646,7 +682,7 @@ SIB_EXPORT int sib_routed_combine(const void* ys, const int* where, const float*
     const size_t total = (size_t)rows * width;
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(routed_combine_kernel<T>, dim3(grid_for(total)),
                                                  dim3(256), 0, (cudaStream_t)stream, (const T*)ys,
-                                                 where, weights, (const T*)base, (T*)out, width, top,
-                                                 total));
+                                                 where, weights, (const T*)base, base_weight, (T*)out, width,
+                                                 top, total));
     return sib_check_launch("routed_combine");
 }

@@ -7,6 +7,7 @@ function with per-architecture branches (src/model/layer.rs:1255-1392).
 
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List, Mapping, Optional, Tuple
 
 import torch
@@ -50,6 +51,10 @@ def _sites(spec: ModelSpec):
         for site, norm in layer.norms.items():
             yield (layer.prefix + layer.names[site], parts.part_class("norm", norm.kind),
                    (norm.params, H), layer.tensor_names.get(site, {}))
+        if layer.mixer_input is not None:
+            yield (layer.prefix + layer.names["mixer_input"],
+                   parts.part_class("mixer_input", layer.mixer_input.kind),
+                   (layer.mixer_input.params, H), layer.tensor_names.get("mixer_input", {}))
         if layer.tail is not None:
             yield (layer.prefix + layer.names["tail"], parts.part_class("tail", layer.tail.kind),
                    (layer.tail.params, H), layer.tensor_names.get("tail", {}))
@@ -125,6 +130,10 @@ class DecoderModel:
             if layer.tail is not None:
                 extra["tail"] = parts.part_class("tail", layer.tail.kind)(
                     layer.tail.params, H, _sub(weights, layer.prefix + layer.names["tail"]), rt)
+            if layer.mixer_input is not None:
+                extra["mixer_input"] = parts.part_class("mixer_input", layer.mixer_input.kind)(
+                    layer.mixer_input.params, H,
+                    _sub(weights, layer.prefix + layer.names["mixer_input"]), rt)
             self.blocks.append(parts.part_class("block", layer.block)(mixer, ff, norms, rt, **extra))
         self.pass_mix = None
         if spec.pass_mix is not None:
@@ -134,6 +143,8 @@ class DecoderModel:
             spec.final_norm.params, H, _sub(weights, spec.names["final_norm"]), rt)
         self.head = parts.part_class("head", spec.head.kind)(
             spec.head.params, H, V, _sub(weights, spec.names["head"]), rt, self.embedding)
+        if getattr(self.head, "input_scale", 1.0) != 1.0:
+            self.final_norm.scale_output(self.head.input_scale)
 
     def named_state(self) -> Dict[str, "StateNeed"]:
         """Per-slot state that belongs to no schedule entry (the embedding's), by name."""
@@ -141,11 +152,16 @@ class DecoderModel:
         return {"embedding": need()} if need is not None else {}
 
     def cache_needs(self) -> List[Optional[CacheNeed]]:
-        """One entry per schedule position; None where the run borrows a cache."""
+        """One entry per schedule position; what a mixer needs is left out where the run
+        borrows a cache, a part at its input keeps a state of its own in every run."""
         needs: List[Optional[CacheNeed]] = []
         for e in self.spec.schedule:
-            needs.append(None if e.cache_of is not None
-                         else self.blocks[e.layer].mixer.cache_need())
+            block = self.blocks[e.layer]
+            need = None if e.cache_of is not None else block.mixer.cache_need()
+            at_input = getattr(block, "mixer_input", None)
+            if at_input is not None and at_input.state_need() is not None:
+                need = replace(need or CacheNeed(), inputs=at_input.state_need())
+            needs.append(need)
         return needs
 
     @property
@@ -186,13 +202,19 @@ class DecoderModel:
                 normed = None
             # (a run that begins a pass norms the mixed stream itself)
             last = pos + 1 == len(schedule) or schedule[pos + 1].begins_pass
-            nxt = None if last else self.blocks[schedule[pos + 1].layer].first_norm
+            following = None if last else self.blocks[schedule[pos + 1].layer]
+            nxt = following.first_norm if following is not None else None
+            extra = {}
+            if getattr(following, "mixer_input", None) is not None and getattr(block, "hands_over", False):
+                # (the block may run what the next one does to its normed rows in its own last launch)
+                extra["next_input"] = (following.mixer_input, pos + 1)
             cache_entry = pos if e.cache_of is None else e.cache_of
             if self.rt.chain is not None and not getattr(block, "chain_safe", False):
                 with chain_suspended(self.rt):
-                    normed = block.forward(h, normed, ctx, pos, cache_entry, e.cache_of is None, nxt)
+                    normed = block.forward(h, normed, ctx, pos, cache_entry, e.cache_of is None, nxt,
+                                           **extra)
             else:
-                normed = block.forward(h, normed, ctx, pos, cache_entry, e.cache_of is None, nxt)
+                normed = block.forward(h, normed, ctx, pos, cache_entry, e.cache_of is None, nxt, **extra)
         return h
 
     def logits(self, h: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:

@@ -31,8 +31,10 @@ ACT_GELU_TANH, ACT_SILU = 0, 1          # of the gated feed-forward
 ACT_RELU_SQUARED = 2                    # of the feed-forward without a gate (activate)
 ACT_TANH = 3                            # tanh, value by value (activate)
 GATE_SILU, GATE_SIGMOID = 0, 1          # of head_norm_gate
-SCORE_SOFTMAX_TOP, SCORE_SIGMOID = 0, 1     # of the routers: what a chosen expert's weight is
-FORM_CLIPPED_GATED, FORM_PLAIN_GELU = 0, 1  # of the routed experts: what an expert computes
+# of the routers: what a chosen expert's weight is
+SCORE_SOFTMAX_TOP, SCORE_SIGMOID, SCORE_SOFTMAX_ALL = 0, 1, 2
+# of the routed experts: what an expert computes
+FORM_CLIPPED_GATED, FORM_PLAIN_GELU, FORM_GATED_SILU = 0, 1, 2
 
 _lib = None
 
@@ -243,26 +245,29 @@ def _timed(work: Callable):
 
 
 def _attention_cache_work(kind, row_pos, k_pool, n_heads, head_dim, window, rows, value_dim=None,
-                          chunk=0):
+                          chunk=0, keep=0):
     """Keys and values a row at ``row_pos`` reads from the cache (reads the positions back:
     only done under a profile)."""
     seen = row_pos.to(torch.int64) + 1
     if chunk > 0:
         seen = row_pos.to(torch.int64) % chunk + 1
     elif window > 0:
-        seen = seen.clamp(max=window)
+        seen = seen.clamp(max=window) + (seen - window).clamp(min=0, max=keep)
     keys = int(seen.sum().item())
     n_kv = k_pool.shape[1]
     nbytes = keys * n_kv * (head_dim + (value_dim or head_dim)) * k_pool.element_size()
     return kind, nbytes, 4.0 * keys * n_heads * head_dim
 
 
-def _prompt_work(kind, qkv, seq_len, n_heads, head_dim, window):
+def _prompt_work(kind, qkv, seq_len, n_heads, head_dim, window, keep=0):
     """Prompts from position 0: (query, key) pairs inside the causal mask and the window."""
     pairs = 0
     for n in seq_len.to(torch.int64).tolist():
         if window and n > window:
             pairs += window * (window + 1) // 2 + (n - window) * window
+            # (first positions that the window keeps: 1, 2, ... keep, keep, ... of them)
+            grows = min(n - window, keep)
+            pairs += grows * (grows + 1) // 2 + (n - window - grows) * keep
         else:
             pairs += n * (n + 1) // 2
     return kind, _nbytes(qkv) + qkv.shape[0] * n_heads * head_dim * qkv.element_size(), \
@@ -519,11 +524,18 @@ def pair_norm_mean(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch
 
 @_timed(lambda logits, bias, ids, weights, *a: ("router_topk", _nbytes(logits, ids, weights), 0))
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor,
-                weights: torch.Tensor, score: int = SCORE_SOFTMAX_TOP) -> None:
+                weights: torch.Tensor, score: int = SCORE_SOFTMAX_TOP, scale: float = 1.0,
+                gate: Optional[torch.Tensor] = None) -> None:
     """Per row of the 32-bit ``logits`` (+ ``bias``): the ``top`` = ids.shape[1] largest (ties: the
     lower index) into ``ids`` (int32) and into ``weights`` the softmax over those alone
-    (SCORE_SOFTMAX_TOP) or each one's own sigmoid (SCORE_SIGMOID)."""
+    (SCORE_SOFTMAX_TOP) or each one's own sigmoid (SCORE_SIGMOID).  SCORE_SOFTMAX_ALL: the softmax
+    over all logits plus ``bias`` chooses, and the weight is the softmax without it, times
+    ``scale``.  ``gate`` (32-bit, one per row): the rows of ``logits`` hold one logit more, whose
+    sigmoid goes there."""
     rows, experts = logits.shape
+    if gate is not None:
+        experts -= 1
+        _f32(gate, rows, "gate")
     top = ids.shape[1]
     _want(logits, torch.float32, "logits")
     _want(ids, torch.int32, "ids")
@@ -532,17 +544,22 @@ def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.T
         _f32(bias, experts, "bias")
     if ids.shape[0] != rows:
         raise KernelError("router_topk: one row of choices per row of logits")
-    _check(library().sib_router_topk(_ptr(logits), _ptr(bias), _ptr(ids), _ptr(weights), c_int(rows),
-                                     c_int(experts), c_int(top), c_int(score), _stream()))
+    _check(library().sib_router_topk(_ptr(logits), c_int(logits.shape[1]), _ptr(bias), _ptr(ids), _ptr(weights),
+                                     _ptr(gate), c_int(rows), c_int(experts), c_int(top), c_int(score),
+                                     c_float(scale), _stream()))
 
 
 @_timed(lambda x, w, bias, ids, weights, *a: ("router_rows", _nbytes(x, w), 2.0 * x.shape[0] * w.numel()))
 def router_rows(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor,
-                weights: torch.Tensor, score: int = SCORE_SOFTMAX_TOP) -> None:
-    """Few rows: z = w x (+ ``bias``) with the 32-bit matrix ``w`` ``[experts, width]`` and the
-    choice of :func:`router_topk`, in one launch; sums are 32-bit."""
+                weights: torch.Tensor, score: int = SCORE_SOFTMAX_TOP, scale: float = 1.0,
+                gate: Optional[torch.Tensor] = None) -> None:
+    """Few rows: z = w x (+ ``bias``) with the 32-bit matrix ``w`` ``[experts, width]`` (one row more
+    with ``gate``, whose logit is the gate's) and the choice of :func:`router_topk`, in one
+    launch; sums are 32-bit."""
     rows, width = x.shape
-    experts, top = w.shape[0], ids.shape[1]
+    experts, top = w.shape[0] - (1 if gate is not None else 0), ids.shape[1]
+    if gate is not None:
+        _f32(gate, rows, "gate")
     _want(x, x.dtype, "x", contiguous=False)
     _want(w, torch.float32, "w")
     _want(ids, torch.int32, "ids")
@@ -552,10 +569,11 @@ def router_rows(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
     if w.shape[1] != width or ids.shape[0] != rows or x.stride(1) != 1:
         raise KernelError("router_rows: shapes do not fit")
     # (with 16 experts and more the logits are made by many blocks and left here for the choice)
-    logits = torch.empty((rows, experts), dtype=torch.float32, device=x.device) if experts >= 16 else None
+    logits = torch.empty((rows, w.shape[0]), dtype=torch.float32, device=x.device) if experts >= 16 else None
     _check(library().sib_router_rows(_ptr(x), c_longlong(x.stride(0)), _code(x.dtype), _ptr(w), _ptr(bias),
-                                     _ptr(ids), _ptr(weights), c_int(rows), c_int(width),
-                                     c_int(experts), c_int(top), c_int(score), _ptr(logits), _stream()))
+                                     _ptr(ids), _ptr(weights), _ptr(gate), c_int(rows), c_int(width),
+                                     c_int(experts), c_int(top), c_int(score), c_float(scale), _ptr(logits),
+                                     _stream()))
 
 
 @_timed(lambda gu, y, row_weight, limit, alpha, *a: ("expert_activate", _nbytes(gu, y), 0))
@@ -564,7 +582,7 @@ def expert_activate(gu: torch.Tensor, y: torch.Tensor, row_weight: Optional[torc
                     group: int = 0) -> torch.Tensor:
     """FORM_CLIPPED_GATED: y = g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up,
     -limit, limit), from rows ``[gate (ff) | up (ff)]``; with ``row_weight`` every row times its
-    32-bit weight.  FORM_PLAIN_GELU: y = gelu(row_weight * up), the exact gelu, from rows ``[up
+    32-bit weight.  FORM_GATED_SILU: y = silu(gate) * up from the same rows.  FORM_PLAIN_GELU: y = gelu(row_weight * up), the exact gelu, from rows ``[up
     (ff)]``.  ``group`` 8: gates and ups lie interleaved in eights (8 gates, then their 8 ups)."""
     rows, ff = y.shape
     _want(gu, y.dtype, "gu", contiguous=False)
@@ -582,17 +600,19 @@ def expert_activate(gu: torch.Tensor, y: torch.Tensor, row_weight: Optional[torc
 _PAIR_ORDER: dict = {}
 
 
-@_timed(lambda x, w_gu, w_down, ids, weights, base, out, limit, alpha, form=0: (
-    "routed_rows", min(ids.numel(), w_down.shape[0]) * (2 if form else 3) * w_down.shape[1] * w_down.shape[2]
-    * x.element_size(), (4.0 if form else 6.0) * ids.numel() * w_down.shape[1] * w_down.shape[2]))
+@_timed(lambda x, w_gu, w_down, ids, weights, base, out, limit, alpha, form=0, base_weight=None: (
+    "routed_rows", min(ids.numel(), w_down.shape[0]) * (2 if form == FORM_PLAIN_GELU else 3) * w_down.shape[1]
+    * w_down.shape[2] * x.element_size(),
+    (4.0 if form == FORM_PLAIN_GELU else 6.0) * ids.numel() * w_down.shape[1] * w_down.shape[2]))
 def routed_rows(x: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
                 weights: torch.Tensor, base: Optional[torch.Tensor], out: torch.Tensor,
-                limit: float, alpha: float, form: int = FORM_CLIPPED_GATED) -> torch.Tensor:
+                limit: float, alpha: float, form: int = FORM_CLIPPED_GATED,
+                base_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The chosen experts of every row, each (row, expert) pair streaming its expert's matrices
     (csrc/routed.cu): ``w_gu`` ``[experts, 2 ff, width]`` (gate rows, then up rows), ``w_down``
     ``[experts, width, ff]``; out = base + sum_k weights[r, k] down(act(gate, up)) in 32-bit.
     FORM_PLAIN_GELU: ``w_gu`` ``[experts, ff, width]`` (up rows alone), out = base + sum_k
-    down(gelu(weights[r, k] * up)).
+    down(gelu(weights[r, k] * up)).  ``base_weight`` (32-bit, one per row) multiplies the base row.
     With more pairs than half the experts the kernels go expert by expert instead (an expert's
     matrices are read once for all the pairs that chose it)."""
     rows, width = x.shape
@@ -609,6 +629,8 @@ def routed_rows(x: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: 
         raise KernelError("routed_rows: shapes do not fit")
     if base is not None:
         _want(base, x.dtype, "base")
+    if base_weight is not None:
+        _f32(base_weight, rows, "base_weight")
     mid = torch.empty((rows * top, ff), dtype=x.dtype, device=x.device)
     pairs = rows * top
     if 2 * pairs > experts and (max(width, ff) + 4 + pairs) * 4 <= 48 * 1024:
@@ -619,21 +641,22 @@ def routed_rows(x: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: 
         ys = torch.empty((pairs, width), dtype=x.dtype, device=x.device)
         _check(library().sib_routed_by_expert(
             _ptr(x), c_longlong(x.stride(0)), _ptr(w_gu), _ptr(w_down), _ptr(ids), _ptr(weights),
-            _ptr(base), _ptr(mid), _ptr(ys), _ptr(order), _ptr(out), _code(x.dtype), c_int(rows),
+            _ptr(base), _ptr(base_weight), _ptr(mid), _ptr(ys), _ptr(order), _ptr(out), _code(x.dtype), c_int(rows),
             c_int(width), c_int(ff), c_int(top), c_int(experts), c_float(limit), c_float(alpha),
             c_int(form), _stream()))
         return out
     _check(library().sib_routed_rows(
         _ptr(x), c_longlong(x.stride(0)), _ptr(w_gu), _ptr(w_down), _ptr(ids), _ptr(weights),
-        _ptr(base), _ptr(mid), _ptr(out), _code(x.dtype), c_int(rows), c_int(width), c_int(ff),
+        _ptr(base), _ptr(base_weight), _ptr(mid), _ptr(out), _code(x.dtype), c_int(rows), c_int(width), c_int(ff),
         c_int(top), c_float(limit), c_float(alpha), c_int(form), _stream()))
     return out
 
 
-@_timed(lambda ys, where, weights, base, out: ("routed_combine", _nbytes(ys, out), 0))
+@_timed(lambda ys, where, weights, base, out, base_weight=None: ("routed_combine", _nbytes(ys, out), 0))
 def routed_combine(ys: torch.Tensor, where: torch.Tensor, weights: Optional[torch.Tensor],
-                   base: Optional[torch.Tensor], out: torch.Tensor) -> torch.Tensor:
-    """out[r] = base[r] + sum_k weights[r, k] ys[where[r, k]] in 32-bit: the rows' sums over the
+                   base: Optional[torch.Tensor], out: torch.Tensor,
+                   base_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[r] = base_weight[r] base[r] (without ``base_weight`` base[r]) + sum_k weights[r, k] ys[where[r, k]] in 32-bit: the rows' sums over the
     outputs of their (row, expert) pairs, which lie sorted by expert.  ``weights`` None: the plain
     sum."""
     rows, width = out.shape
@@ -647,7 +670,9 @@ def routed_combine(ys: torch.Tensor, where: torch.Tensor, weights: Optional[torc
         raise KernelError("routed_combine: shapes do not fit")
     if base is not None:
         _want(base, out.dtype, "base")
-    _check(library().sib_routed_combine(_ptr(ys), _ptr(where), _ptr(weights), _ptr(base), _ptr(out),
+    if base_weight is not None:
+        _f32(base_weight, rows, "base_weight")
+    _check(library().sib_routed_combine(_ptr(ys), _ptr(where), _ptr(weights), _ptr(base), _ptr(base_weight), _ptr(out),
                                         _code(out.dtype), c_int(rows), c_int(width), c_int(top),
                                         _stream()))
     return out
@@ -691,13 +716,17 @@ def head_prepare(proj: torch.Tensor, qkv: torch.Tensor, bias: Optional[torch.Ten
                  seq_slot, seq_end, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
                  page_table: Optional[torch.Tensor], page_tokens: int, ring_tokens: int,
                  n_heads: int, n_kv: int, key_dim: int, value_dim: int, pad: int,
-                 style: int = ROPE_HALF_SPLIT) -> torch.Tensor:
+                 style: int = ROPE_HALF_SPLIT, norm_after: bool = False,
+                 temp: Optional[torch.Tensor] = None, magnitude: float = 1.0,
+                 fixed_tokens: int = 0) -> torch.Tensor:
     """From a projected row ``[q heads | k heads | v heads | ...]`` to the packed q|k|v rows
     the attention kernels read, heads ``pad`` wide (csrc/head_prepare.cu): bias, per-head RMS
     norm of q and k with a gain, partial rotation (``style``: half-split pairs or
     neighbouring ones), values mixed with ``v_first`` (a view
     ``[rows, n_kv * its own head width]`` of an earlier layer's packed rows) by ``lam``, and
-    k and v written into the paged cache."""
+    k and v written into the paged cache.  ``magnitude`` multiplies the rotation's cosines and
+    sines; ``norm_after``: q and k are divided by their root mean square per head behind the
+    rotation (no gains); ``temp``: one factor per query head, applied last."""
     rows = proj.shape[0]
     _want(proj, qkv.dtype, "proj", contiguous=False)
     _want(qkv, qkv.dtype, "qkv")
@@ -707,7 +736,7 @@ def head_prepare(proj: torch.Tensor, qkv: torch.Tensor, bias: Optional[torch.Ten
     if tuple(qkv.shape) != (rows, (n_heads + 2 * n_kv) * pad):
         raise KernelError("head_prepare: the packed rows do not fit the head counts")
     for t, n, nm in ((bias, need, "bias"), (q_gain, key_dim, "q_gain"), (k_gain, key_dim, "k_gain"),
-                     (inv_freq, rotary_dim // 2, "inv_freq"), (lam, 1, "lam")):
+                     (inv_freq, rotary_dim // 2, "inv_freq"), (lam, 1, "lam"), (temp, n_heads, "temp")):
         if t is not None:
             _want(t, torch.float32, nm)
             if t.numel() != n:
@@ -736,7 +765,7 @@ def head_prepare(proj: torch.Tensor, qkv: torch.Tensor, bias: Optional[torch.Ten
         _ptr(seq_end), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), c_int(max_pages),
         c_int(page_tokens), c_int(ring_tokens), c_int(rows), c_int(n_heads), c_int(n_kv),
         c_int(key_dim), c_int(value_dim), c_int(pad), c_int(1 if style == ROPE_INTERLEAVED else 0),
-        _stream()))
+        c_int(1 if norm_after else 0), _ptr(temp), c_float(magnitude), c_int(fixed_tokens), _stream()))
     return qkv
 
 
@@ -762,6 +791,65 @@ def pool_store(qkv: torch.Tensor, view, ctx, n_heads: int, n_kv: int, pad: int) 
         _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_end), _ptr(ctx.seq_row0),
         _code(qkv.dtype), c_int(ctx.n_seqs), c_int(ctx.max_count), c_int(n_heads), c_int(n_kv),
         c_int(pad), c_int(view.need.pool), _stream()))
+
+
+def _conv_checks(w: torch.Tensor, state: Optional[torch.Tensor], channels: int, taps: int):
+    _f32(w, taps * channels, "w")
+    if taps > 1:
+        _want(state, torch.float32, "state")
+        if state.dim() != 2 or state.shape[1] < (taps - 1) * channels:
+            raise KernelError("short_conv: the state holds [slots, (taps - 1) * channels]")
+    return _ptr(state), c_longlong(state.stride(0) if state is not None else 0)
+
+
+@_timed(lambda x, y, *a: ("short_conv", _nbytes(x, y), 0))
+def short_conv(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], ctx) -> torch.Tensor:
+    """y = x + conv(x): a causal convolution over time on each channel (csrc/short_conv.cu).  ``w``
+    32-bit ``[taps, channels]`` (the last row weighs the row itself), ``state`` 32-bit ``[slots,
+    (taps - 1) * channels]``: the last inputs of every slot's sequence, brought to the step's end."""
+    rows, channels = x.shape
+    _want(x, y.dtype, "x")
+    _want(y, y.dtype, "y")
+    if tuple(y.shape) != (rows, channels) or rows != ctx.n_rows:
+        raise KernelError("short_conv: x and y must be the step's rows")
+    taps = w.shape[0]
+    ptr, stride = _conv_checks(w, state, channels, taps)
+    # (in a recorded step of prompts a sequence's rows change between replays)
+    single = ctx.max_count == 1 and rows == ctx.n_seqs
+    _check(library().sib_short_conv(
+        _ptr(x), _ptr(y), _code(y.dtype), _ptr(w), ptr, stride, _ptr(ctx.row_pos), _ptr(ctx.row_seq),
+        _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_end), _ptr(ctx.seq_row0), c_int(rows),
+        c_int(ctx.n_seqs), c_int(channels), c_int(taps), c_int(1 if single else 0), _stream()))
+    return y
+
+
+def add_norm_conv_supports(channels: int) -> bool:
+    return bool(library().sib_add_norm_conv_supports(c_int(channels)))
+
+
+@_timed(lambda a, post_gain, post_eps, h, pre_gain, pre_eps, w, state, y, ctx: (
+    "add_norm_conv", _nbytes(a, y) + 2 * _nbytes(h) + 2 * y.numel() * 4 * (w.shape[0] - 1), 0))
+def add_norm_conv(a: torch.Tensor, post_gain: Optional[torch.Tensor], post_eps: float, h: torch.Tensor,
+                  pre_gain: torch.Tensor, pre_eps: float, w: torch.Tensor, state: Optional[torch.Tensor],
+                  y: torch.Tensor, ctx) -> torch.Tensor:
+    """Steps of one bfloat16 row per sequence: ``add_rms_norm`` and :func:`short_conv` of its output
+    as one launch."""
+    rows, channels = h.shape
+    _want(h, torch.float32, "h")
+    _want(a, torch.bfloat16, "a")
+    _want(y, torch.bfloat16, "y")
+    if tuple(a.shape) != (rows, channels) or tuple(y.shape) != (rows, channels) or ctx.n_seqs != rows \
+            or ctx.max_count != 1:
+        raise KernelError("add_norm_conv: one row of each sequence")
+    if post_gain is not None:
+        _f32(post_gain, channels, "post_gain")
+    _f32(pre_gain, channels, "pre_gain")
+    ptr, stride = _conv_checks(w, state, channels, w.shape[0])
+    _check(library().sib_add_norm_conv(
+        _ptr(a), _ptr(post_gain), c_float(post_eps), _ptr(h), _ptr(pre_gain), c_float(pre_eps), _ptr(w), ptr,
+        stride, _ptr(ctx.row_seq), _ptr(ctx.seq_slot), _ptr(y), c_int(rows), c_int(ctx.n_seqs), c_int(channels),
+        c_int(w.shape[0]), _stream()))
+    return y
 
 
 @_timed(lambda o, gate, y, *a: ("head_gate", _nbytes(o, y), 0))
@@ -1175,10 +1263,10 @@ def attention_rows_scratch_bytes(rows: int, n_heads: int, head_dim: int, splits:
 @_timed(lambda q, q_stride, k_new, v_new, kv_stride, k_pool, v_pool, page_table, page_tokens,
         ring_tokens, row_pos, row_seq, seq_slot, seq_start, seq_row0, out, scratch, n_heads, n_kv,
         head_dim, scale, softcap, window, splits, sink=None, values_in_keys=False, cells=None,
-        cells_only=False, chunk=0: (
+        cells_only=False, chunk=0, keep=0, fixed_tokens=0: (
             ("attention_rows (blocks)", _nbytes(out), 0) if cells_only else
             _attention_cache_work("attention_rows (cache)", row_pos, k_pool, n_heads, head_dim,
-                                  window, out.shape[0], chunk=chunk) if k_pool is not None else
+                                  window, out.shape[0], chunk=chunk, keep=keep) if k_pool is not None else
             ("attention_rows (prompt)", 2 * _nbytes(out) * (1 + 2 * n_kv / n_heads),
              2.0 * (row_pos.to(torch.int64) + 1).sum().item() * 2 * n_heads * head_dim)))
 def attention_rows(q: torch.Tensor, q_stride: int, k_new: Optional[torch.Tensor],
@@ -1189,10 +1277,12 @@ def attention_rows(q: torch.Tensor, q_stride: int, k_new: Optional[torch.Tensor]
                    scratch: Optional[torch.Tensor], n_heads: int, n_kv: int, head_dim: int,
                    scale: float, softcap: float, window: int, splits: int,
                    sink: Optional[torch.Tensor] = None, values_in_keys: bool = False,
-                   cells=None, cells_only: bool = False, chunk: int = 0) -> torch.Tensor:
+                   cells=None, cells_only: bool = False, chunk: int = 0, keep: int = 0,
+                   fixed_tokens: int = 0) -> torch.Tensor:
     """General attention of independent rows (see csrc/attention_rows.cu).  ``chunk`` > 0
     (without a window): a row sees the positions of its own chunk of that many, chunks
-    counted from the sequence's first position.  ``sink``: one
+    counted from the sequence's first position.  ``keep`` > 0 (with a window): the sequence's
+    first ``keep`` positions stay visible; ``fixed_tokens`` positions lie ahead of the ring.  ``sink``: one
     32-bit value per query head whose exponential joins the softmax's denominator.
     ``values_in_keys``: a value is its key's cell (``v_new`` / ``v_pool`` are not read).
     ``cells``: a cache view (``KVView``) with cells of pooled blocks; a row then also sees
@@ -1230,7 +1320,7 @@ def attention_rows(q: torch.Tensor, q_stride: int, k_new: Optional[torch.Tensor]
         c_int(cells.need.pool if cells is not None else 0),
         c_int(cells.cell_table.shape[1] if cells is not None else 0),
         c_int(cells.cell_page_tokens if cells is not None else 0),
-        c_int(1 if cells_only else 0), _stream()))
+        c_int(1 if cells_only else 0), c_int(keep), c_int(fixed_tokens), _stream()))
     return out
 
 
@@ -1299,15 +1389,17 @@ def attention_decode_resident_warps(n_heads: int, n_kv: int, head_dim: int, warp
 
 @_timed(lambda q, q_stride, k_pool, v_pool, page_table, page_tokens, ring_tokens, row_pos, row_seq,
         seq_slot, out, scratch, tickets, n_heads, n_kv, head_dim, scale, softcap, window, splits,
-        warps=4, fresh=0, chunk=0, sink=None: _attention_cache_work(
-            "attention_decode", row_pos, k_pool, n_heads, head_dim, window, out.shape[0], chunk=chunk))
+        warps=4, fresh=0, chunk=0, sink=None, keep=0, fixed_tokens=0: _attention_cache_work(
+            "attention_decode", row_pos, k_pool, n_heads, head_dim, window, out.shape[0], chunk=chunk,
+            keep=keep))
 def attention_decode(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                      page_table: torch.Tensor, page_tokens: int, ring_tokens: int, row_pos,
                      row_seq, seq_slot, out: torch.Tensor, scratch: Optional[torch.Tensor],
                      tickets: Optional[torch.Tensor], n_heads: int, n_kv: int, head_dim: int,
                      scale: float, softcap: float, window: int, splits: int,
                      warps: int = 4, fresh: int = 0, chunk: int = 0,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, keep: int = 0,
+                     fixed_tokens: int = 0) -> torch.Tensor:
     """Attention of single rows over the bfloat16 cache (see csrc/attention_decode.cu).
     ``splits`` blocks of ``warps`` warps share the keys of a (row, kv head); with more than one they
     need ``scratch`` for their partial results and ``tickets``: int32 counters, one
@@ -1316,7 +1408,8 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor, v_poo
     rows a sequence has in this step); keys below them are fetched while that kernel still
     runs.  0: every load waits for it.  ``chunk`` > 0 (without a window): a row sees the
     positions of its own chunk; ``sink``: one 32-bit value per query head whose exponential
-    joins the softmax's denominator."""
+    joins the softmax's denominator; ``keep`` > 0 (with a window): the sequence's first ``keep``
+    positions stay visible, ``fixed_tokens`` positions lie ahead of the ring."""
     global _launches
     rows = out.shape[0]
     _want(out, torch.bfloat16, "out")
@@ -1340,7 +1433,8 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor, v_poo
         c_int(page_table.shape[1]), c_int(page_tokens), c_int(ring_tokens), _ptr(row_pos),
         _ptr(row_seq), _ptr(seq_slot), _ptr(out), _ptr(scratch), _ptr(tickets), c_int(rows),
         c_int(n_heads), c_int(n_kv), c_int(head_dim), c_float(scale), c_float(softcap),
-        c_int(window), c_int(splits), c_int(warps), c_int(fresh), c_int(chunk), _ptr(sink), _stream()))
+        c_int(window), c_int(splits), c_int(warps), c_int(fresh), c_int(chunk), _ptr(sink),
+        c_int(keep), c_int(fixed_tokens), _stream()))
     return out
 
 
@@ -1350,13 +1444,14 @@ def attention_prefill_supports(n_heads: int, n_kv: int, head_dim: int) -> bool:
 
 
 @_timed(lambda qkv, out, seq_row0, seq_len, n_seqs, max_len, n_heads, n_kv, head_dim, scale,
-        softcap, window: _prompt_work("attention_prefill (mma.sync)", qkv, seq_len, n_heads,
-                                      head_dim, window))
+        softcap, window, keep=0: _prompt_work("attention_prefill (mma.sync)", qkv, seq_len, n_heads,
+                                              head_dim, window, keep))
 def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n_seqs: int,
                       max_len: int, n_heads: int, n_kv: int, head_dim: int, scale: float,
-                      softcap: float, window: int) -> torch.Tensor:
+                      softcap: float, window: int, keep: int = 0) -> torch.Tensor:
     """Attention of packed bfloat16 prompts that start at position 0 over their
-    own (rotated) keys and values (see csrc/attention_prefill.cu)."""
+    own (rotated) keys and values (see csrc/attention_prefill.cu).  ``keep`` > 0 (with a window):
+    the first ``keep`` positions stay visible."""
     _want(qkv, torch.bfloat16, "qkv")
     _want(out, torch.bfloat16, "out")
     if out.shape[0] != qkv.shape[0] or out.shape[1] != n_heads * head_dim:
@@ -1364,7 +1459,7 @@ def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n
     _check(library().sib_attention_prefill(
         _ptr(qkv), c_int(qkv.shape[1]), _ptr(out), _ptr(seq_row0), _ptr(seq_len), c_int(n_seqs),
         c_int(max_len), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_float(scale),
-        c_float(softcap), c_int(window), _stream()))
+        c_float(softcap), c_int(window), c_int(keep), _stream()))
     return out
 
 
@@ -1386,7 +1481,8 @@ def attention_prefill_tc_split(n_seqs: int, max_len: int, n_heads: int, n_kv: in
 
 
 def attention_prefill_tc_plan(lens: Sequence[int], n_heads: int, n_kv: int, head_dim: int,
-                              window: int, first_query: Optional[Sequence[int]] = None):
+                              window: int, first_query: Optional[Sequence[int]] = None,
+                              keep: int = 0):
     """(work items, bytes of scratch memory, ticket counters) of a launch for prompts of these
     lengths that runs as a balanced list of work items; (0, 0, 0) if it would run as a grid.
     ``first_query``: per sequence, the position from which rows are queries."""
@@ -1396,14 +1492,14 @@ def attention_prefill_tc_plan(lens: Sequence[int], n_heads: int, n_kv: int, head
     q0 = None if first_query is None else (c_int * len(lens))(*[int(n) for n in first_query])
     n_items = library().sib_attention_prefill_tc_plan(arr, q0, c_int(len(lens)), c_int(n_heads),
                                                       c_int(n_kv), c_int(head_dim), c_int(window),
-                                                      byref(nbytes), byref(n_tickets))
+                                                      c_int(keep), byref(nbytes), byref(n_tickets))
     return int(n_items), int(nbytes.value), int(n_tickets.value)
 
 
 @_timed(lambda qkv, out, seq_row0, seq_len, n_seqs, max_len, n_heads, n_kv, head_dim, scale,
         softcap, window, scratch=None, tickets=None, host_lens=None, seq_q0=None,
-        host_q0=None, sink=None, extra=None: _prompt_work(
-            "attention_prefill_tc (tcgen05)", qkv, seq_len, n_heads, head_dim, window))
+        host_q0=None, sink=None, extra=None, keep=0: _prompt_work(
+            "attention_prefill_tc (tcgen05)", qkv, seq_len, n_heads, head_dim, window, keep))
 def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n_seqs: int,
                          max_len: int, n_heads: int, n_kv: int, head_dim: int, scale: float,
                          softcap: float, window: int, scratch: Optional[torch.Tensor] = None,
@@ -1412,8 +1508,9 @@ def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len
                          seq_q0: Optional[torch.Tensor] = None,
                          host_q0: Optional[Sequence[int]] = None,
                          sink: Optional[torch.Tensor] = None,
-                         extra: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """The prompt attention on tcgen05 (see csrc/attention_prefill_tc.cu).  ``sink``: one 32-bit
+                         extra: Optional[torch.Tensor] = None, keep: int = 0) -> torch.Tensor:
+    """The prompt attention on tcgen05 (see csrc/attention_prefill_tc.cu).  ``keep`` > 0 (with a
+    window, no cap): the first ``keep`` positions stay visible.  ``sink``: one 32-bit
     value per head whose exponential joins every row's denominator (no cap then).  ``extra``:
     32-bit ``[rows, heads, head_dim + 2]``, per row and head the (max, sum, accumulator) of keys
     that another kernel has summed (``attention_rows`` with ``cells_only``), joined with this
@@ -1445,7 +1542,7 @@ def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len
         None if host_lens is None else (c_int * len(host_lens))(*[int(n) for n in host_lens]),
         _ptr(seq_q0),
         None if host_q0 is None else (c_int * len(host_q0))(*[int(n) for n in host_q0]),
-        _ptr(sink), _ptr(extra), _stream()))
+        _ptr(sink), _ptr(extra), c_int(keep), _stream()))
     return out
 
 
@@ -1453,7 +1550,8 @@ def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len
 def gather_kv_rows(packed: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                    page_table: torch.Tensor, seq_slot: torch.Tensor, seq_from: torch.Tensor,
                    seq_upto: torch.Tensor, seq_row0: torch.Tensor, most: int, page_tokens: int,
-                   ring_tokens: int, n_heads: int, n_kv: int, head_dim: int) -> torch.Tensor:
+                   ring_tokens: int, n_heads: int, n_kv: int, head_dim: int,
+                   fixed_tokens: int = 0) -> torch.Tensor:
     """Keys and values of the positions [seq_from[b], seq_upto[b]) that sequence b holds in
     the paged cache, into rows seq_row0[b] + position of the packed q|k|v buffer (q columns
     of those rows: zero).  ``most``: the most positions of any sequence."""
@@ -1469,7 +1567,7 @@ def gather_kv_rows(packed: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
         _ptr(packed), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _ptr(seq_slot), _ptr(seq_from),
         _ptr(seq_upto), _ptr(seq_row0), c_int(seq_slot.numel()), c_int(most), c_int(n_heads),
         c_int(n_kv), c_int(head_dim), c_int(page_table.shape[1]), c_int(page_tokens),
-        c_int(ring_tokens), _stream()))
+        c_int(ring_tokens), c_int(fixed_tokens), _stream()))
     return packed
 
 

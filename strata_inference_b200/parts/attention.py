@@ -36,6 +36,14 @@ the projection and the attention kernel, in 32-bit):
 ``qk_norm``     {"eps": e}: q and k are divided by their root mean square per head and
                 multiplied by ``q_norm.weight`` / ``k_norm.weight`` (one per dimension,
                 shared by the heads), before the rotation.
+                Options: ``weight`` False (no weights: the division alone), ``after_rotation``
+                True (behind the rotation instead of before it; without weights only).
+``head_temp``   one stored number per query head (``temp``) that multiplies the head's scores;
+                it is applied to the head's query, in 32-bit, behind norm and rotation.
+``keep_first``  K > 0 (with a ``window``, without a soft cap): a row also sees the sequence's
+                first K positions.  The cache keeps them for good, ahead of the window's ring
+                (``KVNeed.keep_first``).  Every attention kernel walks the tiles of kept
+                positions first and then the window's.
 ``value_mix``   "first": this layer's values are also what later layers mix in;
                 "mix": v <- (1 - l) v + l v_first with l = ``value_mix.weight`` (one number)
                 and v_first the "first" layer's values of the same token; the mixed values
@@ -69,7 +77,8 @@ everything else (32-bit, shapes those two do not take, recorded prompt steps) th
 kernel.
 
 Worked-on heads (any of the options from ``value_dim`` to ``pool``) are rotated in half-split or neighbouring pairs,
-as the position part says, and are attended to by the general kernel when a window is set.
+as the position part says; with pooled blocks they are attended to by the general kernel where
+the tcgen05 prompt kernel does not run.
 """
 
 from __future__ import annotations
@@ -144,7 +153,8 @@ class Attention:
     def _extras(params: Mapping) -> bool:
         """Whether the heads are worked on between the projection and the attention."""
         return bool(params.get("bias") or params.get("qk_norm") or params.get("value_mix")
-                    or params.get("head_gate") or params.get("pool")
+                    or params.get("head_gate") or params.get("pool") or params.get("head_temp")
+                    or params.get("keep_first") or params["position"].get("yarn")
                     or int(params.get("value_dim") or params["head_dim"]) != params["head_dim"]
                     or int(params["head_dim"]) % 16 != 0)      # (padded to the next 16)
 
@@ -159,7 +169,7 @@ class Attention:
             "o_proj.weight": TensorDecl((hidden, nh * vd)),
         }
         if params.get("borrows_cache"):
-            if params.get("bias") or params.get("qk_norm") or params.get("value_mix") or params.get("pool"):
+            if any(params.get(k) for k in ("bias", "qk_norm", "value_mix", "pool", "head_temp", "keep_first")):
                 raise ConfigError("attention: a layer that reads another's keys and values has no "
                                   "biases, norms, mixed values or pooled blocks of its own")
             del out["k_proj.weight"], out["v_proj.weight"]
@@ -169,7 +179,9 @@ class Attention:
             out["q_proj.bias"] = TensorDecl((nh * hd,), init="norm")
             out["k_proj.bias"] = TensorDecl((nkv * hd,), init="norm")
             out["v_proj.bias"] = TensorDecl((nkv * vd,), init="norm")
-        if params.get("qk_norm"):
+        if params.get("head_temp"):
+            out["temp"] = TensorDecl((nh,), init="norm")
+        if params.get("qk_norm") and params["qk_norm"].get("weight", True):
             out["q_norm.weight"] = TensorDecl((hd,), init="norm")
             out["k_norm.weight"] = TensorDecl((hd,), init="norm")
         if params.get("value_mix"):
@@ -206,7 +218,9 @@ class Attention:
             out["qkv_proj.bias"] = Resident((n_qkv,), torch.float32, (
                 Piece("q_proj.bias", 0), Piece("k_proj.bias", nh * hd),
                 Piece("v_proj.bias", (nh + nkv) * hd)))
-        if params.get("qk_norm"):
+        if params.get("head_temp"):
+            out["temp"] = Resident((nh,), torch.float32, (Piece("temp"),))
+        if params.get("qk_norm") and params["qk_norm"].get("weight", True):
             out["q_norm.gain"] = Resident((hd,), torch.float32, (Piece("q_norm.weight"),))
             out["k_norm.gain"] = Resident((hd,), torch.float32, (Piece("k_norm.weight"),))
         if params.get("value_mix") == "mix":
@@ -236,6 +250,12 @@ class Attention:
             raise ConfigError("attention: a chunked mask goes without a window and pooled blocks")
         if (self.chunk or self.sink is not None) and float(params.get("logit_softcap") or 0.0):
             raise ConfigError("attention: a chunked mask or a sink goes without a soft cap")
+        self.keep = int(params.get("keep_first") or 0)
+        if self.keep < 0 or (self.keep and (self.window <= 0 or params.get("pool") or self.softcap)):
+            raise ConfigError("attention: kept first positions go with a window, and without pooled blocks "
+                              "and a soft cap")
+        if self.keep and (self.chunk or self.sink is not None):
+            raise ConfigError("attention: kept first positions with a chunked mask or a sink are not built")
         if self.nh <= 0 or self.nkv <= 0 or self.nh % self.nkv:
             raise ConfigError(f"attention: {self.nh} heads cannot share {self.nkv} kv heads")
         self.vd = int(params.get("value_dim") or self.hd)
@@ -255,6 +275,12 @@ class Attention:
         if self.extras:
             norm = params.get("qk_norm")
             self.qk_eps = float(norm["eps"]) if norm else 0.0
+            self.norm_after = bool(norm and norm.get("after_rotation"))
+            if norm and self.norm_after == bool(norm.get("weight", True)):
+                raise ConfigError("attention: q and k are normed with weights before the rotation, or without "
+                                  "weights behind it")
+            self.temp = weights.get("temp")
+            self.magnitude = float(getattr(self.position, "magnitude", 1.0))
             self.bias = weights.get("qkv_proj.bias")
             self.q_gain, self.k_gain = weights.get("q_norm.gain"), weights.get("k_norm.gain")
             self.value_mix = params.get("value_mix") or None
@@ -276,14 +302,18 @@ class Attention:
         self._block_warps = tuple(int(w) for w in os.environ.get("SIB_DECODE_WARPS", "8,4,2").split(","))
 
     def cache_need(self) -> Optional[CacheNeed]:
-        return CacheNeed(kv=KVNeed(self.nkv, self.kw, self.window, pool=self.pool, chunk=self.chunk))
+        return CacheNeed(kv=KVNeed(self.nkv, self.kw, self.window, pool=self.pool, chunk=self.chunk,
+                                   keep_first=self.keep))
 
     # ------------------------------------------------------------------
     def _longest(self, ctx, capacity: int) -> int:
         longest = (min(ctx.span or capacity, capacity)) if ctx.graph_capture else ctx.max_end
         if self.chunk > 0:
             return min(longest, self.chunk)
-        return min(longest, self.window) if self.window > 0 else longest
+        if self.window > 0:
+            # (the tiles of kept first positions may reach into one tile more than the positions need)
+            return min(longest, self.window + -(-self.keep // 16) * 16)
+        return longest
 
     def _splits(self, ctx, capacity: int) -> int:
         """How many runs of keys the general kernel cuts a (row, head) into, one
@@ -310,14 +340,14 @@ class Attention:
             self._resident_warps = {w: native.attention_decode_resident_warps(self.nh, self.nkv, self.kw, w)
                                     for w in (8, 4)}
         # (a chunk that does not begin at a tile's first key reaches into one tile more, as a window does)
-        edge = self.window or (self.chunk if self.chunk % 16 else 0)
+        edge = (self.window + -(-self.keep // 16) * 16 if self.window else 0) or (self.chunk if self.chunk % 16 else 0)
         return decode_shape(max(1, ctx.n_rows * self.nkv), self._longest(ctx, capacity), edge,
                             self._resident_warps[4], self._resident_warps[8], self._block_warps)
 
     def _pieces_pay(self, ctx) -> bool:
         """Whether copying what the step's sequences hold (read, write, read again by the
         prompt kernel) moves less than reading it row by row does."""
-        seen = float(self.window) if self.window > 0 else float("inf")
+        seen = float(self.window + self.keep) if self.window > 0 else float("inf")
         by_row = sum(n * min(seen, st + n / 2) for st, n in zip(ctx.starts, ctx.counts))
         copied = sum(min(seen + n, st + n) for st, n in zip(ctx.starts, ctx.counts))
         return by_row > 3 * copied
@@ -331,7 +361,7 @@ class Attention:
         over the cache, as single-token steps do it, every row reads its sequence's whole
         past: 4 096 tokens in pieces of 512 took 183 ms instead of 15 ms in one piece.)"""
         rt, nh, nkv, hd = self.rt, self.nh, self.nkv, self.kw
-        memo = ctx.memo.setdefault(("pieces", self.window), {})
+        memo = ctx.memo.setdefault(("pieces", self.window, self.keep), {})
         if not memo:
             starts, counts = ctx.starts, ctx.counts
             ends = [st + n for st, n in zip(starts, counts)]
@@ -344,7 +374,10 @@ class Attention:
             memo.update(row0=row0, ends=ends, first=first, rows=acc, d_row0=dev(row0), d_ends=dev(ends),
                         d_first=dev(first), d_starts=dev(starts),
                         most=max(e - f for e, f in zip(ends, first)))
-            memo["plan"] = native.attention_prefill_tc_plan(ends, nh, nkv, hd, self.window, starts)
+            # (kept first positions that lie ahead of what the window needs)
+            kept = [min(self.keep, f) for f in first]
+            memo.update(kept=max(kept), d_kept=dev(kept), d_zero=dev([0] * len(kept)))
+            memo["plan"] = native.attention_prefill_tc_plan(ends, nh, nkv, hd, self.window, starts, self.keep)
         width = (nh + 2 * nkv) * hd
         # (one packed buffer and one output buffer a step: the layers use them in turn)
         shared = ctx.memo.setdefault(("pieces", "buffers", width, nh * hd), {})
@@ -357,7 +390,11 @@ class Attention:
         packed, whole = shared["packed"], shared["whole"]
         native.gather_kv_rows(packed, view.k, view.v, view.page_table, ctx.seq_slot, memo["d_first"],
                               memo["d_ends"], memo["d_row0"], memo["most"], view.page_tokens,
-                              view.ring_tokens, nh, nkv, hd)
+                              view.ring_tokens, nh, nkv, hd, view.fixed_tokens)
+        if memo["kept"]:
+            native.gather_kv_rows(packed, view.k, view.v, view.page_table, ctx.seq_slot, memo["d_zero"],
+                                  memo["d_kept"], memo["d_row0"], memo["kept"], view.page_tokens,
+                                  view.ring_tokens, nh, nkv, hd, view.fixed_tokens)
         r = 0
         for row0, st, n in zip(memo["row0"], ctx.starts, ctx.counts):
             packed[row0 + st:row0 + st + n, :nh * hd].copy_(qkv[r:r + n, :nh * hd])
@@ -370,7 +407,7 @@ class Attention:
                                     max(memo["ends"]), nh, nkv, hd, self.scale, self.softcap,
                                     self.window, rt.scratch(need) if need else None,
                                     rt.tickets(n_tickets) if need else None, lens,
-                                    memo["d_starts"], ctx.starts if lens else None)
+                                    memo["d_starts"], ctx.starts if lens else None, keep=self.keep)
         r = 0
         for row0, st, n in zip(memo["row0"], ctx.starts, ctx.counts):
             out[r:r + n].copy_(whole[row0 + st:row0 + st + n])
@@ -473,9 +510,9 @@ class Attention:
             # the same step still sees (a captured step adds one position: always fine)
             room = view.ring_tokens - max(self.window, self.pool) + 1
             for start, n in zip(ctx.starts, ctx.counts):
-                if n > room and start + n > view.ring_tokens:
+                if n > room and start + n > view.fixed_tokens + view.ring_tokens:
                     raise ValueError(
-                        f"a step may add at most {max(room, view.ring_tokens - start)} positions "
+                        f"a step may add at most {max(room, view.fixed_tokens + view.ring_tokens - start)} positions "
                         f"to a sequence of {start} whose layers keep a window of {self.window} "
                         f"in a ring of {view.ring_tokens}; got {n}")
 
@@ -497,7 +534,9 @@ class Attention:
                                 ctx.row_pos, ctx.row_seq, ctx.seq_slot, ctx.seq_end,
                                 view.k if owns_cache else None, view.v if owns_cache else None,
                                 view.page_table if owns_cache else None, view.page_tokens,
-                                view.ring_tokens, nh, nkv, self.hd, self.vd, hd, style=self.rope_style)
+                                view.ring_tokens, nh, nkv, self.hd, self.vd, hd, style=self.rope_style,
+                                norm_after=self.norm_after, temp=self.temp, magnitude=self.magnitude,
+                                fixed_tokens=view.fixed_tokens)
             if self.pool:
                 native.pool_store(qkv, view, ctx, nh, nkv, hd)
             if self.value_mix == "first":
@@ -544,7 +583,7 @@ class Attention:
                      and not (self.pool and self.softcap))
         if self.chunk > 0 or self.sink is not None:
             out = self._attend_masked(qkv, out, ctx, view, owns_cache, cache_entry)
-        elif (self.pool or (self.extras and self.window)) and not tc_prompt:
+        elif self.pool and not tc_prompt:
             # blocks before the window join the softmax: the general kernel, which reads the
             # step's own keys from the packed rows, earlier ones from the cache and the blocks'
             # cells from their store
@@ -579,7 +618,7 @@ class Attention:
             n_items = 0
             if lens is not None:
                 n_items, need, n_tickets = native.attention_prefill_tc_plan(lens, nh, self.nkv, hd,
-                                                                            self.window)
+                                                                            self.window, keep=self.keep)
             if n_items == 0:
                 lens = None
                 need, n_tickets = native.attention_prefill_tc_split(ctx.n_seqs, ctx.max_count, nh,
@@ -587,19 +626,21 @@ class Attention:
             native.attention_prefill_tc(qkv, out, ctx.seq_row0, ctx.seq_end, ctx.n_seqs,
                                         ctx.max_count, nh, self.nkv, hd, self.scale, self.softcap,
                                         self.window, rt.scratch(need) if need else None,
-                                        rt.tickets(n_tickets) if need else None, lens, extra=extra)
+                                        rt.tickets(n_tickets) if need else None, lens, extra=extra,
+                                        keep=self.keep)
         elif fresh and qkv.dtype == torch.bfloat16 and \
                 native.attention_prefill_supports(nh, self.nkv, hd):
             native.attention_prefill(qkv, out, ctx.seq_row0, ctx.seq_end, ctx.n_seqs,
                                      ctx.max_count, nh, self.nkv, hd, self.scale, self.softcap,
-                                     self.window)
+                                     self.window, self.keep)
         elif fresh:
             k_new = qkv[:, nh * hd:]
             v_new = qkv[:, (nh + nkv) * hd:]
             native.attention_rows(qkv, width, k_new, v_new, width, None, None, None,
                                   view.page_tokens, view.ring_tokens, ctx.row_pos, ctx.row_seq,
                                   ctx.seq_slot, ctx.seq_start, ctx.seq_row0, out, None, nh,
-                                  self.nkv, hd, self.scale, self.softcap, self.window, 1)
+                                  self.nkv, hd, self.scale, self.softcap, self.window, 1, keep=self.keep,
+                                  fixed_tokens=view.fixed_tokens)
         elif (qkv.dtype == torch.bfloat16 and not ctx.graph_capture
               and ctx.max_count >= rt.piece_attention_rows and _USE_TCGEN05_PREFILL and self.scale > 0
               and native.attention_prefill_tc_supports(nh, self.nkv, hd, (nh + 2 * self.nkv) * hd)
@@ -616,7 +657,8 @@ class Attention:
                                     view.ring_tokens, ctx.row_pos, ctx.row_seq, ctx.seq_slot, out,
                                     scratch, tickets, nh, self.nkv, hd, self.scale, self.softcap,
                                     self.window, splits, warps,
-                                    fresh=ctx.max_count if rt.early_keys else 0)
+                                    fresh=ctx.max_count if rt.early_keys else 0, keep=self.keep,
+                                    fixed_tokens=view.fixed_tokens)
         else:
             splits = self._splits(ctx, ctx.cache.max_seq_len)
             scratch = None
@@ -625,8 +667,9 @@ class Attention:
             native.attention_rows(qkv, width, None, None, width, view.k, view.v, view.page_table,
                                   view.page_tokens, view.ring_tokens, ctx.row_pos, ctx.row_seq,
                                   ctx.seq_slot, ctx.seq_start, ctx.seq_row0, out, scratch, nh,
-                                  self.nkv, hd, self.scale, self.softcap, self.window, splits)
-        if self.extras:
+                                  self.nkv, hd, self.scale, self.softcap, self.window, splits,
+                                  keep=self.keep, fixed_tokens=view.fixed_tokens)
+        if self.extras and (self.head_gate or self.vd != hd):
             y = torch.empty((R, nh * self.vd), dtype=out.dtype, device=out.device)
             gate = proj[:, self.n_qkv:self.n_qkv + nh] if self.head_gate else None
             out = native.head_gate(out, gate, y, nh, self.vd, hd)
@@ -737,6 +780,8 @@ class LatentAttention:
         if position is not None:
             if not hasattr(position, "rotary"):
                 raise ConfigError("latent_attention: the position part must offer rotary()")
+            if getattr(position, "magnitude", 1.0) != 1.0:
+                raise ConfigError("latent_attention: a rotation with a magnitude other than 1 is not built")
             self.inv_freq, self.rot, style = position.rotary()
             if self.rot and style != native.ROPE_INTERLEAVED:
                 raise ConfigError("latent_attention: the rotated columns are rotated in neighbouring pairs")

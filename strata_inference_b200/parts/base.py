@@ -16,6 +16,11 @@ Interfaces (duck-typed; the toy parts of the tests implement exactly these):
     position being run, ``cache_entry`` the schedule position whose cache it
     uses (the same unless the schedule lends it another's), ``owns_cache``
     whether it may write there.
+``MixerInput``
+    ``tensors(params, hidden)``, ``state_need() -> StateNeed | None``, ``forward(x, ctx, entry) -> x'``:
+    works on the mixer's normed input rows; its state (``ctx.input_state(entry)``) is its own in
+    every schedule position.  One that also has ``fused_with_norm(ctx)`` and ``add_norm(y, post, h,
+    nxt, ctx, entry)`` can take over the residual step ahead of it (parts/block.py).
 ``FeedForward``
     ``tensors(params, hidden)``, ``forward(x, ctx) -> y``.
 ``Norm``
@@ -473,6 +478,10 @@ class StepContext:
 
     def state(self, entry: int) -> torch.Tensor:
         return self.cache.state_view(entry)
+
+    def input_state(self, entry: int) -> torch.Tensor:
+        """State of the part at the mixer's input of schedule position ``entry``."""
+        return self.cache.input_state_view(entry)
 
 
 def build_part(part_class, args: Tuple, stored, rt: Runtime, *extra):

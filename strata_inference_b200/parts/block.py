@@ -20,6 +20,11 @@ for the next sub-layer" as one kernel (csrc/norm.cu add_rms_norm), reaching
 over to the next block's first norm when the model passes it; Dynamic Tanh norms around an
 add are fused in the same way (add_dyt_norm).
 
+A sandwich or pre-norm block may carry a *mixer input* (a registered "mixer_input" part, such as
+``short_conv``): it works on the pre-mixer norm's rows before the mixer reads them,
+h += post_mixer(mixer(input(pre_mixer(h)))).  Where the part allows it, its work joins the
+launch that makes those rows: the residual step of the block before (``next_input``).
+
 ``parallel`` (one norm, both sub-layers read its output, one add):
 
     n = pre_mixer(h);   h += mixer(n) + feed_forward(n)
@@ -53,8 +58,11 @@ class SandwichBlock:
     norm_sites = ("pre_mixer", "post_mixer", "pre_feed_forward", "post_feed_forward")
     required_sites = ("pre_mixer", "pre_feed_forward")
 
+    hands_over = True       # forward() takes ``next_input``
+
     def __init__(self, mixer, feed_forward, norms: Mapping[str, object], rt,
-                 residual_scale: float = 1.0):
+                 residual_scale: float = 1.0, mixer_input=None):
+        self.mixer_input = mixer_input
         self.residual_scale = float(residual_scale)
         for site in self.required_sites:
             if norms.get(site) is None and (feed_forward is not None or site == "pre_mixer"):
@@ -78,7 +86,7 @@ class SandwichBlock:
         deferred results through the runtime and ``kernels.native`` only, and its norms are
         the kind the residual kernel applies."""
         norms = (self.pre_mixer, self.post_mixer, self.pre_ff, self.post_ff)
-        return (self.residual_scale == 1.0 and getattr(self.mixer, "chain_safe", False)
+        return (self.residual_scale == 1.0 and self.mixer_input is None and getattr(self.mixer, "chain_safe", False)
                 and getattr(self.feed_forward, "chain_safe", False)
                 and all(_fusable(n) and (n is None or n.gain is not None) for n in norms))
 
@@ -88,6 +96,7 @@ class SandwichBlock:
         its mixer and feed-forward promise to read sequences, slots and counts on the
         device only (the block itself and the norms work row by row)."""
         return (getattr(self.mixer, "captures_prompts", False)
+                and (self.mixer_input is None or getattr(self.mixer_input, "captures_prompts", False))
                 and (self.feed_forward is None
                      or getattr(self.feed_forward, "captures_prompts", False)))
 
@@ -113,17 +122,34 @@ class SandwichBlock:
         h.add_(y.to(torch.float32), alpha=self.residual_scale)
         return nxt.forward(h, out_dtype=self.rt.dtype) if nxt is not None else None
 
+    def _last_step(self, y: torch.Tensor, post, h: torch.Tensor, nxt, ctx, next_input) -> Optional[torch.Tensor]:
+        """The block's last residual step; with the next block's mixer input in it where that
+        part and the norms allow it (then marked in the step's memo)."""
+        if next_input is not None:
+            part, entry = next_input
+            if (hasattr(part, "add_norm") and self.residual_scale == 1.0 and _fusable(post)
+                    and getattr(nxt, "fusable_rms", False) and nxt.gain is not None
+                    and part.fused_with_norm(ctx)):
+                self.rt.flush()
+                out = part.add_norm(y, post, h, nxt, ctx, entry)
+                ctx.memo[("mixer input done", entry)] = True
+                return out
+        return self._add_then_norm(y, post, h, nxt)
+
     def forward(self, h: torch.Tensor, normed: Optional[torch.Tensor], ctx, entry: int,
-                cache_entry: int, owns_cache: bool, next_norm=None) -> Optional[torch.Tensor]:
+                cache_entry: int, owns_cache: bool, next_norm=None, next_input=None) -> Optional[torch.Tensor]:
         if normed is None:
             self.rt.flush()
             normed = self.pre_mixer.forward(h, out_dtype=self.rt.dtype)
+        if self.mixer_input is not None and not ctx.memo.get(("mixer input done", entry)):
+            self.rt.flush()
+            normed = self.mixer_input.forward(normed, ctx, entry)
         a = self.mixer.forward(normed, ctx, entry, cache_entry, owns_cache)
         if self.feed_forward is None:
-            return self._add_then_norm(a, self.post_mixer, h, next_norm)
+            return self._last_step(a, self.post_mixer, h, next_norm, ctx, next_input)
         n2 = self._add_then_norm(a, self.post_mixer, h, self.pre_ff)
         f = self.feed_forward.forward(n2, ctx)
-        return self._add_then_norm(f, self.post_ff, h, next_norm)
+        return self._last_step(f, self.post_ff, h, next_norm, ctx, next_input)
 
 
 class PreNormBlock(SandwichBlock):

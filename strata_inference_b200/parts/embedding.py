@@ -18,7 +18,8 @@ start of every pass of a model whose layers are walked several times).
 Head: the product of the (final-normed) wanted rows with the output matrix,
 which is the embedding table when ``tied`` (src/engine/generate.rs:1106-1110),
 then ``cap * tanh(logits / cap)`` when ``logit_softcap`` > 0.  Logits are
-32-bit.
+32-bit.  ``logit_scale`` s (default 1): logits = s * (W y), a factor on the final norm's 32-bit
+output ahead of its rounding (``input_scale``, which the model's final norm takes into its gain).
 """
 
 from __future__ import annotations
@@ -174,6 +175,7 @@ class LMHead:
                  weights: Mapping[str, torch.Tensor], rt, embedding: Optional[TokenEmbedding]):
         self.rt = rt
         self.cap = float(params.get("logit_softcap") or 0.0)
+        self.input_scale = float(params.get("logit_scale", 1.0))
         if params.get("tied", True):
             if embedding is None:
                 raise ValueError("a tied head needs the embedding")

@@ -28,6 +28,13 @@ expert, and the shared one, is down(gelu(up x)) with the exact gelu and no gate 
 row's weight multiplies what ENTERS its expert, y = sum_k expert_k(p_k x) + shared(x); as the
 experts have no biases, up(p x) = p up(x), so the weight is applied in 32-bit to the up
 product's output in front of the gelu.
+``form`` "gated_silu": an expert, and the shared one, is down(silu(gate x) * (up x)).  ``score``
+"softmax_all": s = softmax(z) over all experts; the ``top`` largest s + ``correction`` (a stored
+number per expert, with ``correction`` True) choose, and a chosen expert's weight is its s,
+without the correction and not normalized, times ``router_scale`` (default 1).
+``shared["gate"]`` True: the shared expert's output is multiplied by sigmoid(shared.gate.weight x),
+one number per row (the gate's row lies behind the router's, so that one 32-bit product makes
+both; the factor is applied in 32-bit where the experts' outputs are summed).
 Few rows, and every recorded step: each (row, expert) pair streams its expert's matrices
 (csrc/routed.cu routed_rows).  Many rows: the pairs are sorted by expert on the device into a
 layout [experts, most rows of any expert, width] (that one number is read on the host; a recorded
@@ -202,8 +209,10 @@ class ClippedGatedMLP:
         return rt.linear(mid, self.w_down)
 
 
-_FORMS = {"clipped_gated": native.FORM_CLIPPED_GATED, "plain_gelu": native.FORM_PLAIN_GELU}
-_SCORES = {"softmax_top": native.SCORE_SOFTMAX_TOP, "sigmoid": native.SCORE_SIGMOID}
+_FORMS = {"clipped_gated": native.FORM_CLIPPED_GATED, "plain_gelu": native.FORM_PLAIN_GELU,
+          "gated_silu": native.FORM_GATED_SILU}
+_SCORES = {"softmax_top": native.SCORE_SOFTMAX_TOP, "sigmoid": native.SCORE_SIGMOID,
+           "softmax_all": native.SCORE_SOFTMAX_ALL}
 
 
 class RoutedExperts:
@@ -227,7 +236,18 @@ class RoutedExperts:
         if form not in _FORMS or score not in _SCORES:
             raise ConfigError(f"routed_experts: form {form!r} and score {score!r}; known: "
                               f"{', '.join(_FORMS)}; {', '.join(_SCORES)}")
+        if bool(params.get("correction")) and score != "softmax_all":
+            raise ConfigError("routed_experts: a correction goes with the score 'softmax_all'")
         return _FORMS[form]
+
+    @staticmethod
+    def _shared_gate(params: Mapping) -> bool:
+        return bool(params.get("shared") and params["shared"].get("gate"))
+
+    @staticmethod
+    def _shared_mlp(params: Mapping):
+        """The shared expert of gated SiLU experts is the dense gated feed-forward, as it is."""
+        return {"intermediate_size": int(params["shared"]["intermediate_size"]), "activation": "silu"}
 
     @classmethod
     def tensors(cls, params: Mapping, hidden: int) -> Dict[str, TensorDecl]:
@@ -235,7 +255,11 @@ class RoutedExperts:
         out = {"router.weight": TensorDecl((E, hidden))}
         if params.get("router_bias", True):
             out["router.bias"] = TensorDecl((E,), init="norm")
-        gated = cls._form(params) == native.FORM_CLIPPED_GATED
+        if params.get("correction"):
+            out["correction"] = TensorDecl((E,), init="norm")
+        if cls._shared_gate(params):
+            out["shared.gate.weight"] = TensorDecl((1, hidden))
+        gated = cls._form(params) != native.FORM_PLAIN_GELU
         for e in range(E):
             if gated:
                 out[f"experts.{e}.gate_proj.weight"] = TensorDecl((ff, hidden))
@@ -254,7 +278,8 @@ class RoutedExperts:
         rows, then its up rows; experts without a gate: [experts, ff, hidden], the up rows
         alone) and their down matrices as one [experts, hidden, ff]; the router's matrix 32-bit."""
         E, top, ff, sff = cls._sizes(params)
-        gated = cls._form(params) == native.FORM_CLIPPED_GATED
+        form = cls._form(params)
+        gated = form != native.FORM_PLAIN_GELU
         per = 2 if gated else 1
         gu, down = [], []
         for e in range(E):
@@ -262,11 +287,22 @@ class RoutedExperts:
                 gu.append(Piece(f"experts.{e}.gate_proj.weight", e * 2 * ff))
             gu.append(Piece(f"experts.{e}.up_proj.weight", e * per * ff + (ff if gated else 0)))
             down.append(Piece(f"experts.{e}.down_proj.weight", e * hidden))
-        out = {"router.weight": Resident((E, hidden), torch.float32, (Piece("router.weight"),)),
+        router = (Piece("router.weight", 0),)
+        if cls._shared_gate(params):
+            router += (Piece("shared.gate.weight", E),)
+        out = {"router.weight": Resident((E + len(router) - 1, hidden), torch.float32, router),
                "experts.gate_up.weight": Resident((E * per * ff, hidden), pieces=tuple(gu)),
                "experts.down.weight": Resident((E * hidden, ff), pieces=tuple(down))}
         if params.get("router_bias", True):
             out["router.bias"] = Resident((E,), torch.float32, (Piece("router.bias"),))
+        if params.get("correction"):
+            out["router.bias"] = Resident((E,), torch.float32, (Piece("correction"),))
+        if sff and form == native.FORM_GATED_SILU:
+            for name, res in GatedMLP.resident(cls._shared_mlp(params), hidden).items():
+                out["shared." + name] = Resident(res.shape, res.dtype, tuple(
+                    Piece("shared." + q.source, q.row_offset, q.group, q.group_stride) for q in res.pieces),
+                    res.offset)
+            return out
         if sff and not gated:
             out["shared.gate_up.weight"] = Resident((sff, hidden), pieces=(Piece("shared.up_proj.weight"),))
         elif sff:
@@ -283,27 +319,38 @@ class RoutedExperts:
         self.form = self._form(params)
         self.score = _SCORES[params.get("score", "softmax_top")]
         self.plain = self.form == native.FORM_PLAIN_GELU
+        self.clipped = self.form == native.FORM_CLIPPED_GATED
         self.per = 1 if self.plain else 2          # matrix rows per middle column
-        self.limit = 0.0 if self.plain else float(params["limit"])
+        self.limit = float(params["limit"]) if self.clipped else 0.0
+        self.router_scale = float(params.get("router_scale", 1.0))
+        self.shared_gate = self._shared_gate(params)
         self.alpha = float(params.get("alpha", 1.702))
         self.w_router = weights["router.weight"]
         self.b_router = weights.get("router.bias")
         self.w_gu = rt.cast_matrix(weights["experts.gate_up.weight"]).view(self.E, self.per * self.ff, hidden)
         self.w_down = rt.cast_matrix(weights["experts.down.weight"]).view(self.E, hidden, self.ff)
-        self.shared_limit = float(params["shared"]["limit"]) if self.sff and not self.plain else 0.0
-        self.w_sgu = rt.cast_matrix(weights["shared.gate_up.weight"]) if self.sff else None
-        self.w_sdown = rt.cast_matrix(weights["shared.down.weight"]) if self.sff else None
+        self.shared_limit = float(params["shared"]["limit"]) if self.sff and self.clipped else 0.0
+        self.shared: Optional[GatedMLP] = None
+        self.w_sgu = self.w_sdown = None
+        if self.sff and self.form == native.FORM_GATED_SILU:
+            self.shared = GatedMLP(self._shared_mlp(params), hidden, {
+                k[len("shared."):]: v for k, v in weights.items() if k.startswith("shared.")}, rt)
+        elif self.sff:
+            self.w_sgu = rt.cast_matrix(weights["shared.gate_up.weight"])
+            self.w_sdown = rt.cast_matrix(weights["shared.down.weight"])
         # up to this many rows every (row, expert) pair streams its own expert's matrices
         self.pair_rows = 32
 
     def choose(self, x: torch.Tensor):
-        """(ids int32 [rows, top], weights 32-bit [rows, top]) of the rows' experts."""
+        """(ids int32 [rows, top], weights 32-bit [rows, top]) of the rows' experts, and the
+        shared expert's weight per row (32-bit [rows], None without such a gate)."""
         R = x.shape[0]
+        gate = torch.empty(R, dtype=torch.float32, device=x.device) if self.shared_gate else None
         if R <= self.pair_rows and (self.hidden + self.E + 4) * 4 <= 48 * 1024:
             ids = torch.empty((R, self.top), dtype=torch.int32, device=x.device)
             p = torch.empty((R, self.top), dtype=torch.float32, device=x.device)
-            native.router_rows(x, self.w_router, self.b_router, ids, p, self.score)
-            return ids, p
+            native.router_rows(x, self.w_router, self.b_router, ids, p, self.score, self.router_scale, gate)
+            return ids, p, gate
         x32 = x if x.dtype == torch.float32 else native.cast_rows(
             x, torch.empty(x.shape, dtype=torch.float32, device=x.device))
         with native.profile_region("library product (router, 32-bit)", (R + self.E) * self.hidden * 4,
@@ -311,15 +358,17 @@ class RoutedExperts:
             z = torch.matmul(x32, self.w_router.t())
         ids = torch.empty((R, self.top), dtype=torch.int32, device=x.device)
         p = torch.empty((R, self.top), dtype=torch.float32, device=x.device)
-        native.router_topk(z, self.b_router, ids, p, self.score)
-        return ids, p
+        native.router_topk(z, self.b_router, ids, p, self.score, self.router_scale, gate)
+        return ids, p, gate
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         rt, R = self.rt, x.shape[0]
         rt.flush()
-        ids, p = self.choose(x)
+        ids, p, base_weight = self.choose(x)
         base: Optional[torch.Tensor] = None
-        if self.sff and self.plain:
+        if self.shared is not None:
+            base = self.shared.forward(x, ctx)
+        elif self.sff and self.plain:
             # (the gelu is an epilogue of the up product where a hand-written product runs)
             base = rt.linear(rt.linear(x, self.w_sgu, epilogue=native.EPI_GELU), self.w_sdown)
         elif self.sff:
@@ -332,7 +381,7 @@ class RoutedExperts:
         streams = self.hidden * 4 <= 48 * 1024 and self.top * self.ff * 4 <= 48 * 1024
         if R <= self.pair_rows and streams and R * self.top < 65536:
             return native.routed_rows(x, self.w_gu, self.w_down, ids, p, base, out, self.limit, self.alpha,
-                                      self.form)
+                                      self.form, base_weight)
         # The pairs sorted by expert and laid out [experts, most, width] with `most` the largest
         # number of rows any expert got (the one number read on the host; rows behind an
         # expert's own are zeros): all experts run as ONE batched library product for gate and
@@ -374,7 +423,7 @@ class RoutedExperts:
                                    2.0 * E * most * W * self.ff):
             ys = torch.bmm(mid.view(E, most, self.ff), self.w_down.transpose(1, 2))
         return native.routed_combine(ys.view(E * most, W), where.view(R, top), None if self.plain else p,
-                                     base, out)
+                                     base, out, base_weight)
 
 
 register_feed_forward("gated_mlp", GatedMLP)

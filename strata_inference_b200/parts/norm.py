@@ -47,6 +47,10 @@ class RMSNorm:
         self.rt = rt
         self.gain = weights["gain"]
 
+    def scale_output(self, factor: float) -> None:
+        """The norm's output times a constant, in 32-bit (a head's scale on its logits)."""
+        self.gain = self.gain * factor
+
     def forward(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         n = x.shape[0] if rows is None else rows.numel()
@@ -101,6 +105,10 @@ class DynamicTanh:
         self.hidden = hidden
         self.rt = rt
         self.weight, self.b, self.alpha = weights["weight"], weights["b"], weights["alpha"]
+
+    def scale_output(self, factor: float) -> None:
+        """The norm's output times a constant, in 32-bit (a head's scale on its logits)."""
+        self.weight, self.b = self.weight * factor, self.b * factor
 
     @property
     def triple(self):

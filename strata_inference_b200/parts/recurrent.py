@@ -296,6 +296,8 @@ class Retention:
         if not hasattr(position, "rotary"):
             raise ConfigError("retention: the position part must offer rotary()")
         self.inv_freq, self.rot, style = position.rotary()
+        if getattr(position, "magnitude", 1.0) != 1.0:
+            raise ConfigError("retention: a rotation with a magnitude other than 1 is not built")
         if self.rot and style != native.ROPE_HALF_SPLIT:
             raise ConfigError("retention: q and k are rotated in half-split pairs")
         self.w_in = rt.cast_matrix(weights["in_proj.weight"])

@@ -15,6 +15,7 @@ from ..config.spec import ConfigError, PartSpec
 _REGISTRIES: Dict[str, Dict[str, type]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position": {},
     "block": {}, "embedding": {}, "head": {}, "joint": {}, "tail": {},
+    "mixer_input": {},
 }
 
 
@@ -60,6 +61,12 @@ def register_tail(kind: str, cls: type) -> type:
     """A part that runs behind a layer's sub-layers, on the stream itself: ``forward(x, ctx) -> y``
     with ``gain`` and ``eps`` of the RMS norm that y passes before it is added."""
     return _register("tail", kind, cls)
+
+
+def register_mixer_input(kind: str, cls: type) -> type:
+    """A part between a layer's first norm and its mixer: ``forward(x, ctx, entry) -> x'``, with
+    ``state_need()`` for what it keeps per slot and schedule entry."""
+    return _register("mixer_input", kind, cls)
 
 
 def part_class(role: str, kind: str) -> type:
