@@ -292,7 +292,7 @@ SIB_EXPORT int sib_add_norm_conv(const void* a, const float* post_gain, float po
                 "add_norm_conv: an argument is missing, or the state is too small");
     SIB_REQUIRE(((uintptr_t)a % 16) == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)y % 16) == 0 &&
                     ((uintptr_t)post_gain % 16) == 0 && ((uintptr_t)pre_gain % 16) == 0 && ((uintptr_t)w % 16) == 0 &&
-                    ((uintptr_t)state % 16) == 0 && state_stride % 4 == 0,
+                    (taps == 1 || (((uintptr_t)state % 16) == 0 && state_stride % 4 == 0)),
                 "add_norm_conv: operands must be 16-byte aligned");
     ConvArgs p{w, state, state_stride, nullptr, row_seq, seq_slot, nullptr, nullptr, nullptr, rows, channels, taps};
     const int threads = (channels / 8 + 31) / 32 * 32;
