@@ -160,6 +160,8 @@ def kv_bytes_per_step(engine, lengths):
         per_token = 2 * grp.need.n_kv_heads * grp.need.head_dim * grp.k.element_size()
         for n in lengths:
             seen = min(n, grp.need.window) if grp.need.window else n
+            if grp.need.window and getattr(grp.need, "keep_first", 0):
+                seen += min(max(0, n - grp.need.window), grp.need.keep_first)   # first positions kept for good
             if getattr(grp.need, "chunk", 0):
                 seen = (n - 1) % grp.need.chunk + 1                         # the row's own chunk
             if grp.need.window and getattr(grp.need, "pool", 0):
@@ -541,6 +543,23 @@ def besorax_config(size):
             "embedding": {"scale": 1.0}, "residual_mult": 0.5, "layers": layers}
 
 
+def kerolorn_config(size):
+    """Kerolorn at these sizes: every layer attention over a window of 1 024 positions that keeps the
+    first 64 (as many keys as Besorax's chunks of 1 024 hold at their end), a convolution of 4 taps
+    at its input, and Besorax's routed experts' sizes with gate matrices: 32 experts of an eighth of
+    the other models' width of which a row uses 4, beside a shared one of half that width."""
+    width, ff, heads, kv, hd, vocab, n_layers = KARUPEL_SIZES[size]
+    layer = {"type": "attention",
+             "mixer": {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+                       "mask": {"size": 1024, "keep_first": 64},
+                       "rot": {"base": 1000000.0, "dims": hd,
+                               "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+             "mlp": {"kind": "moe", "router": {"experts": 32, "top": 4, "scale": 2.0}, "expert": {"ff": ff // 8},
+                     "shared": {"ff": ff // 2}}}
+    return {"architecture": "Kerolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "canon": {"taps": 4}, "logit_scale": 0.5, "layers": [layer] * n_layers}
+
+
 def gemma2_config_like(size):
     width, ff, heads, kv, hd, vocab, n_layers = KARUPEL_SIZES[size]
     cfg = baseline_config()
@@ -552,7 +571,8 @@ def gemma2_config_like(size):
 
 def state_bytes_per_step(engine, batch):
     """Bytes of recurrent state a single-token step reads and writes."""
-    return sum(2 * batch * t[0].numel() * t.element_size() for t in engine.cache.state.values())
+    return sum(2 * batch * t[0].numel() * t.element_size()
+               for t in list(engine.cache.state.values()) + list(engine.cache.inputs.values()))
 
 
 def unread_expert_bytes(engine, rows):
@@ -568,14 +588,21 @@ def unread_expert_bytes(engine, rows):
 
 
 def spread_rows(engine):
-    """Dynamic Tanh norms of a randomly drawn model as the identity's neighbour (weight 1, b 0,
-    alpha 1).  Drawn like other norm weights (around 0, spread 0.1) they turn every row into
+    """Norms of a randomly drawn model as the identity's neighbour: RMS gains of 1, Dynamic Tanh norms with weight 1, b 0 and alpha 1, and
+    routers' corrections of 0.  Drawn like other norm weights (around 0, spread 0.1) they turn every row into
     nearly the same vector b, and a router then sends all rows of a step to the same experts:
     the experts' work would be that of the worst imbalance there is."""
     norms = [engine.model.final_norm]
     for blk in engine.model.blocks:
         norms += [getattr(blk, site, None) for site in ("pre_mixer", "post_mixer", "pre_ff", "post_ff")]
+    for blk in engine.model.blocks:
+        if getattr(blk.feed_forward, "b_router", None) is not None:
+            blk.feed_forward.b_router.zero_()
+        if getattr(blk.mixer, "temp", None) is not None:
+            blk.mixer.temp.fill_(1.0)
     for n in norms:
+        if n is not None and getattr(n, "gain", None) is not None:
+            n.gain.fill_(1.0)
         if n is not None and hasattr(n, "alpha") and hasattr(n, "b"):
             n.weight.fill_(1.0)
             n.b.zero_()
@@ -604,7 +631,7 @@ def run_karupel(args, pair=None, title="Karupel beside Gemma2"):
                                                max_slots=max(batches))
             engine = gen.engine
             randomize_pools(engine)
-            if name == "besorax":
+            if name in ("besorax", "kerolorn"):
                 spread_rows(engine)
             weight_bytes = engine.model.weight_bytes()
             row = {"weights_gb": round(weight_bytes / 1e9, 2)}
@@ -683,8 +710,11 @@ def main():
     ap.add_argument("--besorax", action="store_true",
                     help="Besorax beside Vavupel at equal layer sizes: a prompt step and single-token "
                          "steps (with --kernels the per-kernel tables of both)")
+    ap.add_argument("--kerolorn", action="store_true",
+                    help="Kerolorn beside Besorax at equal layer sizes: a prompt step and single-token "
+                         "steps (with --kernels the per-kernel tables of both)")
     ap.add_argument("--size", default="", choices=[""] + sorted(KARUPEL_SIZES),
-                    help="with --karupel, --vavupel, --gegorax or --besorax: one of the sizes (default: all)")
+                    help="with --karupel, --vavupel, --gegorax, --besorax or --kerolorn: one of the sizes (default: all)")
     ap.add_argument("--shape", default="2b", choices=sorted(SHAPES),
                     help="layer sizes: the 2B shape (the recorded line) or the 9B / 27B shapes")
     args = ap.parse_args()
@@ -708,6 +738,9 @@ def main():
     if args.besorax:
         return run_karupel(args, (("besorax", besorax_config), ("vavupel", vavupel_config)),
                            "Besorax beside Vavupel")
+    if args.kerolorn:
+        return run_karupel(args, (("kerolorn", kerolorn_config), ("besorax", besorax_config)),
+                           "Kerolorn beside Besorax")
     if args.karupel:
         return run_karupel(args)
     if args.kernels:

@@ -148,6 +148,94 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(HeadPrepareArgs p) {
     }
 }
 
+// The common case in 16-byte accesses: bfloat16, every head HD wide (64, 128 or 256), no biases and
+// no mixed values, neighbouring pairs on a multiple of 8 dimensions.  A thread owns 8 neighbouring
+// dimensions of the heads it works on, HD / 8 neighbouring lanes a head: a row's cosines and sines
+// are taken once a thread, ahead of the wait for the projection (positions, slots and page tables
+// are written by the host before the step), and serve all its heads.
+template <int HD>
+__global__ void __launch_bounds__(128) head_prepare_bf16_kernel(HeadPrepareArgs p) {
+    constexpr int LPH = HD / 8, UPB = 128 / LPH;
+    pdl_trigger();
+    const int r = blockIdx.x, d0 = ((int)threadIdx.x % LPH) * 8;
+    const int units = p.n_heads + 2 * p.n_kv;
+    const int pos = p.row_pos[r];
+    __nv_bfloat16 *k_cell = nullptr, *v_cell = nullptr;      // the row's cell of kv head 0
+    if (p.k_pool) {
+        const int b = p.row_seq[r], slot = p.seq_slot[b];
+        if (slot >= 0 && cell_written(pos, p.seq_end[b], p.fixed_tokens, p.ring_tokens)) {
+            const int cell = cell_of(pos, p.fixed_tokens, p.ring_tokens);
+            const int page = p.page_table[(size_t)slot * p.max_pages + cell / p.page_tokens];
+            const size_t at = ((size_t)page * p.n_kv * p.page_tokens + cell % p.page_tokens) * HD;
+            k_cell = (__nv_bfloat16*)p.k_pool + at;
+            v_cell = (__nv_bfloat16*)p.v_pool + at;
+        }
+    }
+    const bool turns = p.inv_freq && d0 < p.rot;
+    float c[4], s[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float ang = turns ? (float)pos * p.inv_freq[d0 / 2 + i] : 0.f;
+        c[i] = turns ? cosf(ang) * p.magnitude : 1.f;
+        s[i] = turns ? sinf(ang) * p.magnitude : 0.f;
+    }
+    pdl_wait();
+    const __nv_bfloat16* src = (const __nv_bfloat16*)p.proj + (size_t)r * p.proj_stride + d0;
+    __nv_bfloat16* dst = (__nv_bfloat16*)p.qkv + (size_t)r * units * HD + d0;
+    for (int u0 = blockIdx.y * UPB; u0 < units; u0 += gridDim.y * UPB) {     // (the same for a whole warp)
+        const int unit = u0 + (int)threadIdx.x / LPH;
+        const bool live = unit < units;
+        uint4 raw = make_uint4(0, 0, 0, 0);
+        if (live) raw = *reinterpret_cast<const uint4*>(src + (size_t)unit * HD);
+        if (live && unit >= p.n_heads + p.n_kv) {
+            *reinterpret_cast<uint4*>(dst + (size_t)unit * HD) = raw;
+            if (v_cell)
+                *reinterpret_cast<uint4*>(v_cell + (size_t)(unit - p.n_heads - p.n_kv) * p.page_tokens * HD + d0) = raw;
+        }
+        const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+        float x[8];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            x[2 * i] = __uint_as_float(w[i] << 16);
+            x[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+        }
+        auto head_sum = [&]() {                  // of the squares, over the head's lanes
+            float t = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) t += x[i] * x[i];
+#pragma unroll
+            for (int o = LPH / 2; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+            return t;
+        };
+        const bool is_q = unit < p.n_heads;
+        if (p.norm == NORM_BEFORE) {
+            const float inv = 1.0f / sqrtf(head_sum() / (float)HD + p.eps);
+            const float* gain = (is_q ? p.q_gain : p.k_gain) + d0;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] *= inv * gain[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float a = x[2 * i], b = x[2 * i + 1];
+            x[2 * i] = a * c[i] - b * s[i];
+            x[2 * i + 1] = b * c[i] + a * s[i];
+        }
+        float factor = p.temp && live && is_q ? p.temp[unit] : 1.f;
+        if (p.norm == NORM_AFTER) factor *= 1.0f / sqrtf(head_sum() / (float)HD + p.eps);
+        if (!live || unit >= p.n_heads + p.n_kv) continue;
+        uint32_t o[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const __nv_bfloat162 pr = __floats2bfloat162_rn(x[2 * i] * factor, x[2 * i + 1] * factor);
+            o[i] = *reinterpret_cast<const uint32_t*>(&pr);
+        }
+        const uint4 out = make_uint4(o[0], o[1], o[2], o[3]);
+        *reinterpret_cast<uint4*>(dst + (size_t)unit * HD) = out;
+        if (!is_q && k_cell)
+            *reinterpret_cast<uint4*>(k_cell + (size_t)(unit - p.n_heads) * p.page_tokens * HD + d0) = out;
+    }
+}
+
 SIB_EXPORT int sib_head_prepare(
     const void* proj, long long proj_stride, void* qkv, int dtype, const float* bias,
     const float* q_gain, const float* k_gain, float eps, const float* inv_freq, int rot,
@@ -179,6 +267,18 @@ SIB_EXPORT int sib_head_prepare(
                       ring_tokens, eps, norm_after ? NORM_AFTER : (q_gain ? NORM_BEFORE : NORM_NONE), temp,
                       magnitude, fixed_tokens, neighbours};
     const int units = n_heads + 2 * n_kv;
+    if (dtype == SIB_BF16 && kd == vd && kd == pad && (pad == 64 || pad == 128 || pad == 256) && !bias && !v_first &&
+        (rot == 0 || (neighbours && rot % 8 == 0)) && proj_stride % 8 == 0 && ((uintptr_t)proj % 16) == 0 &&
+        ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)k_pool % 16) == 0 && ((uintptr_t)v_pool % 16) == 0 && rows < (1 << 30)) {
+        // few rows: a row's heads over several blocks; many: a block a row
+        const int per = 128 / (pad / 8), passes = (units + per - 1) / per;
+        const dim3 grid(rows, rows < 512 ? (passes < 65535 ? passes : 65535) : 1);
+        cudaStream_t s = (cudaStream_t)stream;
+        if (pad == 64) sib_launch_chained(head_prepare_bf16_kernel<64>, grid, dim3(128), 0, s, p);
+        else if (pad == 128) sib_launch_chained(head_prepare_bf16_kernel<128>, grid, dim3(128), 0, s, p);
+        else sib_launch_chained(head_prepare_bf16_kernel<256>, grid, dim3(128), 0, s, p);
+        return sib_check_launch("head_prepare");
+    }
     const size_t smem = (size_t)4 * pad * sizeof(float);
     SIB_REQUIRE(smem <= 48 * 1024, "head_prepare: heads of %d are too wide", pad);
     SIB_REQUIRE(rows < 65536 * 32767ll && (units + 3) / 4 < 65536, "head_prepare: too many rows");

@@ -69,8 +69,10 @@ template <> struct Pack<__nv_bfloat16> {
 };
 
 // A thread takes V channels of RUN neighbouring rows (V 1: any layout).  SINGLE: every sequence
-// has one row, and the thread that read a slot's state moves it on.
-template <typename T, int V, int RUN, bool SINGLE>
+// has one row, and the thread that read a slot's state moves it on.  TAPS > 0 (= p.taps): a run
+// inside one sequence whose first row has all its predecessors in this step asks for its rows
+// at once and goes from row to row in registers.
+template <typename T, int V, int RUN, bool SINGLE, int TAPS = 0>
 __global__ void __launch_bounds__(128)
 short_conv_kernel(const T* __restrict__ x, T* __restrict__ y, ConvArgs p) {
     pdl_trigger();
@@ -78,8 +80,32 @@ short_conv_kernel(const T* __restrict__ x, T* __restrict__ y, ConvArgs p) {
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (c >= p.channels) return;
     const int C = p.channels, taps = p.taps;
-    const int r1 = min((int)(blockIdx.y + 1) * RUN, p.rows);
-    for (int r = blockIdx.y * RUN; r < r1; ++r) {
+    const int r0 = blockIdx.y * RUN, r1 = min(r0 + RUN, p.rows);
+    if constexpr (TAPS > 0 && V > 1 && !SINGLE) {
+        const int b0 = p.row_seq[r0];
+        if (r0 + RUN <= p.rows && p.row_seq[r0 + RUN - 1] == b0 && p.row_pos[r0] - p.seq_start[b0] >= TAPS - 1) {
+            float in[RUN + TAPS - 1][V];
+#pragma unroll
+            for (int k = 0; k < RUN + TAPS - 1; ++k) Pack<T>::load(x + (size_t)(r0 - (TAPS - 1) + k) * C + c, in[k]);
+            float acc[RUN][V];
+#pragma unroll
+            for (int q = 0; q < RUN; ++q)
+#pragma unroll
+                for (int i = 0; i < V; ++i) acc[q][i] = in[q + TAPS - 1][i];
+#pragma unroll
+            for (int j = TAPS - 1; j >= 0; --j)
+#pragma unroll
+                for (int i = 0; i < V; ++i) {
+                    const float w = p.w[(size_t)j * C + c + i];
+#pragma unroll
+                    for (int q = 0; q < RUN; ++q) acc[q][i] += w * in[q + j][i];
+                }
+#pragma unroll
+            for (int q = 0; q < RUN; ++q) Pack<T>::store(y + (size_t)(r0 + q) * C + c, acc[q]);
+            return;
+        }
+    }
+    for (int r = r0; r < r1; ++r) {
         const int b = p.row_seq[r], slot = p.seq_slot[b];
         const int back = p.row_pos[r] - p.seq_start[b];          // rows of this step before this one
         float* hist = slot >= 0 ? p.state + (size_t)slot * p.state_stride : nullptr;
@@ -265,6 +291,12 @@ SIB_EXPORT int sib_short_conv(const void* x, void* y, int dtype, const float* w,
             sib_launch_chained(short_conv_kernel<T, Pack<T>::V, 1, true>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
         else if (single)
             sib_launch_chained(short_conv_kernel<T, 1, 1, true>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
+        else if (wide && taps == 4)
+            sib_launch_chained(short_conv_kernel<T, Pack<T>::V, RUN, false, 4>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
+        else if (wide && taps == 3)
+            sib_launch_chained(short_conv_kernel<T, Pack<T>::V, RUN, false, 3>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
+        else if (wide && taps == 2)
+            sib_launch_chained(short_conv_kernel<T, Pack<T>::V, RUN, false, 2>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
         else if (wide)
             sib_launch_chained(short_conv_kernel<T, Pack<T>::V, RUN, false>, grid, dim3(128), 0, s, (const T*)x, (T*)y, p);
         else
