@@ -284,7 +284,20 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 //               the first block's barrier
 // Every mbarrier wait is bounded; both blocks meet at a cluster barrier before they
 // free their tensor memory and leave.
+//
+// GROUPED products: the rows of x lie sorted by group (the expert they chose) and every group has a
+// matrix of its own, W[groups * rows per group, K].  The tiles of 256 activation rows are a list
+// that an earlier kernel wrote (routed.cu expert_plan): first row, rows, group; the host knows
+// neither how many there are nor how the rows fell.  A tile's rows behind its own belong to other
+// groups and are not stored.  The column tiles of a row tile are neighbours in the walk, and so
+// are the row tiles of a group, so that a group's matrix comes from memory about once.
+//   GROUP_PLAIN   y = x . W_g^T, p.N outputs, p.N matrix rows per group
+//   GROUP_GATED   a group's matrix is [p.N gate rows; p.N up rows]: a tile of 128 outputs takes 128
+//                 gate rows into the first block's half and the matching up rows into the second's, so
+//                 that a gate and its up value are 128 accumulator columns apart, and stores
+//                 act(gate) * up (the gated epilogues)
 // ---------------------------------------------------------------------------
+enum { GROUP_NONE = 0, GROUP_PLAIN = 1, GROUP_GATED = 2 };
 static constexpr int PAIR_BN = 256;        // weight rows per tile (128 per block in shared memory)
 static constexpr int PAIR_STAGES = 6;
 
@@ -372,10 +385,10 @@ __device__ __forceinline__ void store_run<float>(float* dst, const float (&o)[32
     }
 }
 
-template <typename OutT>
+template <typename OutT, int GROUP = GROUP_NONE>
 __global__ void __launch_bounds__(192)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                         GemmArgs p) {
+                         GemmArgs p, const int* __restrict__ list) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     constexpr uint32_t A_BYTES = 128 * BK * 2, B_BYTES = (PAIR_BN / 2) * BK * 2;
     constexpr uint32_t STAGE = A_BYTES + B_BYTES;
@@ -390,7 +403,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = cluster_ctarank();
     const int pair = blockIdx.x >> 1, pairs = gridDim.x >> 1;
-    const int tiles_m = (p.R + 255) / 256, tiles_n = (p.N + PAIR_BN - 1) / PAIR_BN;
+    constexpr int OUT_N = GROUP == GROUP_GATED ? PAIR_BN / 2 : PAIR_BN;      // outputs of a tile
+    const int tiles_m = GROUP ? list[0] : (p.R + 255) / 256, tiles_n = (p.N + OUT_N - 1) / OUT_N;
     const int n_tiles = tiles_m * tiles_n;
     const int k_blocks = (p.K + BK - 1) / BK;
 
@@ -424,8 +438,16 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
             uint32_t it = 0;     // k-blocks loaded so far
             bool ok = true;
             for (int tile = pair; tile < n_tiles && ok; tile += pairs) {
-                const int m0 = (tile % tiles_m) * 256 + 128 * (int)rank;
-                const int n0 = (tile / tiles_m) * PAIR_BN + (PAIR_BN / 2) * (int)rank;
+                int m0, n0;
+                if constexpr (GROUP == GROUP_NONE) {
+                    m0 = (tile % tiles_m) * 256 + 128 * (int)rank;
+                    n0 = (tile / tiles_m) * PAIR_BN + (PAIR_BN / 2) * (int)rank;
+                } else {
+                    const int* at = list + 1 + 3 * (tile / tiles_n);
+                    m0 = at[0] + 128 * (int)rank;
+                    n0 = GROUP == GROUP_GATED ? at[2] * 2 * p.N + (tile % tiles_n) * OUT_N + p.N * (int)rank
+                                              : at[2] * p.N + (tile % tiles_n) * OUT_N + (PAIR_BN / 2) * (int)rank;
+                }
                 for (int kb = 0; kb < k_blocks; ++kb, ++it) {
                     const int s = it % PAIR_STAGES;
                     const uint32_t round = it / PAIR_STAGES;
@@ -477,16 +499,37 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
             const uint32_t b = done & 1;
             if (!mbar_wait(&acc_full[b], (done >> 1) & 1)) { if (lane == 0) *failed = 3; ok = false; break; }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-            const int r = (tile % tiles_m) * 256 + 128 * (int)rank + 32 * quarter + lane;   // activation row
-            const int n0 = (tile / tiles_m) * PAIR_BN;
+            const int in_tile = 128 * (int)rank + 32 * quarter + lane;
+            int r, n0, r_end;                                       // activation row; first output
+            if constexpr (GROUP == GROUP_NONE) {
+                r = (tile % tiles_m) * 256 + in_tile;
+                n0 = (tile / tiles_m) * PAIR_BN;
+                r_end = p.R;
+            } else {
+                const int* at = list + 1 + 3 * (tile / tiles_n);
+                r = at[0] + in_tile;
+                r_end = at[0] + at[1];
+                n0 = (tile % tiles_n) * OUT_N;
+            }
 #pragma unroll 1
-            for (int c0 = 0; c0 < PAIR_BN; c0 += 32) {
+            for (int c0 = 0; c0 < OUT_N; c0 += 32) {
                 uint32_t v[32];
+                if (GROUP != GROUP_NONE) __syncwarp();      // (the lanes' rows end apart; the load is the warp's)
                 tmem_ld32(tmem + ((uint32_t)(32 * quarter) << 16) + 256 * b + (uint32_t)c0, v);
                 const int n = n0 + c0;
-                if (r >= p.R || n >= p.N) continue;
                 float o[32];
-                if (gemm_gated(p.epilogue)) {
+                if constexpr (GROUP == GROUP_GATED) {
+                    uint32_t u[32];
+                    tmem_ld32(tmem + ((uint32_t)(32 * quarter) << 16) + 256 * b + (uint32_t)(OUT_N + c0), u);
+                    if (r >= r_end || n >= p.N) continue;
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        o[j] = gemm_gated_pair(__uint_as_float(v[j]), __uint_as_float(u[j]), p.epilogue, p.cap);
+                    store_run<OutT>(y + (size_t)r * p.y_stride + n, o, min(32, p.N - n));
+                    continue;
+                }
+                if (r >= r_end || n >= p.N) continue;
+                if (GROUP == GROUP_NONE && gemm_gated(p.epilogue)) {
                     // weight rows come as 8 gates then their 8 ups: 32 columns make 16 outputs
 #pragma unroll
                     for (int g = 0; g < 2; ++g)
@@ -598,18 +641,20 @@ static int launch_gemm(const CUtensorMap& mw, const CUtensorMap& mx, const GemmA
     return sib_check_launch("gemm_tcgen05");
 }
 
-template <typename OutT>
+// `list` with GROUP: the row tiles, of which there are at most `most_tiles`.
+template <typename OutT, int GROUP = GROUP_NONE>
 static int launch_pair(const CUtensorMap& mx, const CUtensorMap& mw, const GemmArgs& p, int sm_count,
-                       cudaStream_t s) {
+                       cudaStream_t s, const int* list = nullptr, int most_tiles = 0) {
     const size_t smem = 1024 + (size_t)PAIR_STAGES * (128 * BK * 2 + (PAIR_BN / 2) * BK * 2) +
                         (2 * PAIR_STAGES + 4) * 8 + 16;
-    auto kernel = gemm_tcgen05_pair_kernel<OutT>;
+    auto kernel = gemm_tcgen05_pair_kernel<OutT, GROUP>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) {
         sib_set_error("gemm_tcgen05: shared memory: %s", cudaGetErrorString(e));
         return (int)e;
     }
-    const int n_tiles = ((p.R + 255) / 256) * ((p.N + PAIR_BN - 1) / PAIR_BN);
+    const int out_n = GROUP == GROUP_GATED ? PAIR_BN / 2 : PAIR_BN;
+    const int n_tiles = (GROUP ? most_tiles : (p.R + 255) / 256) * ((p.N + out_n - 1) / out_n);
     const int pairs = n_tiles < sm_count / 2 ? n_tiles : sm_count / 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(2 * pairs, 1, 1);
@@ -623,7 +668,7 @@ static int launch_pair(const CUtensorMap& mx, const CUtensorMap& mw, const GemmA
     attr[0].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    e = cudaLaunchKernelEx(&cfg, kernel, mx, mw, p);
+    e = cudaLaunchKernelEx(&cfg, kernel, mx, mw, p, list);
     if (e != cudaSuccess) {
         sib_set_error("gemm_tcgen05: launch of the paired kernel failed: %s", cudaGetErrorString(e));
         return (int)e;
@@ -701,4 +746,39 @@ SIB_EXPORT int sib_gemm_tcgen05_one_block(const void* W, const void* x, void* y,
                                           int N, int K, long long x_stride, int y_stride,
                                           int epilogue, float cap, void* stream) {
     return gemm_tcgen05(W, x, y, out_dtype, R, N, K, x_stride, y_stride, epilogue, cap, 1, stream);
+}
+
+// Products of rows sorted by group with their groups' matrices (see GROUPED above).  `W`: [groups *
+// N, K], or with a gated epilogue [groups * 2 N, K] (a group's N gate rows, then its N up rows); y:
+// [R, N] bfloat16; `list` (device): the number of row tiles, then first row, rows and group of each,
+// at most `most_tiles` of them.
+SIB_EXPORT int sib_gemm_tcgen05_grouped(const void* W, const void* x, void* y, const int* list, int most_tiles,
+                                        int groups, int R, int N, int K, int epilogue, float cap, void* stream) {
+    if (R == 0) return 0;
+    SIB_REQUIRE(R > 0 && N > 0 && K > 0 && K % 8 == 0 && groups > 0 && most_tiles > 0 && list,
+                "gemm_tcgen05_grouped: R=%d N=%d K=%d (a multiple of 8) groups=%d", R, N, K, groups);
+    const bool gated = epilogue == GEMM_EPI_SWIGLU || epilogue == GEMM_EPI_CLIPPED;
+    SIB_REQUIRE(gated || epilogue == GEMM_EPI_NONE, "gemm_tcgen05_grouped: epilogue %d is not built", epilogue);
+    SIB_REQUIRE(epilogue != GEMM_EPI_CLIPPED || cap > 0.f, "gemm_tcgen05_grouped: the clipped gate's limit must be positive");
+    SIB_REQUIRE(((uintptr_t)W % 16) == 0 && ((uintptr_t)x % 16) == 0,
+                "gemm_tcgen05_grouped: operands must be 16-byte aligned");
+    const long long w_rows = (long long)groups * N * (gated ? 2 : 1);
+    SIB_REQUIRE(w_rows + 2ll * N < (1ll << 31) && (long long)most_tiles * ((N + 127) / 128) < (1ll << 31),
+                "gemm_tcgen05_grouped: too many matrix rows (%lld)", w_rows);
+    int dev = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    SIB_REQUIRE(e == cudaSuccess && dev >= 0 && dev < 64, "gemm_tcgen05_grouped: no current device");
+    int* error_flag = sib_error_word(SIB_ERR_GEMM_TCGEN05);
+    if (!error_flag) return -1;
+    if (!g_sm_count[dev]) {
+        e = cudaDeviceGetAttribute(&g_sm_count[dev], cudaDevAttrMultiProcessorCount, dev);
+        SIB_REQUIRE(e == cudaSuccess && g_sm_count[dev] >= 2, "gemm_tcgen05_grouped: %s", cudaGetErrorString(e));
+    }
+    CUtensorMap mx, mw;
+    if (make_map(&mx, x, R, K, K, 128)) return -1;
+    if (make_map(&mw, W, (int)w_rows, K, K, PAIR_BN / 2)) return -1;
+    GemmArgs p{y, error_flag, R, N, K, N, epilogue, cap};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (gated) return launch_pair<__nv_bfloat16, GROUP_GATED>(mx, mw, p, g_sm_count[dev], s, list, most_tiles);
+    return launch_pair<__nv_bfloat16, GROUP_PLAIN>(mx, mw, p, g_sm_count[dev], s, list, most_tiles);
 }

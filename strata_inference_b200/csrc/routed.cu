@@ -12,6 +12,10 @@
 //                    the order of the choice, on top of an optional base row.
 //   routed_expert_*  many pairs in a recorded step: expert-major, each expert's matrices read
 //                    from memory once for all the pairs that chose it, then routed_combine.
+//   expert_plan      many rows: where every (row, expert) pair lies when the pairs are sorted by expert,
+//                    and the list of tiles of 256 sorted rows that the grouped products walk
+//                    (gemm_tcgen05.cu); all on the device.
+//   spread_rows      the rows of x copied to their pairs' places in that order.
 //   routed_combine   many rows (experts run as products over sorted rows): the same sum
 //                    from the pairs' outputs, found through the sort's inverse.
 //
@@ -495,6 +499,67 @@ routed_expert_down_kernel(const T* __restrict__ mid, const T* __restrict__ w_dow
     }
 }
 
+// One block.  `where[pair]`: the pair's place among the pairs sorted by expert (the order inside an
+// expert is arbitrary: no row's result depends on it).  `list`: how many tiles of up to 256 sorted
+// rows there are, then first row, rows and expert of each; no tile spans two experts.
+__global__ void __launch_bounds__(1024)
+expert_plan_kernel(const int* __restrict__ ids, int pairs, int experts, int* __restrict__ where,
+                   int* __restrict__ list) {
+    __shared__ int count[1024], rows_to[1024], tiles_to[1024];
+    pdl_trigger();
+    pdl_wait();
+    const int t = threadIdx.x;
+    count[t] = 0;
+    __syncthreads();
+    for (int i = t; i < pairs; i += 1024) atomicAdd(&count[ids[i]], 1);
+    __syncthreads();
+    const int mine = count[t], my_tiles = (mine + 255) / 256;
+    rows_to[t] = mine;
+    tiles_to[t] = my_tiles;
+    __syncthreads();
+    for (int d = 1; d < 1024; d <<= 1) {         // inclusive sums
+        const int r = t >= d ? rows_to[t - d] : 0, n = t >= d ? tiles_to[t - d] : 0;
+        __syncthreads();
+        rows_to[t] += r;
+        tiles_to[t] += n;
+        __syncthreads();
+    }
+    const int row0 = rows_to[t] - mine, tile0 = tiles_to[t] - my_tiles;
+    if (t < experts)
+        for (int k = 0; k < my_tiles; ++k) {
+            int* at = list + 1 + 3 * (tile0 + k);
+            at[0] = row0 + 256 * k;
+            at[1] = min(256, mine - 256 * k);
+            at[2] = t;
+        }
+    if (t == 1023) list[0] = tiles_to[t];
+    count[t] = row0;
+    __syncthreads();
+    for (int i = t; i < pairs; i += 1024) where[i] = atomicAdd(&count[ids[i]], 1);
+}
+
+// xs[where[r, k]] = x[r]: a block per row.  16 bytes at a time where the rows allow it.
+template <typename T>
+__global__ void __launch_bounds__(128)
+spread_rows_kernel(const T* __restrict__ x, long long x_stride, const int* __restrict__ where,
+                   T* __restrict__ xs, int width, int top, bool wide) {
+    pdl_trigger();
+    pdl_wait();
+    const int r = blockIdx.x;
+    const T* row = x + (size_t)r * x_stride;
+    if (wide) {
+        constexpr int PER = 16 / (int)sizeof(T);
+        for (int c = threadIdx.x; c < width / PER; c += 128) {
+            const uint4 v = reinterpret_cast<const uint4*>(row)[c];
+            for (int k = 0; k < top; ++k)
+                reinterpret_cast<uint4*>(xs + (size_t)where[r * top + k] * width)[c] = v;
+        }
+    } else {
+        for (int c = threadIdx.x; c < width; c += 128)
+            for (int k = 0; k < top; ++k) xs[(size_t)where[r * top + k] * width + c] = row[c];
+    }
+}
+
 template <typename T>
 __global__ void routed_combine_kernel(const T* __restrict__ ys, const int* __restrict__ where,
                                       const float* __restrict__ weights, const T* __restrict__ base,
@@ -685,4 +750,35 @@ SIB_EXPORT int sib_routed_combine(const void* ys, const int* where, const float*
                                                  where, weights, (const T*)base, base_weight, (T*)out, width,
                                                  top, total));
     return sib_check_launch("routed_combine");
+}
+
+// The most row tiles that `pairs` pairs of `experts` experts can make.
+static long long most_row_tiles(long long pairs, int experts) {
+    return pairs / 256 + (pairs < experts ? pairs : experts);
+}
+
+SIB_EXPORT int sib_expert_plan(const int* ids, int rows, int top, int experts, int* where, int* list,
+                               int list_tiles, void* stream) {
+    if (rows == 0) return 0;
+    const long long pairs = (long long)rows * top;
+    SIB_REQUIRE(rows > 0 && top > 0 && experts > 0 && experts <= 1024 && pairs < (1ll << 30),
+                "expert_plan: rows=%d top=%d experts=%d (at most 1024)", rows, top, experts);
+    SIB_REQUIRE(ids && where && list && list_tiles >= most_row_tiles(pairs, experts),
+                "expert_plan: room for %d tiles, up to %lld are needed", list_tiles, most_row_tiles(pairs, experts));
+    sib_launch_chained(expert_plan_kernel, dim3(1), dim3(1024), 0, (cudaStream_t)stream, ids, (int)pairs, experts,
+                       where, list);
+    return sib_check_launch("expert_plan");
+}
+
+SIB_EXPORT int sib_spread_rows(const void* x, long long x_stride, const int* where, void* xs, int dtype,
+                               int rows, int width, int top, void* stream) {
+    if (rows == 0) return 0;
+    SIB_REQUIRE(rows > 0 && width > 0 && top > 0 && x && where && xs, "spread_rows: rows=%d width=%d top=%d",
+                rows, width, top);
+    const int per = dtype == SIB_F32 ? 4 : 8;
+    const bool wide = width % per == 0 && x_stride % per == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)xs % 16) == 0;
+    SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(spread_rows_kernel<T>, dim3(rows), dim3(128), 0,
+                                                 (cudaStream_t)stream, (const T*)x, x_stride, where, (T*)xs,
+                                                 width, top, wide));
+    return sib_check_launch("spread_rows");
 }

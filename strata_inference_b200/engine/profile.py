@@ -90,8 +90,8 @@ def profile_prompt_graph(engine, slot: int, tokens, replays: int = 3) -> Tuple[L
     n = len(eager.events)
     torch.cuda.synchronize()
     begin, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    if any(getattr(getattr(b, "feed_forward", None), "reads_sizes_on_host", False)
-           for b in engine.model.blocks):
+    if any(hasattr(b.feed_forward, "reads_sizes_on_host") and b.feed_forward.reads_sizes_on_host(len(tokens))
+           for b in engine.model.blocks if hasattr(b, "feed_forward")):
         # a part that reads sizes on the host for a step of many rows (routed experts: how many
         # rows chose each expert) cannot be captured as launched here: the launches are timed
         # as they are, and the total includes the host's share

@@ -652,6 +652,58 @@ def routed_rows(x: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: 
     return out
 
 
+@_timed(lambda ids, experts: ("expert_plan", 2 * _nbytes(ids), 0))
+def expert_plan(ids: torch.Tensor, experts: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """(``where`` int32 [rows, top]: each (row, expert) pair's place among the pairs sorted by
+    expert; ``tiles`` int32: how many tiles of up to 256 sorted rows there are, then first row, rows
+    and expert of each), both made on the device (csrc/routed.cu)."""
+    _want(ids, torch.int32, "ids")
+    rows, top = ids.shape
+    most = rows * top // 256 + min(experts, rows * top)
+    where = torch.empty((rows, top), dtype=torch.int32, device=ids.device)
+    tiles = torch.empty(1 + 3 * most, dtype=torch.int32, device=ids.device)
+    _check(library().sib_expert_plan(_ptr(ids), c_int(rows), c_int(top), c_int(experts), _ptr(where), _ptr(tiles),
+                                     c_int(most), _stream()))
+    return where, tiles
+
+
+@_timed(lambda x, where, xs: ("spread_rows", _nbytes(x, xs), 0))
+def spread_rows(x: torch.Tensor, where: torch.Tensor, xs: torch.Tensor) -> torch.Tensor:
+    """xs[where[r, k]] = x[r]: the rows at their pairs' places in the order of the experts."""
+    rows, width = x.shape
+    _want(x, xs.dtype, "x", contiguous=False)
+    _want(xs, xs.dtype, "xs")
+    _want(where, torch.int32, "where")
+    if x.stride(1) != 1 or where.shape[0] != rows or tuple(xs.shape) != (where.numel(), width):
+        raise KernelError("spread_rows: one place per pair")
+    _check(library().sib_spread_rows(_ptr(x), c_longlong(x.stride(0)), _ptr(where), _ptr(xs), _code(xs.dtype),
+                                     c_int(rows), c_int(width), c_int(where.shape[1]), _stream()))
+    return xs
+
+
+@_timed(lambda x, w, tiles, out, *a, **kw: (
+    f"gemm_tcgen05_grouped {w.shape[0]} x {w.shape[1]}x{w.shape[2]}", _nbytes(x, w, out),
+    2.0 * x.shape[0] * w.shape[1] * w.shape[2]))
+def gemm_tcgen05_grouped(x: torch.Tensor, w: torch.Tensor, tiles: torch.Tensor, out: torch.Tensor,
+                         epilogue: int = EPI_NONE, cap: float = 0.0) -> torch.Tensor:
+    """Rows sorted by group times their groups' matrices on tcgen05 (csrc/gemm_tcgen05.cu): ``w``
+    ``[groups, N, K]``, ``tiles`` as :func:`expert_plan` makes them; ``out`` ``[rows, N]``.
+    EPI_SWIGLU and EPI_CLIPPED (``cap`` the limit): ``w`` ``[groups, 2 N, K]``, N gate rows and then N
+    up rows, and out = act(gate) * up (the clipped gate's constant is 1.702)."""
+    for t, nm in ((x, "x"), (w, "w"), (out, "out")):
+        _want(t, torch.bfloat16, nm)
+    _want(tiles, torch.int32, "tiles")
+    (R, K), (groups, w_rows, w_k), n_out = x.shape, w.shape, out.shape[1]
+    most = (tiles.numel() - 1) // 3
+    if w_k != K or out.shape[0] != R or w_rows != n_out * (2 if epilogue in GATED_EPILOGUES else 1) \
+            or most < R // 256 + min(groups, R):
+        raise KernelError("gemm_tcgen05_grouped: shapes do not fit")
+    _check(library().sib_gemm_tcgen05_grouped(
+        _ptr(w), _ptr(x), _ptr(out), _ptr(tiles), c_int(most), c_int(groups), c_int(R), c_int(n_out), c_int(K),
+        c_int(epilogue), c_float(cap), _stream()))
+    return out
+
+
 @_timed(lambda ys, where, weights, base, out, base_weight=None: ("routed_combine", _nbytes(ys, out), 0))
 def routed_combine(ys: torch.Tensor, where: torch.Tensor, weights: Optional[torch.Tensor],
                    base: Optional[torch.Tensor], out: torch.Tensor,

@@ -35,6 +35,10 @@ without the correction and not normalized, times ``router_scale`` (default 1).
 ``shared["gate"]`` True: the shared expert's output is multiplied by sigmoid(shared.gate.weight x),
 one number per row (the gate's row lies behind the router's, so that one 32-bit product makes
 both; the factor is applied in 32-bit where the experts' outputs are summed).
+More than 128 bfloat16 rows of gated experts (recorded or not): the pairs are sorted by expert on the
+device and all experts run as two grouped tcgen05 products over tiles of 256 sorted rows
+(csrc/gemm_tcgen05.cu), the gated activation in the first one's epilogue; the host reads nothing,
+and experts with many rows cost what their rows cost.
 Few rows, and every recorded step: each (row, expert) pair streams its expert's matrices
 (csrc/routed.cu routed_rows).  Many rows: the pairs are sorted by expert on the device into a
 layout [experts, most rows of any expert, width] (that one number is read on the host; a recorded
@@ -44,6 +48,7 @@ products around one activation launch.
 
 from __future__ import annotations
 
+import os
 from typing import Dict, Mapping
 
 import torch
@@ -217,7 +222,15 @@ _SCORES = {"softmax_top": native.SCORE_SOFTMAX_TOP, "sigmoid": native.SCORE_SIGM
 
 class RoutedExperts:
     captures_prompts = True   # a recorded step reads the choices on the device only
-    reads_sizes_on_host = True   # a launched step of many rows reads how many rows chose each expert
+
+    def reads_sizes_on_host(self, rows: int) -> bool:
+        """Whether a launched step of so many rows reads on the host how many rows chose each expert."""
+        return rows > self.pair_rows and not self._grouped(rows)
+
+    def _grouped(self, rows: int) -> bool:
+        return (rows >= self.grouped_rows and self.rt.dtype == torch.bfloat16 and self.hidden % 8 == 0
+                and self.ff % 8 == 0 and self.E <= 1024
+                and (self.form == native.FORM_GATED_SILU or (self.clipped and self.alpha == 1.702)))
 
     @staticmethod
     def _sizes(params: Mapping):
@@ -340,6 +353,8 @@ class RoutedExperts:
             self.w_sdown = rt.cast_matrix(weights["shared.down.weight"])
         # up to this many rows every (row, expert) pair streams its own expert's matrices
         self.pair_rows = 32
+        # from this many rows on gated experts run as grouped products (SIB_GROUPED_EXPERTS=0: never)
+        self.grouped_rows = 129 if os.environ.get("SIB_GROUPED_EXPERTS", "1") != "0" else 1 << 40
 
     def choose(self, x: torch.Tensor):
         """(ids int32 [rows, top], weights 32-bit [rows, top]) of the rows' experts, and the
@@ -382,6 +397,15 @@ class RoutedExperts:
         if R <= self.pair_rows and streams and R * self.top < 65536:
             return native.routed_rows(x, self.w_gu, self.w_down, ids, p, base, out, self.limit, self.alpha,
                                       self.form, base_weight)
+        if self._grouped(R):
+            where, tiles = native.expert_plan(ids, self.E)
+            xs = native.spread_rows(x, where, torch.empty((R * self.top, self.hidden), dtype=x.dtype, device=x.device))
+            mid = torch.empty((R * self.top, self.ff), dtype=x.dtype, device=x.device)
+            native.gemm_tcgen05_grouped(xs, self.w_gu, tiles, mid, native.EPI_CLIPPED if self.clipped else
+                                        native.EPI_SWIGLU, self.limit)
+            # (the sorted rows have been read: their place takes the outputs)
+            ys = native.gemm_tcgen05_grouped(mid, self.w_down, tiles, xs)
+            return native.routed_combine(ys, where, p, base, out, base_weight)
         # The pairs sorted by expert and laid out [experts, most, width] with `most` the largest
         # number of rows any expert got (the one number read on the host; rows behind an
         # expert's own are zeros): all experts run as ONE batched library product for gate and

@@ -904,3 +904,57 @@ def test_command_line_generates_from_a_model_folder(tmp_path):
     for k, tok in enumerate(tokens):
         row = logits[len(prompt) + k - 1]
         assert (row.max() - row[tok]).item() <= 1e-4 * row.abs().max().item()
+
+
+@pytest.mark.parametrize("rows, top, experts", [(1, 1, 1), (130, 2, 5), (300, 3, 40), (700, 1, 3), (900, 4, 1024)])
+def test_pairs_sorted_by_expert(rows, top, experts):
+    """Every pair gets a place of its own, experts one after the other; the tiles cover the places,
+    none spans two experts or is longer than 256."""
+    from strata_inference_b200.kernels import native
+    g = torch.Generator().manual_seed(rows)
+    # (uneven: low-numbered experts are chosen far more often)
+    score = torch.rand((rows, experts), generator=g) ** (1.0 + torch.arange(experts) * 8.0 / experts)
+    ids = score.topk(top, dim=1).indices.to(torch.int32)
+    where, tiles = native.expert_plan(ids.cuda(), experts)
+    where, tiles = where.cpu(), tiles.cpu().tolist()
+    assert sorted(where.view(-1).tolist()) == list(range(rows * top))
+    by_place = torch.empty(rows * top, dtype=torch.int32)
+    by_place[where.view(-1).long()] = ids.view(-1)
+    assert (by_place[1:] >= by_place[:-1]).all()
+    at = 0
+    for k in range(tiles[0]):
+        row0, n, e = tiles[1 + 3 * k:4 + 3 * k]
+        assert row0 == at and 0 < n <= 256 and (by_place[row0:row0 + n] == e).all()
+        at += n
+    assert at == rows * top
+    x = torch.randn((rows, 20), generator=g).cuda()
+    xs = native.spread_rows(x, where.cuda(), torch.empty((rows * top, 20), device="cuda"))
+    assert torch.equal(xs[where.view(-1).long().cuda()].view(rows, top, 20), x[:, None].expand(rows, top, 20))
+
+
+@pytest.mark.parametrize("counts, N, K", [([256, 1, 0, 300], 128, 64), ([5, 700, 0, 0, 33, 257], 200, 136), ([130], 72, 512),
+                                          ([0, 40, 40, 40, 600, 12, 90], 384, 256)])
+def test_grouped_products(counts, N, K):
+    """Sorted rows times their groups' matrices: plain, and gate and up with the SiLU and the clipped
+    gate, widths that are and are not whole tiles, groups without a row."""
+    from strata_inference_b200.kernels import native
+    g = torch.Generator().manual_seed(N)
+    ids = torch.cat([torch.full((c,), e, dtype=torch.int32) for e, c in enumerate(counts)])
+    where, tiles = native.expert_plan(ids[:, None].cuda(), len(counts))
+    x = torch.randn((len(ids), K), generator=g).to(torch.bfloat16)
+    w = (torch.randn((len(counts), 2 * N, K), generator=g) / math.sqrt(K)).to(torch.bfloat16)
+    ref = torch.stack([w[int(e)].double() @ r for e, r in zip(ids, x.double())])
+    out = torch.full((len(ids), 2 * N), float("nan"), dtype=torch.bfloat16, device="cuda")
+    native.gemm_tcgen05_grouped(x.cuda(), w.cuda(), tiles, out)
+    assert (out.cpu().double() - ref).abs().max() <= 1e-2 * ref.abs().max()
+    for epi, cap in ((native.EPI_SWIGLU, 0.0), (native.EPI_CLIPPED, 1.2)):
+        a, u = ref[:, :N], ref[:, N:]
+        if cap:
+            a, u = a.clamp(max=cap), u.clamp(-cap, cap)
+            want = a * torch.sigmoid(1.702 * a) * (u + 1.0)
+        else:
+            want = a * torch.sigmoid(a) * u
+        out = torch.full((len(ids), N), float("nan"), dtype=torch.bfloat16, device="cuda")
+        native.gemm_tcgen05_grouped(x.cuda(), w.cuda(), tiles, out, epi, cap)
+        assert (out.cpu().double() - want).abs().max() <= 1e-2 * want.abs().max()
+    assert native.gemm_tcgen05_error() == 0
