@@ -588,10 +588,11 @@ def unread_expert_bytes(engine, rows):
 
 
 def spread_rows(engine):
-    """Norms of a randomly drawn model as the identity's neighbour: RMS gains of 1, Dynamic Tanh norms with weight 1, b 0 and alpha 1, and
-    routers' corrections of 0.  Drawn like other norm weights (around 0, spread 0.1) they turn every row into
-    nearly the same vector b, and a router then sends all rows of a step to the same experts:
-    the experts' work would be that of the worst imbalance there is."""
+    """Norms of a randomly drawn model as the identity's neighbour: RMS gains and heads' factors of 1,
+    Dynamic Tanh norms with weight 1, b 0 and alpha 1, and routers' corrections of 0.  Drawn like
+    other norm weights (around 0, spread 0.1) Dynamic Tanh turns every row into nearly the same
+    vector b, and corrections outweigh the scores: a router then sends all rows of a step to the
+    same experts, and the experts' work would be that of the worst imbalance there is."""
     norms = [engine.model.final_norm]
     for blk in engine.model.blocks:
         norms += [getattr(blk, site, None) for site in ("pre_mixer", "post_mixer", "pre_ff", "post_ff")]
