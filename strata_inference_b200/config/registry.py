@@ -95,6 +95,8 @@ def _register_builtin() -> None:
     register_architecture(("Besorax", "besorax"), BesoraxConfig.from_dict, besorax_spec, besorax_sizes)
     from .kerolorn import KerolornConfig, kerolorn_sizes, kerolorn_spec
     register_architecture(("Kerolorn", "kerolorn"), KerolornConfig.from_dict, kerolorn_spec, kerolorn_sizes)
+    from .simetar import SimetarConfig, simetar_sizes, simetar_spec
+    register_architecture(("Simetar", "simetar"), SimetarConfig.from_dict, simetar_spec, simetar_sizes)
 
 
 _register_builtin()

@@ -27,6 +27,8 @@ struct AttnPrefillArgs {
     int n_heads, n_kv;
     int window, keep;           // keep > 0 (with a window): the first `keep` positions stay visible
     float scale, softcap;
+    const float* sink;          // [n_heads] or null: e^{sink_h} joins each row's denominator
+    int close_cap;              // with a cap: tanh_close instead of tanh_fast
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -63,6 +65,8 @@ __device__ __forceinline__ float tanh_fast(float x) {
     asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
+// From one exponential and one division: 1 - 2 / (1 + e^2x), absolute error about 2^-21.
+__device__ __forceinline__ float tanh_close(float x) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x)); }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
@@ -201,7 +205,7 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 float v = s[j][i] * p.scale;
-                if (p.softcap > 0.f) v = p.softcap * tanh_fast(v * inv_cap);
+                if (p.softcap > 0.f) v = p.softcap * (p.close_cap ? tanh_close(v * inv_cap) : tanh_fast(v * inv_cap));
                 if (!inside) {
                     const int key = kt * 64 + 8 * j + 2 * t + (i & 1);
                     const int qp = (i < 2) ? qpos0 : qpos1;
@@ -277,6 +281,8 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(AttnPrefillArgs 
         const int pos = p0 + row % MP;
         if (pos >= n) continue;
         const int head = kvh * G + row / MP;
+        // (a sink: one more term of the denominator; every row sees itself, so its maximum is finite)
+        if (p.sink) l_run[r] += __expf(p.sink[head] - m_run[r]);
         const float inv = 1.0f / l_run[r];
         __nv_bfloat16* dst = p.out + (size_t)(row0 + pos) * p.n_heads * HD + (size_t)head * HD;
 #pragma unroll
@@ -315,7 +321,8 @@ static int launch_prefill(const AttnPrefillArgs& p, int n_seqs, int max_len, cud
 SIB_EXPORT int sib_attention_prefill(const void* qkv, int width, void* out, const int* seq_row0,
                                      const int* seq_len, int n_seqs, int max_len, int n_heads,
                                      int n_kv, int head_dim, float scale, float softcap,
-                                     int window, int keep, void* stream) {
+                                     int window, int keep, const float* sink, int close_cap,
+                                     void* stream) {
     if (n_seqs == 0 || max_len == 0) return 0;
     SIB_REQUIRE(sib_attention_prefill_supports(n_heads, n_kv, head_dim),
                 "attention_prefill: heads=%d kv_heads=%d head_dim=%d is not a shape this kernel "
@@ -328,7 +335,7 @@ SIB_EXPORT int sib_attention_prefill(const void* qkv, int width, void* out, cons
                     keep >= 0 && (keep == 0 || window > 0),
                 "attention_prefill: seqs=%d max_len=%d window=%d keep=%d", n_seqs, max_len, window, keep);
     AttnPrefillArgs p{(const __nv_bfloat16*)qkv, (__nv_bfloat16*)out, seq_row0, seq_len, width,
-                      n_heads, n_kv, window, keep, scale, softcap};
+                      n_heads, n_kv, window, keep, scale, softcap, sink, close_cap};
     cudaStream_t s = (cudaStream_t)stream;
     const int G = n_heads / n_kv;
 #define BY_G(HD)                                                              \

@@ -252,9 +252,18 @@ __device__ __forceinline__ float row_max(const uint32_t (&raw)[64], int j_lo, in
     return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
 
+// tanh from one 2^x and one reciprocal: 1 - 2 / (1 + e^2x), absolute error about 2^-22 (where
+// tanh_fast's is about 2^-11: with a cap of 20 that is a hundredth of a score).
+__device__ __forceinline__ float tanh_close(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(1.0f + exp2_fast(x * 2.8853900817779268f)));
+    return fmaf(-2.0f, y, 1.0f);
+}
+
 // 64 probabilities 2^(score - ref) as 32 packed bfloat16 pairs (in place of the raw
-// products); returns their sum.  CAP: score = c2 * tanh(product * c1), else product * c1.
-template <bool CAP, int MASK>
+// products); returns their sum.  CAP 1 (2: with the closer tanh): score = c2 * tanh(product * c1),
+// 0: product * c1.
+template <int CAP, int MASK>
 __device__ __forceinline__ float probabilities(uint32_t (&raw)[64], float c1, float c2, float ref,
                                                int j_lo, int j_hi, int j_keep = 0) {
     float sum[4] = {0.f, 0.f, 0.f, 0.f};
@@ -265,7 +274,8 @@ __device__ __forceinline__ float probabilities(uint32_t (&raw)[64], float c1, fl
         for (int h = 0; h < 2; ++h) {
             const int j = 2 * k + h;
             float x = __uint_as_float(raw[j]);
-            if (CAP) x = fmaf(c2, tanh_fast(x * c1), -ref);
+            if (CAP == 2) x = fmaf(c2, tanh_close(x * c1), -ref);
+            else if (CAP) x = fmaf(c2, tanh_fast(x * c1), -ref);
             else x = fmaf(x, c1, -ref);
             if (MASK) x = sees<MASK>(j, j_lo, j_hi, j_keep) ? x : -INFINITY;
             e[h] = exp2_fast(x);
@@ -294,6 +304,7 @@ struct TcArgs {
     // that another kernel has summed (scaled scores, natural exponentials), joined with this
     // kernel's own before the last division: pooled blocks before the window
     const float* extra;
+    int close_cap;           // with a cap: tanh_close instead of tanh_fast
 };
 
 // SPLIT.  When the grid is small against the device, a block (or pair) of query rows with
@@ -606,7 +617,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
             if (!swap_with_partner(t, mx_raw, other)) { if (lane == 0) *failed = 9; ok = false; break; }
             mx_raw = fmaxf(mx_raw, other);
             float mx = mx_raw * c1;
-            if (capped) mx = c2 * tanh_fast(mx);
+            if (capped) mx = c2 * (p.close_cap ? tanh_close(mx) : tanh_fast(mx));
             if (mx_raw == -INFINITY) mx = -INFINITY;
             // the reference the exponentials are taken against: raised only by big steps
             float factor = 1.f;
@@ -635,13 +646,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map, TcArgs p,
                 }
             }
             const float ref = m_ref == -INFINITY ? 0.f : m_ref;
-            if (capped) {
-                if (whole) l += probabilities<true, 0>(raw, c1, c2, ref, j_lo, j_hi);
-                else l += probabilities<true, 1>(raw, c1, c2, ref, j_lo, j_hi);
+            if (capped && p.close_cap) {
+                if (whole) l += probabilities<2, 0>(raw, c1, c2, ref, j_lo, j_hi);
+                else l += probabilities<2, 1>(raw, c1, c2, ref, j_lo, j_hi);
+            } else if (capped) {
+                if (whole) l += probabilities<1, 0>(raw, c1, c2, ref, j_lo, j_hi);
+                else l += probabilities<1, 1>(raw, c1, c2, ref, j_lo, j_hi);
             } else {
-                if (whole) l += probabilities<false, 0>(raw, c1, c2, ref, j_lo, j_hi);
-                else if (j_keep > 0) l += probabilities<false, 2>(raw, c1, c2, ref, j_lo, j_hi, j_keep);
-                else l += probabilities<false, 1>(raw, c1, c2, ref, j_lo, j_hi);
+                if (whole) l += probabilities<0, 0>(raw, c1, c2, ref, j_lo, j_hi);
+                else if (j_keep > 0) l += probabilities<0, 2>(raw, c1, c2, ref, j_lo, j_hi, j_keep);
+                else l += probabilities<0, 1>(raw, c1, c2, ref, j_lo, j_hi);
             }
             // P over the first 64 columns of the score tile (both threads have read theirs)
             tmem_st32(s_addr + 32 * half, reinterpret_cast<uint32_t(&)[32]>(raw));
@@ -1072,9 +1086,9 @@ SIB_EXPORT int sib_attention_prefill_tc(const void* qkv, int width, int total_ro
                                         float scale, float softcap, int window, void* scratch,
                                         long long scratch_bytes, int* tickets, int n_tickets,
                                         const int* host_lens, const int* seq_q0, const int* host_q0,
-                                        const float* sink, const float* extra, int keep, void* stream) {
+                                        const float* sink, const float* extra, int keep, int close_cap,
+                                        void* stream) {
     if (n_seqs == 0 || max_len == 0) return 0;
-    SIB_REQUIRE(sink == nullptr || softcap == 0.f, "attention_prefill_tc: a sink together with a cap is not built");
     SIB_REQUIRE(extra == nullptr || (softcap == 0.f && sink == nullptr && ((uintptr_t)extra % 4) == 0),
                 "attention_prefill_tc: another kernel's partial results go with no cap and no sink");
     SIB_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && softcap == 0.f)),
@@ -1136,7 +1150,7 @@ SIB_EXPORT int sib_attention_prefill_tc(const void* qkv, int width, int total_ro
     }
     if (items.n > 0) split_tiles = 0;
     TcArgs p{(__nv_bfloat16*)out, seq_row0, seq_len, seq_q0, error_flag, (float*)scratch, tickets,
-             split_tiles, n_heads, n_kv, window, keep, scale, softcap, sink, extra};
+             split_tiles, n_heads, n_kv, window, keep, scale, softcap, sink, extra, close_cap};
     cudaStream_t s = (cudaStream_t)stream;
 #define BY_G(HD, PAIR)                                                         \
     do {                                                                       \

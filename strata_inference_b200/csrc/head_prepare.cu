@@ -16,6 +16,7 @@
 //
 //   head_gate      y[r, h, :vd] = o[r, h, :vd] * sigmoid(gate[r, h])    (gate optional)
 //     which also drops the filled-up columns again.
+//   element_gate   the same with one gate per element of the concatenated heads.
 //
 // Plain counterpart: tests/plain_karupel.py attention_mixer().
 #include "common.cuh"
@@ -399,6 +400,72 @@ SIB_EXPORT int sib_head_gate(const void* o, const void* gate, long long gate_str
 }
 
 // ---------------------------------------------------------------------------
+// element_gate: y[r, h * vd + e] = o[r * row_stride + h * head_stride + e] * sigmoid(gate[r, h * vd + e]),
+// one gate per element of the concatenated heads.  The heads may lie `head_stride` apart and the
+// rows `row_stride` (wider heads are narrowed; [heads, rows, vd] results of a batched product are
+// put in row order on the way).  V: elements a thread takes (8: 16-byte accesses, bfloat16).
+// ---------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+element_gate_kernel(const T* o, long long row_stride, long long head_stride,
+                    const T* gate, long long gate_stride, T* y, int width, int vd,
+                    size_t total) {
+    pdl_trigger();
+    pdl_wait();
+    const int groups = width / V;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
+         idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t r = idx / groups;
+        const int c = (int)(idx - r * groups) * V;
+        const int h = c / vd;
+        const T* op = o + r * row_stride + (size_t)h * head_stride + (c - h * vd);
+        const T* gp = gate + r * gate_stride + c;
+        if constexpr (V == 1) {
+            y[r * width + c] = from_f32<T>(to_f32(*op) / (1.0f + expf(-to_f32(*gp))));
+        } else {
+            const uint4 a = *reinterpret_cast<const uint4*>(op), g = *reinterpret_cast<const uint4*>(gp);
+            const uint32_t aw[4] = {a.x, a.y, a.z, a.w}, gw[4] = {g.x, g.y, g.z, g.w};
+            uint32_t ow[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float lo = __uint_as_float(aw[i] << 16) / (1.0f + expf(-__uint_as_float(gw[i] << 16)));
+                const float hi = __uint_as_float(aw[i] & 0xffff0000u) /
+                                 (1.0f + expf(-__uint_as_float(gw[i] & 0xffff0000u)));
+                const __nv_bfloat162 pr = __floats2bfloat162_rn(lo, hi);
+                ow[i] = *reinterpret_cast<const uint32_t*>(&pr);
+            }
+            *reinterpret_cast<uint4*>(y + r * width + c) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
+        }
+    }
+}
+
+SIB_EXPORT int sib_element_gate(const void* o, long long row_stride, long long head_stride, const void* gate,
+                                long long gate_stride, void* y, int dtype, int rows, int n_heads, int vd,
+                                void* stream) {
+    if (rows == 0) return 0;
+    SIB_REQUIRE(rows > 0 && n_heads > 0 && vd > 0 && o && gate && y, "element_gate: rows=%d heads=%d width=%d", rows,
+                n_heads, vd);
+    const int width = n_heads * vd;
+    const bool wide = dtype == SIB_BF16 && vd % 8 == 0 && row_stride % 8 == 0 && head_stride % 8 == 0 &&
+                      gate_stride % 8 == 0 && ((uintptr_t)o % 16) == 0 && ((uintptr_t)gate % 16) == 0 &&
+                      ((uintptr_t)y % 16) == 0;
+    const size_t total = (size_t)rows * (wide ? width / 8 : width);
+    const size_t want = (total + 255) / 256;
+    const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+    cudaStream_t s = (cudaStream_t)stream;
+    if (wide) {
+        sib_launch_chained(element_gate_kernel<__nv_bfloat16, 8>, grid, dim3(256), 0, s, (const __nv_bfloat16*)o,
+                           row_stride, head_stride, (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)y, width,
+                           vd, total);
+    } else {
+        SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(element_gate_kernel<T, 1>, grid, dim3(256), 0, s, (const T*)o,
+                                                     row_stride, head_stride, (const T*)gate, gate_stride, (T*)y,
+                                                     width, vd, total));
+    }
+    return sib_check_launch("element_gate");
+}
+
+// ---------------------------------------------------------------------------
 // latent_prepare: what lies between the projections and the attention kernel of an
 // attention whose keys and values of all heads are made from ONE low-rank row per position
 // (the latent c, width `rank`) plus ONE rotated key part shared by the heads (width `rd`).
@@ -412,8 +479,9 @@ SIB_EXPORT int sib_head_gate(const void* o, const void* gate, long long gate_str
 //   key unit:   c = x / sqrt(mean(x^2) + eps) * w   over x = down[:rank];   the shared part
 //               down[rank : rank + rd] rotated;  the row goes to `k_rows` and to the cache
 //   query unit: [q_lat[h, r, :] | q_h's last rd columns rotated | 0]  ->  q_rows[r, h, :]
-// Rotation: the first `rot` (<= rd) columns in neighbouring pairs (2i, 2i + 1) by the angle
-// pos * inv_freq[i].
+// Rotation: the first `rot` (<= rd) columns in neighbouring pairs (2i, 2i + 1), or in half-split
+// ones (i, i + rot / 2), by the angle pos * inv_freq[i]; cosine and sine both times `magnitude`.
+// Without a key unit (`k_rows` null: a layer that reads another's rows) the query units alone.
 // Plain counterpart: tests/plain_vavupel.py latent_attention().
 // ---------------------------------------------------------------------------
 struct LatentPrepareArgs {
@@ -433,6 +501,8 @@ struct LatentPrepareArgs {
     int rows, n_heads, qd, rd, rank, pad, rot;
     int max_pages, page_tokens, ring_tokens;
     float eps;
+    int half_split;
+    float magnitude;
     // the down projection's rows (rank + rd) where they do not follow the query heads in `proj`
     // (queries that come from a product of their own); null: they do
     const void* down;
@@ -441,12 +511,16 @@ struct LatentPrepareArgs {
 
 template <typename T>
 __device__ __forceinline__ float rotated_pair(const T* part, int d, int rot, const float* inv_freq,
-                                              float pos) {
+                                              float pos, int half_split, float magnitude) {
     float x = to_f32(part[d]);
     if (d < rot) {
-        const float ang = pos * inv_freq[d >> 1];
-        const float c = cosf(ang), s = sinf(ang);
-        x = (d & 1) ? x * c + to_f32(part[d - 1]) * s : x * c - to_f32(part[d + 1]) * s;
+        const int half = rot / 2;
+        const int i = half_split ? (d < half ? d : d - half) : d >> 1;
+        const bool first = half_split ? d < half : !(d & 1);
+        const int other = half_split ? (d < half ? d + half : d - half) : d ^ 1;
+        const float ang = pos * inv_freq[i];
+        const float c = cosf(ang) * magnitude, s = sinf(ang) * magnitude;
+        x = first ? x * c - to_f32(part[other]) * s : x * c + to_f32(part[other]) * s;
     }
     return x;
 }
@@ -471,11 +545,12 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(LatentPrepareArgs p
         for (int d = lane; d < p.pad; d += 32) {
             T y = from_f32<T>(0.f);
             if (d < p.rank) y = lat[d];
-            else if (d < p.rank + p.rd) y = from_f32<T>(rotated_pair<T>(part, d - p.rank, rot, p.inv_freq, pos));
+            else if (d < p.rank + p.rd) y = from_f32<T>(rotated_pair<T>(part, d - p.rank, rot, p.inv_freq, pos, p.half_split, p.magnitude));
             out[d] = y;
         }
         return;
     }
+    if (p.k_rows == nullptr) return;         // (this layer reads another's rows)
     T* dst = nullptr;
     if (p.k_pool) {
         const int b = p.row_seq[r];
@@ -504,7 +579,8 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(LatentPrepareArgs p
     for (int d = lane; d < p.pad; d += 32) {
         float x = 0.f;
         if (d < p.rank) x = to_f32(down[d]) * inv * p.c_gain[d];
-        else if (d < p.rank + p.rd) x = rotated_pair<T>(down + p.rank, d - p.rank, rot, p.inv_freq, pos);
+        else if (d < p.rank + p.rd) x = rotated_pair<T>(down + p.rank, d - p.rank, rot, p.inv_freq, pos, p.half_split,
+                                                          p.magnitude);
         const T y = from_f32<T>(x);
         out[d] = y;
         if (dst) dst[d] = y;
@@ -516,14 +592,14 @@ SIB_EXPORT int sib_latent_prepare(
     const float* c_gain, float eps, const float* inv_freq, int rot, const int* row_pos,
     const int* row_seq, const int* seq_slot, const int* seq_end, void* k_pool, const int* page_table,
     int max_pages, int page_tokens, int ring_tokens, int rows, int n_heads, int qd, int rd, int rank,
-    int pad, const void* down, long long down_stride, void* stream) {
+    int pad, const void* down, long long down_stride, int half_split, float magnitude, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && n_heads > 0 && qd > 0 && rd >= 0 && rank > 0 && pad >= rank + rd,
                 "latent_prepare: rows=%d heads=%d widths %d + %d, rank %d in rows of %d", rows, n_heads,
                 qd, rd, rank, pad);
     SIB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= rd && (rot == 0 || inv_freq != nullptr),
                 "latent_prepare: %d rotated dimensions of %d", rot, rd);
-    SIB_REQUIRE(row_pos && c_gain && k_rows && (q_lat != nullptr) == (q_rows != nullptr),
+    SIB_REQUIRE(row_pos && (k_rows ? c_gain != nullptr : q_rows && !k_pool) && (q_lat != nullptr) == (q_rows != nullptr),
                 "latent_prepare: an argument is missing");
     SIB_REQUIRE(k_pool == nullptr || (page_table && row_seq && seq_slot && seq_end && page_tokens > 0 &&
                                       max_pages > 0),
@@ -531,7 +607,7 @@ SIB_EXPORT int sib_latent_prepare(
     SIB_REQUIRE((n_heads + 4) / 4 < 65536, "latent_prepare: too many heads (%d)", n_heads);
     LatentPrepareArgs p{proj, q_lat, q_rows, k_rows, c_gain, rot ? inv_freq : nullptr, row_pos, row_seq,
                         seq_slot, seq_end, k_pool, page_table, proj_stride, rows, n_heads, qd, rd, rank,
-                        pad, rot, max_pages, page_tokens, ring_tokens, eps, down, down_stride};
+                        pad, rot, max_pages, page_tokens, ring_tokens, eps, half_split, magnitude, down, down_stride};
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(latent_prepare_kernel<T>, dim3(rows, (n_heads + 4) / 4),
                                                  dim3(128), 0, (cudaStream_t)stream, p));
     return sib_check_launch("latent_prepare");
@@ -556,6 +632,8 @@ struct LatentExpandArgs {
     const int* row_pos;
     long long proj_stride;
     int rows, n_heads, qd, rd, vd, rank, pad, hw, rot;
+    int half_split;
+    float magnitude;
 };
 
 template <typename T>
@@ -576,7 +654,8 @@ __global__ void __launch_bounds__(128) latent_expand_kernel(LatentExpandArgs p) 
         for (int d = lane; d < p.hw; d += 32) {
             T y = zero;
             if (d < p.qd) y = head[d];
-            else if (d < p.qd + p.rd) y = from_f32<T>(rotated_pair<T>(head + p.qd, d - p.qd, rot, p.inv_freq, pos));
+            else if (d < p.qd + p.rd) y = from_f32<T>(rotated_pair<T>(head + p.qd, d - p.qd, rot, p.inv_freq, pos,
+                                                                               p.half_split, p.magnitude));
             out[d] = y;
         }
     } else if (kind == 1) {
@@ -594,7 +673,7 @@ SIB_EXPORT int sib_latent_expand(const void* proj, long long proj_stride, const 
                                  const void* k_heads, const void* v_heads, void* qkv, int dtype,
                                  const float* inv_freq, int rot, const int* row_pos, int rows,
                                  int n_heads, int qd, int rd, int vd, int rank, int pad, int hw,
-                                 void* stream) {
+                                 int half_split, float magnitude, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && n_heads > 0 && qd > 0 && rd >= 0 && vd > 0 && hw >= qd + rd && hw >= vd &&
                     pad >= rank + rd,
@@ -605,7 +684,7 @@ SIB_EXPORT int sib_latent_expand(const void* proj, long long proj_stride, const 
     SIB_REQUIRE(proj && k_rows && k_heads && v_heads && qkv && row_pos, "latent_expand: an argument is missing");
     SIB_REQUIRE((3 * n_heads + 3) / 4 < 65536, "latent_expand: too many heads (%d)", n_heads);
     LatentExpandArgs p{proj, k_rows, k_heads, v_heads, qkv, rot ? inv_freq : nullptr, row_pos, proj_stride,
-                       rows, n_heads, qd, rd, vd, rank, pad, hw, rot};
+                       rows, n_heads, qd, rd, vd, rank, pad, hw, rot, half_split, magnitude};
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(latent_expand_kernel<T>, dim3(rows, (3 * n_heads + 3) / 4),
                                                  dim3(128), 0, (cudaStream_t)stream, p));
     return sib_check_launch("latent_expand");

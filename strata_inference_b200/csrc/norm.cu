@@ -1,4 +1,5 @@
-// RMS norm, alone and fused with the residual add around it.
+// RMS norm, alone and fused with the residual add around it (further down: Dynamic Tanh and the
+// layer norm in the same two forms).
 //
 //   rms(x, g) = x * 1/sqrt(mean(x^2) + eps) * g        (statistics in f32)
 //
@@ -535,4 +536,225 @@ SIB_EXPORT int sib_pair_norm_mean(const void* a, const void* b, const float* wa,
                                                  (cudaStream_t)stream, (const T*)a, (const T*)b, wa,
                                                  wb, (T*)y, width, eps));
     return sib_check_launch("pair_norm_mean");
+}
+
+// ---------------------------------------------------------------------------
+// Layer norm with weight and bias, alone (with a row gather) and fused with the residual add
+// around it, as the RMS norm is:
+//     ln(x) = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b
+//     h[r, :] += post ? ln_post(a[r, :]) : a[r, :]
+//     out[r, :] = pre ? ln_pre(h[r, :]) : h[r, :]        (only if out)
+// Everything is 32-bit; the mean is taken first and the variance from the deviations (two sums
+// over the row, so that a large mean costs no digits).
+// (What the kernel ahead writes is not marked __restrict__: the compiler may move a load through
+// such a pointer ahead of the wait for that kernel.)
+// Plain counterpart: tests/plain_simetar.py layer_norm().
+// ---------------------------------------------------------------------------
+template <typename Tin, typename Tout>
+__global__ void layer_norm_kernel(const Tin* x, const int* __restrict__ rows,
+                                  const float* __restrict__ w, const float* __restrict__ b,
+                                  Tout* out, int hidden, float eps) {
+    extern __shared__ float row[];
+    __shared__ float scratch[33];
+    pdl_trigger();
+    pdl_wait();
+    const int i = blockIdx.x;
+    const Tin* src = x + (size_t)(rows ? rows[i] : i) * hidden;
+    float sum = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+        const float v = to_f32(src[c]);
+        row[c] = v;
+        sum += v;
+    }
+    const float mean = block_sum(sum, scratch) / (float)hidden;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+        const float d = row[c] - mean;
+        ss += d * d;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    Tout* dst = out + (size_t)i * hidden;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+        dst[c] = from_f32<Tout>((row[c] - mean) * inv * w[c] + b[c]);
+}
+
+struct LayerNormPair {
+    const float* post_w;       // null: what is added is not normed
+    const float* post_b;
+    const float* pre_w;        // null: the rows of h go out as they are
+    const float* pre_b;
+    float post_eps, pre_eps;
+};
+
+template <typename T>
+__global__ void add_layer_norm_kernel(const T* a, float* h, T* out,
+                                      int hidden, LayerNormPair p) {
+    extern __shared__ float row[];
+    __shared__ float scratch[33];
+    pdl_trigger();
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * hidden;
+    // (a thread only ever touches its own columns of `row`)
+    auto statistics = [&](float sum, float eps, float& mean, float& inv) {
+        mean = block_sum(sum, scratch) / (float)hidden;
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+            const float d = row[c] - mean;
+            ss += d * d;
+        }
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    };
+    float sum = 0.f, mean = 0.f, inv = 1.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+        const float v = to_f32(a[base + c]);
+        row[c] = v;
+        sum += v;
+    }
+    if (p.post_w) statistics(sum, p.post_eps, mean, inv);
+    sum = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+        const float v = h[base + c] + (p.post_w ? (row[c] - mean) * inv * p.post_w[c] + p.post_b[c] : row[c]);
+        h[base + c] = v;
+        row[c] = v;
+        sum += v;
+    }
+    if (!out) return;
+    if (p.pre_w) statistics(sum, p.pre_eps, mean, inv);
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+        out[base + c] = from_f32<T>(p.pre_w ? (row[c] - mean) * inv * p.pre_w[c] + p.pre_b[c] : row[c]);
+}
+
+// One block per row, one group of 8 columns per thread, the row in registers: every load is issued
+// before anything is computed, weights and biases before the kernel ahead has finished.
+__global__ void __launch_bounds__(1024)
+add_layer_norm_bf16_kernel(const __nv_bfloat16* a, float* h, __nv_bfloat16* out, int hidden, LayerNormPair p) {
+    __shared__ float scratch[33];
+    pdl_trigger();
+    const int c = 8 * threadIdx.x;
+    const bool live = c < hidden;
+    const float n = (float)hidden;
+    auto load8 = [&](const float* from, float (&o)[8]) {
+        const float4 lo = *reinterpret_cast<const float4*>(from), hi = *reinterpret_cast<const float4*>(from + 4);
+        o[0] = lo.x; o[1] = lo.y; o[2] = lo.z; o[3] = lo.w;
+        o[4] = hi.x; o[5] = hi.y; o[6] = hi.z; o[7] = hi.w;
+    };
+    float pw[8], pb[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) pw[e] = pb[e] = 0.f;
+    if (live && p.post_w) {
+        load8(p.post_w + c, pw);
+        load8(p.post_b + c, pb);
+    }
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * hidden + c;
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    float s[8], v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s[e] = 0.f;
+    if (live) {
+        raw = *reinterpret_cast<const uint4*>(a + base);
+        load8(h + base, s);
+    }
+    const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        v[2 * k] = __uint_as_float(w[k] << 16);
+        v[2 * k + 1] = __uint_as_float(w[k] & 0xffff0000u);
+    }
+    auto statistics = [&](const float (&x)[8], float eps, float& mean, float& inv) {
+        float sum = 0.f, ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += x[e];           // (columns that do not exist hold zeros)
+        mean = block_sum(sum, scratch) / n;
+        if (live) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss += (x[e] - mean) * (x[e] - mean);
+        }
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / n + eps);
+    };
+    float mean = 0.f, inv = 1.f;
+    if (p.post_w) {
+        statistics(v, p.post_eps, mean, inv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = live ? (v[e] - mean) * inv * pw[e] + pb[e] : 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s[e] += v[e];
+    if (live) {
+        *reinterpret_cast<float4*>(h + base) = make_float4(s[0], s[1], s[2], s[3]);
+        *reinterpret_cast<float4*>(h + base + 4) = make_float4(s[4], s[5], s[6], s[7]);
+    }
+    if (!out) return;
+    if (p.pre_w) {
+        statistics(s, p.pre_eps, mean, inv);
+        if (live) {
+            load8(p.pre_w + c, pw);
+            load8(p.pre_b + c, pb);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s[e] = (s[e] - mean) * inv * pw[e] + pb[e];
+    }
+    if (live) {
+        uint32_t o[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const __nv_bfloat162 pr = __floats2bfloat162_rn(s[2 * k], s[2 * k + 1]);
+            o[k] = *reinterpret_cast<const uint32_t*>(&pr);
+        }
+        *reinterpret_cast<uint4*>(out + base) = make_uint4(o[0], o[1], o[2], o[3]);
+    }
+}
+
+SIB_EXPORT int sib_layer_norm(const void* x, int in_dtype, const int* rows, const float* w, const float* b,
+                              float eps, void* out, int out_dtype, int n_rows, int hidden, void* stream) {
+    if (n_rows == 0) return 0;
+    SIB_REQUIRE(n_rows > 0 && hidden > 0 && w && b, "layer_norm: rows=%d hidden=%d", n_rows, hidden);
+    const size_t smem = (size_t)hidden * sizeof(float);
+    SIB_REQUIRE(smem <= (size_t)kMaxRowBytes, "layer_norm: hidden=%d needs %zu bytes of shared memory; at most "
+                "%d are supported", hidden, smem, kMaxRowBytes);
+    const int threads = norm_threads(hidden);
+    cudaStream_t s = (cudaStream_t)stream;
+#define LAUNCH(TIN, TOUT)                                                                        \
+    do {                                                                                         \
+        int rc = allow_row(layer_norm_kernel<TIN, TOUT>, smem);                                  \
+        if (rc) return rc;                                                                       \
+        sib_launch_chained(layer_norm_kernel<TIN, TOUT>, dim3(n_rows), dim3(threads), smem, s,   \
+                           (const TIN*)x, rows, w, b, (TOUT*)out, hidden, eps);                  \
+    } while (0)
+    if (in_dtype == SIB_F32 && out_dtype == SIB_F32) LAUNCH(float, float);
+    else if (in_dtype == SIB_F32 && out_dtype == SIB_BF16) LAUNCH(float, __nv_bfloat16);
+    else if (in_dtype == SIB_BF16 && out_dtype == SIB_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
+    else if (in_dtype == SIB_BF16 && out_dtype == SIB_F32) LAUNCH(__nv_bfloat16, float);
+    else SIB_REQUIRE(false, "layer_norm: unknown element types %d -> %d", in_dtype, out_dtype);
+#undef LAUNCH
+    return sib_check_launch("layer_norm");
+}
+
+SIB_EXPORT int sib_add_layer_norm(const void* a, int dtype, const float* post_w, const float* post_b,
+                                  float post_eps, float* h, const float* pre_w, const float* pre_b,
+                                  float pre_eps, void* out, int n_rows, int hidden, void* stream) {
+    if (n_rows == 0) return 0;
+    SIB_REQUIRE(n_rows > 0 && hidden > 0, "add_layer_norm: rows=%d hidden=%d", n_rows, hidden);
+    SIB_REQUIRE((post_w != nullptr) == (post_b != nullptr) && (pre_w != nullptr) == (pre_b != nullptr) &&
+                    (pre_w == nullptr || out != nullptr),
+                "add_layer_norm: a norm needs its weight and its bias (and the next one out)");
+    const LayerNormPair p{post_w, post_b, pre_w, pre_b, post_eps, pre_eps};
+    cudaStream_t s = (cudaStream_t)stream;
+    auto wide = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
+    if (dtype == SIB_BF16 && hidden % 8 == 0 && hidden / 8 <= 1024 && wide(a) && wide(h) && wide(out) &&
+        wide(post_w) && wide(post_b) && wide(pre_w) && wide(pre_b)) {
+        sib_launch_chained(add_layer_norm_bf16_kernel, dim3(n_rows), dim3((hidden / 8 + 31) / 32 * 32), 0, s,
+                           (const __nv_bfloat16*)a, h, (__nv_bfloat16*)out, hidden, p);
+        return sib_check_launch("add_layer_norm");
+    }
+    const size_t smem = (size_t)hidden * sizeof(float);
+    SIB_REQUIRE(smem <= (size_t)kMaxRowBytes, "add_layer_norm: hidden=%d needs %zu bytes of shared memory; at "
+                "most %d are supported", hidden, smem, kMaxRowBytes);
+    SIB_DISPATCH_DTYPE(dtype, {
+        int rc = allow_row(add_layer_norm_kernel<T>, smem);
+        if (rc) return rc;
+        sib_launch_chained(add_layer_norm_kernel<T>, dim3(n_rows), dim3(norm_threads(hidden)), smem, s, (const T*)a,
+                           h, (T*)out, hidden, p);
+    });
+    return sib_check_launch("add_layer_norm");
 }

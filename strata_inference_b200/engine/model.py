@@ -169,11 +169,13 @@ class DecoderModel:
         """Whether every part promises that a recorded step of prompts may be replayed for
         other prompts (see StepContext): else prompt steps are launched one by one."""
         # (a run that reads another run's cache reads it by slot, for every row: the rows that
-        # fill a recorded step up have none)
+        # fill a recorded step up have none; a mixer that promises ``captures_borrowed`` takes
+        # the lender's packed rows in a step of prompts instead)
         return (getattr(self.embedding, "captures_prompts", False)
                 and (self.pass_mix is None or getattr(self.pass_mix, "captures_prompts", False))
                 and all(getattr(b, "captures_prompts", False) for b in self.blocks)
-                and all(e.cache_of is None for e in self.spec.schedule))
+                and all(e.cache_of is None or getattr(self.blocks[e.layer].mixer, "captures_borrowed", False)
+                        for e in self.spec.schedule))
 
     def hidden_states(self, ctx) -> torch.Tensor:
         """Run every schedule entry over the step's rows; returns the 32-bit

@@ -445,6 +445,54 @@ def add_dyt_norm(a: torch.Tensor, post, h: torch.Tensor, pre, out: Optional[torc
                                       c_int(hidden), c_float(scale), _stream()))
 
 
+@_timed(lambda x, w, b, eps, out, rows=None: (
+    "layer_norm", out.shape[0] * x.shape[1] * x.element_size() + _nbytes(out), 0))
+def layer_norm(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, out: torch.Tensor,
+               rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[i] = (x - mean) / sqrt(var + eps) * w + b over x[rows[i] if rows else i]; 32-bit."""
+    _want(x, x.dtype, "x")
+    _want(out, out.dtype, "out")
+    n, hidden = out.shape
+    _f32(w, hidden, "w")
+    _f32(b, hidden, "b")
+    if x.shape[1] != hidden:
+        raise KernelError("layer_norm: shapes do not fit")
+    if rows is not None:
+        _want(rows, torch.int32, "rows")
+        if rows.numel() != n:
+            raise KernelError("layer_norm: one row index per output row")
+    elif x.shape[0] != n:
+        raise KernelError("layer_norm: x and out differ in rows")
+    _check(library().sib_layer_norm(_ptr(x), _code(x.dtype), _ptr(rows), _ptr(w), _ptr(b), c_float(eps), _ptr(out),
+                                    _code(out.dtype), c_int(n), c_int(hidden), _stream()))
+    return out
+
+
+@_timed(lambda a, post, h, pre, out: ("add_layer_norm", _nbytes(a, out) + 2 * _nbytes(h), 0))
+def add_layer_norm(a: torch.Tensor, post, h: torch.Tensor, pre, out: Optional[torch.Tensor]) -> None:
+    """h += ln_post(a) (or a when ``post`` is None); out = ln_pre(h) (or h as activations when ``pre``
+    is None and out is given).  ``post`` and ``pre``: (weight, bias, eps) of a layer norm."""
+    _want(h, torch.float32, "h")
+    _want(a, a.dtype, "a")
+    rows, hidden = h.shape
+    if tuple(a.shape) != (rows, hidden):
+        raise KernelError("add_layer_norm: a and h differ in shape")
+    for triple, nm in ((post, "post"), (pre, "pre")):
+        if triple is not None:
+            _f32(triple[0], hidden, nm + " weight")
+            _f32(triple[1], hidden, nm + " bias")
+    if out is not None:
+        _want(out, a.dtype, "out")
+        if tuple(out.shape) != (rows, hidden):
+            raise KernelError("add_layer_norm: out and h differ in shape")
+    elif pre is not None:
+        raise KernelError("add_layer_norm: the next norm needs out")
+    pw, pb, pe = post if post is not None else (None, None, 0.0)
+    qw, qb, qe = pre if pre is not None else (None, None, 0.0)
+    _check(library().sib_add_layer_norm(_ptr(a), _code(a.dtype), _ptr(pw), _ptr(pb), c_float(pe), _ptr(h), _ptr(qw),
+                                        _ptr(qb), c_float(qe), _ptr(out), c_int(rows), c_int(hidden), _stream()))
+
+
 @_timed(lambda ctx, table, bigram, last_token, out, *a: ("bigram_embed", 3 * _nbytes(out), 0))
 def bigram_embed(ctx, table: torch.Tensor, bigram: torch.Tensor, last_token: torch.Tensor,
                  out: torch.Tensor, scale: float, buckets: int, mul_prev: int, mul_cur: int) -> torch.Tensor:
@@ -821,6 +869,70 @@ def head_prepare(proj: torch.Tensor, qkv: torch.Tensor, bias: Optional[torch.Ten
     return qkv
 
 
+@_timed(lambda proj, qkv, *a, n_heads, n_kv, key_dim, value_dim, values_from_keys, k_pool=None, **kw: (
+    "row_prepare", proj.shape[0] * (n_heads * key_dim + n_kv * (key_dim + (0 if values_from_keys else value_dim)))
+    * proj.element_size() + _nbytes(qkv)
+    + (2 * qkv.shape[0] * n_kv * (qkv.shape[1] // (n_heads + 2 * n_kv)) * qkv.element_size() if k_pool is not None
+       else 0), 0))
+def row_prepare(proj: torch.Tensor, qkv: torch.Tensor, ctx, *, n_heads: int, n_kv: int, key_dim: int,
+                value_dim: int, values_from_keys: bool, bias: Optional[torch.Tensor] = None,
+                conv: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
+                q_gain: Optional[torch.Tensor] = None, k_gain: Optional[torch.Tensor] = None, eps: float = 0.0,
+                inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, style: int = ROPE_HALF_SPLIT,
+                magnitude: float = 1.0, k_pool: Optional[torch.Tensor] = None,
+                v_pool: Optional[torch.Tensor] = None, page_table: Optional[torch.Tensor] = None,
+                page_tokens: int = 0, ring_tokens: int = 0, fixed_tokens: int = 0) -> torch.Tensor:
+    """From a projected row ``[q heads | k heads | (v heads) | ...]`` to the packed q|k|v rows the
+    attention kernels read (csrc/row_prepare.cu): bias, a causal convolution over time per channel
+    of q and k (``conv`` 32-bit ``[taps, channels]``; ``state`` 32-bit ``[slots, (taps - 1) *
+    channels]`` is brought to the step's end), values that are the keys at that point
+    (``values_from_keys``) or columns of their own, RMS norm of all of a row's q and of all of
+    its k at once with gains, partial rotation, and k and v written into the paged cache."""
+    rows = proj.shape[0]
+    nq, nk = n_heads * key_dim, n_kv * key_dim
+    nv = 0 if values_from_keys else n_kv * value_dim
+    _want(proj, qkv.dtype, "proj", contiguous=False)
+    _want(qkv, qkv.dtype, "qkv")
+    if proj.stride(1) != 1 or proj.shape[1] < nq + nk + nv or rows != ctx.n_rows:
+        raise KernelError("row_prepare: the step's projected rows must hold q, k (and v) side by side")
+    pad = qkv.shape[1] // (n_heads + 2 * n_kv)
+    if tuple(qkv.shape) != (rows, (n_heads + 2 * n_kv) * pad):
+        raise KernelError("row_prepare: the packed rows do not fit the head counts")
+    for t, n, nm in ((bias, nq + nk + nv, "bias"), (q_gain, nq, "q_gain"), (k_gain, nk, "k_gain"),
+                     (inv_freq, rotary_dim // 2, "inv_freq")):
+        if t is not None:
+            _f32(t, n, nm)
+    taps = 0
+    if conv is not None:
+        taps = conv.shape[0]
+        _f32(conv, taps * (nq + nk), "conv")
+        if taps > 1:
+            _want(state, torch.float32, "state")
+            if state.dim() != 2 or state.shape[1] < (taps - 1) * (nq + nk):
+                raise KernelError("row_prepare: the state holds [slots, (taps - 1) * channels]")
+    max_pages = 0
+    if k_pool is not None:
+        want = (n_kv, page_tokens, pad)
+        for t in (k_pool, v_pool):
+            _want(t, qkv.dtype, "cache")
+            if tuple(t.shape[1:]) != want:
+                raise KernelError("row_prepare: pool layout must be [pages, kv_heads, page_tokens, width]")
+        _want(page_table, torch.int32, "page_table")
+        max_pages = page_table.shape[1]
+    # (in a recorded step of prompts a sequence's rows change between replays)
+    single = ctx.max_count == 1 and rows == ctx.n_seqs
+    _check(library().sib_row_prepare(
+        _ptr(proj), c_longlong(proj.stride(0)), _ptr(qkv), _code(qkv.dtype), _ptr(bias), _ptr(conv), c_int(taps),
+        _ptr(state if taps > 1 else None), c_longlong(state.stride(0) if taps > 1 else 0), _ptr(q_gain), _ptr(k_gain),
+        c_float(eps), _ptr(inv_freq), c_int(rotary_dim if inv_freq is not None else 0),
+        c_int(1 if style == ROPE_INTERLEAVED else 0), c_float(magnitude), _ptr(ctx.row_pos), _ptr(ctx.row_seq),
+        _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_end), _ptr(ctx.seq_row0), _ptr(k_pool), _ptr(v_pool),
+        _ptr(page_table), c_int(max_pages), c_int(page_tokens), c_int(ring_tokens), c_int(fixed_tokens), c_int(rows),
+        c_int(ctx.n_seqs), c_int(n_heads), c_int(n_kv), c_int(key_dim), c_int(value_dim), c_int(pad),
+        c_int(1 if values_from_keys else 0), c_int(1 if single else 0), _stream()))
+    return qkv
+
+
 @_timed(lambda qkv, view, *a, **kw: ("pool_store", 2 * _nbytes(qkv) // 3, 0))
 def pool_store(qkv: torch.Tensor, view, ctx, n_heads: int, n_kv: int, pad: int) -> None:
     """For every block of ``view.need.pool`` positions whose last position this step brings:
@@ -926,19 +1038,42 @@ def head_gate(o: torch.Tensor, gate: Optional[torch.Tensor], y: torch.Tensor, n_
     return y
 
 
+@_timed(lambda o, gate, y, *a: ("element_gate", 3 * _nbytes(y), 0))
+def element_gate(o: torch.Tensor, gate: torch.Tensor, y: torch.Tensor, n_heads: int, value_dim: int) -> torch.Tensor:
+    """y[r, h, :] = o[r, h, :value_dim] * sigmoid(gate[r, h, :]), one gate per element.  ``o``: a view
+    ``[rows, n_heads, at least value_dim]`` of any row and head stride, ``gate`` a view ``[rows,
+    n_heads * value_dim]``."""
+    rows = y.shape[0]
+    _want(o, y.dtype, "o", contiguous=False)
+    _want(gate, y.dtype, "gate", contiguous=False)
+    _want(y, y.dtype, "y")
+    width = n_heads * value_dim
+    if tuple(y.shape) != (rows, width) or tuple(gate.shape) != (rows, width) or o.dim() != 3 \
+            or tuple(o.shape[:2]) != (rows, n_heads) or o.shape[2] < value_dim:
+        raise KernelError("element_gate: shapes do not fit the head counts")
+    if o.stride(2) != 1 or gate.stride(1) != 1:
+        raise KernelError("element_gate: a head's elements must be neighbours")
+    _check(library().sib_element_gate(_ptr(o), c_longlong(o.stride(0)), c_longlong(o.stride(1)), _ptr(gate),
+                                      c_longlong(gate.stride(0)), _ptr(y), _code(y.dtype), c_int(rows),
+                                      c_int(n_heads), c_int(value_dim), _stream()))
+    return y
+
+
 @_timed(lambda proj, q_lat, q_rows, k_rows, *a, **kw: ("latent_prepare", _nbytes(q_lat, q_rows, k_rows) * 2, 0))
-def latent_prepare(proj: torch.Tensor, q_lat: torch.Tensor, q_rows: torch.Tensor, k_rows: torch.Tensor,
-                   c_gain: torch.Tensor, eps: float, inv_freq: Optional[torch.Tensor], rot: int, ctx,
+def latent_prepare(proj: torch.Tensor, q_lat: Optional[torch.Tensor], q_rows: Optional[torch.Tensor],
+                   k_rows: Optional[torch.Tensor], c_gain: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rot: int, ctx,
                    k_pool: Optional[torch.Tensor], page_table: Optional[torch.Tensor],
                    page_tokens: int, ring_tokens: int, n_heads: int, q_dim: int, rot_dim: int,
-                   rank: int, pad: int, down: Optional[torch.Tensor] = None) -> None:
+                   rank: int, pad: int, down: Optional[torch.Tensor] = None, style: int = ROPE_INTERLEAVED,
+                   magnitude: float = 1.0) -> None:
     """Between the projections and the attention over a shared latent (csrc/head_prepare.cu):
     ``proj`` rows hold the query heads (``q_dim`` + ``rot_dim`` each) and then the down
     projection (``rank`` + ``rot_dim``), unless ``down`` (a view ``[rows, rank + rot_dim]``) gives
     the latter where the queries come from a product of their own; ``q_lat`` ``[heads, rows, rank]`` are the queries
     already multiplied into the latent's space.  Writes ``q_rows`` ``[rows, heads * pad]``
     (not with ``q_lat`` and ``q_rows`` None), ``k_rows`` ``[rows, pad]`` and the cache cells of
-    the rows."""
+    the rows (not with ``k_rows`` None: a layer that reads another's rows).  ``style`` and
+    ``magnitude``: the rotation's pairs and the factor on its cosines and sines."""
     rows = proj.shape[0]
     _want(proj, proj.dtype, "proj", contiguous=False)
     if (q_lat is None) != (q_rows is None):
@@ -950,13 +1085,17 @@ def latent_prepare(proj: torch.Tensor, q_lat: torch.Tensor, q_rows: torch.Tensor
         _want(t, proj.dtype, nm)
         if tuple(t.shape) != shape:
             raise KernelError(f"latent_prepare: {nm} must be {shape}")
-    if proj.stride(1) != 1 or proj.shape[1] < n_heads * (q_dim + rot_dim) + (0 if down is not None else rank + rot_dim):
+    own = down is None and k_rows is not None        # the down projection follows the query heads
+    if proj.stride(1) != 1 or proj.shape[1] < n_heads * (q_dim + rot_dim) + (rank + rot_dim if own else 0):
         raise KernelError("latent_prepare: a projected row must hold the query heads and the down projection")
     if down is not None:
         _want(down, proj.dtype, "down", contiguous=False)
         if down.stride(1) != 1 or down.shape[0] != rows or down.shape[1] < rank + rot_dim:
             raise KernelError("latent_prepare: down must be [rows, rank + rot_dim]")
-    _f32(c_gain, rank, "c_gain")
+    if k_rows is not None:
+        _f32(c_gain, rank, "c_gain")
+    elif k_pool is not None:
+        raise KernelError("latent_prepare: nothing to store without key rows")
     if rot:
         _f32(inv_freq, rot // 2, "inv_freq")
     max_pages = 0
@@ -971,13 +1110,15 @@ def latent_prepare(proj: torch.Tensor, q_lat: torch.Tensor, q_rows: torch.Tensor
         _ptr(ctx.row_pos), _ptr(ctx.row_seq), _ptr(ctx.seq_slot), _ptr(ctx.seq_end), _ptr(k_pool),
         _ptr(page_table), c_int(max_pages), c_int(page_tokens), c_int(ring_tokens), c_int(rows),
         c_int(n_heads), c_int(q_dim), c_int(rot_dim), c_int(rank), c_int(pad), _ptr(down),
-        c_longlong(down.stride(0) if down is not None else 0), _stream()))
+        c_longlong(down.stride(0) if down is not None else 0), c_int(1 if style == ROPE_HALF_SPLIT else 0),
+        c_float(magnitude), _stream()))
 
 
 @_timed(lambda proj, k_rows, k_heads, v_heads, qkv, *a, **kw: ("latent_expand", _nbytes(k_heads, v_heads, qkv) * 1.3, 0))
 def latent_expand(proj: torch.Tensor, k_rows: torch.Tensor, k_heads: torch.Tensor, v_heads: torch.Tensor,
                   qkv: torch.Tensor, inv_freq: Optional[torch.Tensor], rot: int, row_pos, n_heads: int,
-                  q_dim: int, rot_dim: int, value_dim: int, rank: int, pad: int, head_width: int) -> torch.Tensor:
+                  q_dim: int, rot_dim: int, value_dim: int, rank: int, pad: int, head_width: int,
+                  style: int = ROPE_INTERLEAVED, magnitude: float = 1.0) -> torch.Tensor:
     """Packed rows for the prompt attention kernels from keys and values made per head
     (csrc/head_prepare.cu): ``qkv[r]`` = query heads ``[unrotated | rotated | 0]``, key heads
     ``[k_heads | the row's shared rotated part (from k_rows) | 0]``, value heads ``[v_heads | 0]``,
@@ -998,7 +1139,7 @@ def latent_expand(proj: torch.Tensor, k_rows: torch.Tensor, k_heads: torch.Tenso
         _ptr(proj), c_longlong(proj.stride(0)), _ptr(k_rows), _ptr(k_heads), _ptr(v_heads), _ptr(qkv),
         _code(proj.dtype), _ptr(inv_freq if rot else None), c_int(rot), _ptr(row_pos), c_int(rows),
         c_int(n_heads), c_int(q_dim), c_int(rot_dim), c_int(value_dim), c_int(rank), c_int(pad),
-        c_int(head_width), _stream()))
+        c_int(head_width), c_int(1 if style == ROPE_HALF_SPLIT else 0), c_float(magnitude), _stream()))
     return qkv
 
 
@@ -1496,14 +1637,18 @@ def attention_prefill_supports(n_heads: int, n_kv: int, head_dim: int) -> bool:
 
 
 @_timed(lambda qkv, out, seq_row0, seq_len, n_seqs, max_len, n_heads, n_kv, head_dim, scale,
-        softcap, window, keep=0: _prompt_work("attention_prefill (mma.sync)", qkv, seq_len, n_heads,
-                                              head_dim, window, keep))
+        softcap, window, keep=0, sink=None, close_cap=False: _prompt_work(
+            "attention_prefill (mma.sync)", qkv, seq_len, n_heads, head_dim, window, keep))
 def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n_seqs: int,
                       max_len: int, n_heads: int, n_kv: int, head_dim: int, scale: float,
-                      softcap: float, window: int, keep: int = 0) -> torch.Tensor:
+                      softcap: float, window: int, keep: int = 0, sink: Optional[torch.Tensor] = None,
+                      close_cap: bool = False) -> torch.Tensor:
     """Attention of packed bfloat16 prompts that start at position 0 over their
     own (rotated) keys and values (see csrc/attention_prefill.cu).  ``keep`` > 0 (with a window):
-    the first ``keep`` positions stay visible."""
+    the first ``keep`` positions stay visible.  ``sink``: one 32-bit value per head whose exponential
+    joins the denominator; ``close_cap``: the cap's tanh to 32-bit precision instead of 2^-11."""
+    if sink is not None:
+        _f32(sink, n_heads, "sink")
     _want(qkv, torch.bfloat16, "qkv")
     _want(out, torch.bfloat16, "out")
     if out.shape[0] != qkv.shape[0] or out.shape[1] != n_heads * head_dim:
@@ -1511,7 +1656,7 @@ def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n
     _check(library().sib_attention_prefill(
         _ptr(qkv), c_int(qkv.shape[1]), _ptr(out), _ptr(seq_row0), _ptr(seq_len), c_int(n_seqs),
         c_int(max_len), c_int(n_heads), c_int(n_kv), c_int(head_dim), c_float(scale),
-        c_float(softcap), c_int(window), c_int(keep), _stream()))
+        c_float(softcap), c_int(window), c_int(keep), _ptr(sink), c_int(1 if close_cap else 0), _stream()))
     return out
 
 
@@ -1550,7 +1695,7 @@ def attention_prefill_tc_plan(lens: Sequence[int], n_heads: int, n_kv: int, head
 
 @_timed(lambda qkv, out, seq_row0, seq_len, n_seqs, max_len, n_heads, n_kv, head_dim, scale,
         softcap, window, scratch=None, tickets=None, host_lens=None, seq_q0=None,
-        host_q0=None, sink=None, extra=None, keep=0: _prompt_work(
+        host_q0=None, sink=None, extra=None, keep=0, close_cap=False: _prompt_work(
             "attention_prefill_tc (tcgen05)", qkv, seq_len, n_heads, head_dim, window, keep))
 def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len, n_seqs: int,
                          max_len: int, n_heads: int, n_kv: int, head_dim: int, scale: float,
@@ -1560,10 +1705,12 @@ def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len
                          seq_q0: Optional[torch.Tensor] = None,
                          host_q0: Optional[Sequence[int]] = None,
                          sink: Optional[torch.Tensor] = None,
-                         extra: Optional[torch.Tensor] = None, keep: int = 0) -> torch.Tensor:
+                         extra: Optional[torch.Tensor] = None, keep: int = 0,
+                         close_cap: bool = False) -> torch.Tensor:
     """The prompt attention on tcgen05 (see csrc/attention_prefill_tc.cu).  ``keep`` > 0 (with a
     window, no cap): the first ``keep`` positions stay visible.  ``sink``: one 32-bit
-    value per head whose exponential joins every row's denominator (no cap then).  ``extra``:
+    value per head whose exponential joins every row's denominator.  ``close_cap``: the cap's tanh
+    to 32-bit precision instead of 2^-11.  ``extra``:
     32-bit ``[rows, heads, head_dim + 2]``, per row and head the (max, sum, accumulator) of keys
     that another kernel has summed (``attention_rows`` with ``cells_only``), joined with this
     kernel's own sums before the last division (no cap, no sink then).  With ``scratch``
@@ -1594,7 +1741,7 @@ def attention_prefill_tc(qkv: torch.Tensor, out: torch.Tensor, seq_row0, seq_len
         None if host_lens is None else (c_int * len(host_lens))(*[int(n) for n in host_lens]),
         _ptr(seq_q0),
         None if host_q0 is None else (c_int * len(host_q0))(*[int(n) for n in host_q0]),
-        _ptr(sink), _ptr(extra), c_int(keep), _stream()))
+        _ptr(sink), _ptr(extra), c_int(keep), c_int(1 if close_cap else 0), _stream()))
     return out
 
 

@@ -68,7 +68,24 @@ the projection and the attention kernel, in 32-bit):
                 layer leaves its packed rows for that run, which then attends over them with
                 the prompt kernel instead of row by row over the cache.
 
-A chunked mask or a sink takes these kernels: bfloat16 prompts the tcgen05 prompt kernel, to
+``sink_score``  a number: a sink of that score for every head, with no stored tensor (0 adds one to
+                the softmax's denominator).
+``exact_cap``   True: the soft cap's tanh is taken to 32-bit precision in the prompt kernels too
+                (they otherwise use the hardware's tanh, good to 2^-11).
+``output_gate`` True: the concatenated heads are multiplied element by element by sigmoid(gate_proj
+                x), x the mixer's input, before the output product (csrc/head_prepare.cu element_gate).
+``qk_conv``     taps n > 0: a causal convolution over time on each channel of the projected q and k
+                (``q_conv.weight``, ``k_conv.weight``, [channels, n], no bias), ahead of norm and
+                rotation; the last n - 1 projected rows of a sequence are state of the mixer's own.
+``values_from_keys``  True: a head's values are its keys behind the convolution, ahead of norm and
+                rotation; there is no value projection (``value_dim`` = ``head_dim``).
+``qk_norm``     with ``whole`` True: all of a row's q (and all of its k) share one root mean square,
+                with a weight per channel, before the rotation.
+
+``qk_conv``, ``values_from_keys`` and a whole ``qk_norm`` work on whole projected rows ahead of the heads
+(csrc/row_prepare.cu: one launch from the product's output to packed rows and cache).
+
+A chunked mask, or a sink in a layer that lends or borrows its keys, takes these kernels: bfloat16 prompts the tcgen05 prompt kernel, to
 which every chunk of a prompt is a sequence of its own (rows of one chunk see nothing of
 another, so a chunk's rows are a causal prompt; the rotation has been applied by position
 before) and which takes the sink in its last division; rows over the cache the decode
@@ -88,7 +105,7 @@ from typing import Dict, Mapping, Optional
 
 import torch
 
-from ..cache.paged import CacheNeed, KVNeed
+from ..cache.paged import CacheNeed, KVNeed, StateNeed
 from ..config.spec import ConfigError, PartSpec
 from ..kernels import native
 from ..weights.arena import Piece, Resident, resident_of
@@ -154,14 +171,27 @@ class Attention:
         """Whether the heads are worked on between the projection and the attention."""
         return bool(params.get("bias") or params.get("qk_norm") or params.get("value_mix")
                     or params.get("head_gate") or params.get("pool") or params.get("head_temp")
-                    or params.get("keep_first") or params["position"].get("yarn")
+                    or params.get("keep_first") or params["position"].get("yarn") or params.get("output_gate")
+                    or Attention._row_work(params)
                     or int(params.get("value_dim") or params["head_dim"]) != params["head_dim"]
                     or int(params["head_dim"]) % 16 != 0)      # (padded to the next 16)
+
+    @staticmethod
+    def _row_work(params: Mapping) -> bool:
+        """Whether whole projected rows are worked on ahead of the heads (csrc/row_prepare.cu)."""
+        return bool(params.get("qk_conv") or params.get("values_from_keys")
+                    or (params.get("qk_norm") or {}).get("whole"))
 
     @staticmethod
     def tensors(params: Mapping, hidden: int) -> Dict[str, TensorDecl]:
         nh, nkv, hd = params["num_heads"], params["num_kv_heads"], params["head_dim"]
         vd = int(params.get("value_dim") or hd)
+        if Attention._row_work(params) and any(params.get(k) for k in (
+                "value_mix", "head_gate", "pool", "head_temp", "chunk", "borrows_cache", "lends_cache")):
+            raise ConfigError("attention: rows that are worked on whole go without mixed values, gates and factors "
+                              "per head, pooled blocks, chunks, and keys lent or borrowed")
+        if params.get("values_from_keys") and vd != hd:
+            raise ConfigError(f"attention: values that are keys are {hd} wide, not {vd}")
         out = {
             "q_proj.weight": TensorDecl((nh * hd, hidden)),
             "k_proj.weight": TensorDecl((nkv * hd, hidden)),
@@ -173,17 +203,26 @@ class Attention:
                 raise ConfigError("attention: a layer that reads another's keys and values has no "
                                   "biases, norms, mixed values or pooled blocks of its own")
             del out["k_proj.weight"], out["v_proj.weight"]
+        if params.get("values_from_keys"):
+            del out["v_proj.weight"]
+        if params.get("qk_conv"):
+            out["q_conv.weight"] = TensorDecl((nh * hd, int(params["qk_conv"])), init="norm")
+            out["k_conv.weight"] = TensorDecl((nkv * hd, int(params["qk_conv"])), init="norm")
+        if params.get("output_gate"):
+            out["gate_proj.weight"] = TensorDecl((nh * vd, hidden))
         if params.get("sink"):
             out["sink"] = TensorDecl((nh,), init="norm")
         if params.get("bias"):
             out["q_proj.bias"] = TensorDecl((nh * hd,), init="norm")
             out["k_proj.bias"] = TensorDecl((nkv * hd,), init="norm")
-            out["v_proj.bias"] = TensorDecl((nkv * vd,), init="norm")
+            if not params.get("values_from_keys"):
+                out["v_proj.bias"] = TensorDecl((nkv * vd,), init="norm")
         if params.get("head_temp"):
             out["temp"] = TensorDecl((nh,), init="norm")
         if params.get("qk_norm") and params["qk_norm"].get("weight", True):
-            out["q_norm.weight"] = TensorDecl((hd,), init="norm")
-            out["k_norm.weight"] = TensorDecl((hd,), init="norm")
+            whole = params["qk_norm"].get("whole")
+            out["q_norm.weight"] = TensorDecl((nh * hd if whole else hd,), init="norm")
+            out["k_norm.weight"] = TensorDecl((nkv * hd if whole else hd,), init="norm")
         if params.get("value_mix"):
             # (the layer whose values the others mix in may store a weight too; it is not read)
             out["value_mix.weight"] = TensorDecl((), init="norm",
@@ -205,24 +244,34 @@ class Attention:
                   Piece("v_proj.weight", (nh + nkv) * hd))
         if params.get("borrows_cache"):       # q alone
             n_qkv, pieces = nh * hd, pieces[:1]
+        if params.get("values_from_keys"):    # q and k
+            n_qkv, pieces = (nh + nkv) * hd, pieces[:2]
+        n_in = n_qkv
         if params.get("head_gate"):       # the gates' rows behind q, k and v: one product makes all
-            pieces += (Piece("g_proj.weight", n_qkv),)
+            pieces += (Piece("g_proj.weight", n_in),)
+            n_in += nh
+        if params.get("output_gate"):
+            pieces += (Piece("gate_proj.weight", n_in),)
+            n_in += nh * vd
         out = {
-            "qkv_proj.weight": Resident((n_qkv + (nh if params.get("head_gate") else 0), hidden),
-                                        pieces=pieces),
+            "qkv_proj.weight": Resident((n_in, hidden), pieces=pieces),
             "o_proj.weight": Resident((hidden, nh * vd), pieces=(Piece("o_proj.weight"),)),
         }
         if params.get("sink"):
             out["sink"] = Resident((nh,), torch.float32, (Piece("sink"),))
         if params.get("bias"):
-            out["qkv_proj.bias"] = Resident((n_qkv,), torch.float32, (
-                Piece("q_proj.bias", 0), Piece("k_proj.bias", nh * hd),
-                Piece("v_proj.bias", (nh + nkv) * hd)))
+            biases = (Piece("q_proj.bias", 0), Piece("k_proj.bias", nh * hd), Piece("v_proj.bias", (nh + nkv) * hd))
+            out["qkv_proj.bias"] = Resident((n_qkv,), torch.float32,
+                                            biases[:2] if params.get("values_from_keys") else biases)
+        if params.get("qk_conv"):
+            out["qk_conv.weight"] = Resident(((nh + nkv) * hd, int(params["qk_conv"])), torch.float32, (
+                Piece("q_conv.weight", 0), Piece("k_conv.weight", nh * hd)))
         if params.get("head_temp"):
             out["temp"] = Resident((nh,), torch.float32, (Piece("temp"),))
         if params.get("qk_norm") and params["qk_norm"].get("weight", True):
-            out["q_norm.gain"] = Resident((hd,), torch.float32, (Piece("q_norm.weight"),))
-            out["k_norm.gain"] = Resident((hd,), torch.float32, (Piece("k_norm.weight"),))
+            whole = params["qk_norm"].get("whole")
+            out["q_norm.gain"] = Resident((nh * hd if whole else hd,), torch.float32, (Piece("q_norm.weight"),))
+            out["k_norm.gain"] = Resident((nkv * hd if whole else hd,), torch.float32, (Piece("k_norm.weight"),))
         if params.get("value_mix") == "mix":
             out["value_mix.weight"] = Resident((1,), torch.float32, (Piece("value_mix.weight"),))
         pos: PartSpec = params["position"]
@@ -248,8 +297,19 @@ class Attention:
         self.lends = bool(params.get("lends_cache"))
         if self.chunk < 0 or (self.chunk and (self.window or params.get("pool"))):
             raise ConfigError("attention: a chunked mask goes without a window and pooled blocks")
-        if (self.chunk or self.sink is not None) and float(params.get("logit_softcap") or 0.0):
-            raise ConfigError("attention: a chunked mask or a sink goes without a soft cap")
+        if params.get("sink_score") is not None:
+            if self.sink is not None:
+                raise ConfigError("attention: stored sinks or one score for all, not both")
+            self.sink = torch.full((self.nh,), float(params["sink_score"]), dtype=torch.float32, device=rt.device)
+        self.exact_cap = bool(params.get("exact_cap"))
+        # a chunked mask, or keys lent or borrowed: kernels of its own choice
+        self.masked = self.chunk > 0 or (self.sink is not None and (self.borrows or self.lends))
+        if self.masked and self.softcap:
+            raise ConfigError("attention: a chunked mask, or a sink with keys lent or borrowed, goes without a soft cap")
+        if self.masked and self.window:
+            raise ConfigError("attention: keys lent or borrowed with a sink go without a window")
+        if self.sink is not None and params.get("pool"):
+            raise ConfigError("attention: pooled blocks go without a sink")
         self.keep = int(params.get("keep_first") or 0)
         if self.keep < 0 or (self.keep and (self.window <= 0 or params.get("pool") or self.softcap)):
             raise ConfigError("attention: kept first positions go with a window, and without pooled blocks "
@@ -276,6 +336,16 @@ class Attention:
             norm = params.get("qk_norm")
             self.qk_eps = float(norm["eps"]) if norm else 0.0
             self.norm_after = bool(norm and norm.get("after_rotation"))
+            self.rows_whole = self._row_work(params)
+            if self.rows_whole and norm and not (norm.get("whole") and norm.get("weight", True)):
+                raise ConfigError("attention: rows that are worked on whole are normed whole, with weights")
+            self.taps = int(params.get("qk_conv") or 0)
+            if not 0 <= self.taps <= 64:
+                raise ConfigError(f"attention: a convolution of {self.taps} taps (1 to 64)")
+            self.values_from_keys = bool(params.get("values_from_keys"))
+            self.output_gate = bool(params.get("output_gate"))
+            # (neighbouring threads take neighbouring channels: tap by tap)
+            self.conv = weights["qk_conv.weight"].t().contiguous() if self.taps else None
             if norm and self.norm_after == bool(norm.get("weight", True)):
                 raise ConfigError("attention: q and k are normed with weights before the rotation, or without "
                                   "weights behind it")
@@ -289,7 +359,7 @@ class Attention:
             self.lam = weights.get("value_mix.weight")
             self.head_gate = bool(params.get("head_gate"))
             self.n_qkv = self.nh * self.hd if self.borrows \
-                else (self.nh + self.nkv) * self.hd + self.nkv * self.vd
+                else (self.nh + self.nkv) * self.hd + (0 if self.values_from_keys else self.nkv * self.vd)
             rotary = self.position.rotary() if hasattr(self.position, "rotary") else None
             if rotary is None:
                 raise ConfigError("attention: worked-on heads take a rotary position part (or 'none')")
@@ -302,8 +372,12 @@ class Attention:
         self._block_warps = tuple(int(w) for w in os.environ.get("SIB_DECODE_WARPS", "8,4,2").split(","))
 
     def cache_need(self) -> Optional[CacheNeed]:
+        state = None
+        if self.extras and self.taps > 1:
+            # (whole groups of 4 floats, so that every slot's state begins on a 16-byte boundary)
+            state = StateNeed((-(-(self.taps - 1) * (self.nh + self.nkv) * self.hd // 4) * 4,))
         return CacheNeed(kv=KVNeed(self.nkv, self.kw, self.window, pool=self.pool, chunk=self.chunk,
-                                   keep_first=self.keep))
+                                   keep_first=self.keep), state=state)
 
     # ------------------------------------------------------------------
     def _longest(self, ctx, capacity: int) -> int:
@@ -407,7 +481,8 @@ class Attention:
                                     max(memo["ends"]), nh, nkv, hd, self.scale, self.softcap,
                                     self.window, rt.scratch(need) if need else None,
                                     rt.tickets(n_tickets) if need else None, lens,
-                                    memo["d_starts"], ctx.starts if lens else None, keep=self.keep)
+                                    memo["d_starts"], ctx.starts if lens else None, sink=self.sink,
+                                    keep=self.keep, close_cap=self.exact_cap)
         r = 0
         for row0, st, n in zip(memo["row0"], ctx.starts, ctx.counts):
             out[r:r + n].copy_(whole[row0 + st:row0 + st + n])
@@ -529,14 +604,25 @@ class Attention:
                 v_first = ctx.memo.get("value_mix.first")
                 if v_first is None:
                     raise ValueError("attention: values to mix in, but no earlier layer left any")
-            native.head_prepare(proj, qkv, self.bias, self.q_gain, self.k_gain, self.qk_eps,
-                                rotary[0], rotary[1], v_first, self.lam if v_first is not None else None,
-                                ctx.row_pos, ctx.row_seq, ctx.seq_slot, ctx.seq_end,
-                                view.k if owns_cache else None, view.v if owns_cache else None,
-                                view.page_table if owns_cache else None, view.page_tokens,
-                                view.ring_tokens, nh, nkv, self.hd, self.vd, hd, style=self.rope_style,
-                                norm_after=self.norm_after, temp=self.temp, magnitude=self.magnitude,
-                                fixed_tokens=view.fixed_tokens)
+            if self.rows_whole and not owns_cache:
+                raise ValueError("attention: rows that are worked on whole cannot read another run's cache")
+            if self.rows_whole:
+                native.row_prepare(
+                    proj, qkv, ctx, n_heads=nh, n_kv=nkv, key_dim=self.hd, value_dim=self.vd,
+                    values_from_keys=self.values_from_keys, bias=self.bias, conv=self.conv,
+                    state=ctx.state(entry) if self.taps > 1 else None, q_gain=self.q_gain, k_gain=self.k_gain,
+                    eps=self.qk_eps, inv_freq=rotary[0], rotary_dim=rotary[1], style=self.rope_style,
+                    magnitude=self.magnitude, k_pool=view.k, v_pool=view.v, page_table=view.page_table,
+                    page_tokens=view.page_tokens, ring_tokens=view.ring_tokens, fixed_tokens=view.fixed_tokens)
+            else:
+                native.head_prepare(proj, qkv, self.bias, self.q_gain, self.k_gain, self.qk_eps,
+                                    rotary[0], rotary[1], v_first, self.lam if v_first is not None else None,
+                                    ctx.row_pos, ctx.row_seq, ctx.seq_slot, ctx.seq_end,
+                                    view.k if owns_cache else None, view.v if owns_cache else None,
+                                    view.page_table if owns_cache else None, view.page_tokens,
+                                    view.ring_tokens, nh, nkv, self.hd, self.vd, hd, style=self.rope_style,
+                                    norm_after=self.norm_after, temp=self.temp, magnitude=self.magnitude,
+                                    fixed_tokens=view.fixed_tokens)
             if self.pool:
                 native.pool_store(qkv, view, ctx, nh, nkv, hd)
             if self.value_mix == "first":
@@ -581,7 +667,7 @@ class Attention:
         tc_prompt = (fresh and qkv.dtype == torch.bfloat16 and _USE_TCGEN05_PREFILL and self.scale > 0
                      and not short and native.attention_prefill_tc_supports(nh, self.nkv, hd, width)
                      and not (self.pool and self.softcap))
-        if self.chunk > 0 or self.sink is not None:
+        if self.masked:
             out = self._attend_masked(qkv, out, ctx, view, owns_cache, cache_entry)
         elif self.pool and not tc_prompt:
             # blocks before the window join the softmax: the general kernel, which reads the
@@ -627,20 +713,20 @@ class Attention:
                                         ctx.max_count, nh, self.nkv, hd, self.scale, self.softcap,
                                         self.window, rt.scratch(need) if need else None,
                                         rt.tickets(n_tickets) if need else None, lens, extra=extra,
-                                        keep=self.keep)
+                                        sink=self.sink, keep=self.keep, close_cap=self.exact_cap)
         elif fresh and qkv.dtype == torch.bfloat16 and \
                 native.attention_prefill_supports(nh, self.nkv, hd):
             native.attention_prefill(qkv, out, ctx.seq_row0, ctx.seq_end, ctx.n_seqs,
                                      ctx.max_count, nh, self.nkv, hd, self.scale, self.softcap,
-                                     self.window, self.keep)
+                                     self.window, self.keep, self.sink, self.exact_cap)
         elif fresh:
             k_new = qkv[:, nh * hd:]
             v_new = qkv[:, (nh + nkv) * hd:]
             native.attention_rows(qkv, width, k_new, v_new, width, None, None, None,
                                   view.page_tokens, view.ring_tokens, ctx.row_pos, ctx.row_seq,
                                   ctx.seq_slot, ctx.seq_start, ctx.seq_row0, out, None, nh,
-                                  self.nkv, hd, self.scale, self.softcap, self.window, 1, keep=self.keep,
-                                  fixed_tokens=view.fixed_tokens)
+                                  self.nkv, hd, self.scale, self.softcap, self.window, 1, sink=self.sink,
+                                  keep=self.keep, fixed_tokens=view.fixed_tokens)
         elif (qkv.dtype == torch.bfloat16 and not ctx.graph_capture
               and ctx.max_count >= rt.piece_attention_rows and _USE_TCGEN05_PREFILL and self.scale > 0
               and native.attention_prefill_tc_supports(nh, self.nkv, hd, (nh + 2 * self.nkv) * hd)
@@ -657,8 +743,8 @@ class Attention:
                                     view.ring_tokens, ctx.row_pos, ctx.row_seq, ctx.seq_slot, out,
                                     scratch, tickets, nh, self.nkv, hd, self.scale, self.softcap,
                                     self.window, splits, warps,
-                                    fresh=ctx.max_count if rt.early_keys else 0, keep=self.keep,
-                                    fixed_tokens=view.fixed_tokens)
+                                    fresh=ctx.max_count if rt.early_keys else 0, sink=self.sink,
+                                    keep=self.keep, fixed_tokens=view.fixed_tokens)
         else:
             splits = self._splits(ctx, ctx.cache.max_seq_len)
             scratch = None
@@ -667,9 +753,16 @@ class Attention:
             native.attention_rows(qkv, width, None, None, width, view.k, view.v, view.page_table,
                                   view.page_tokens, view.ring_tokens, ctx.row_pos, ctx.row_seq,
                                   ctx.seq_slot, ctx.seq_start, ctx.seq_row0, out, scratch, nh,
-                                  self.nkv, hd, self.scale, self.softcap, self.window, splits,
+                                  self.nkv, hd, self.scale, self.softcap, self.window, splits, sink=self.sink,
                                   keep=self.keep, fixed_tokens=view.fixed_tokens)
-        if self.extras and (self.head_gate or self.vd != hd):
+        if self.extras and self.output_gate:
+            y = torch.empty((R, nh * self.vd), dtype=out.dtype, device=out.device)
+            at = self.n_qkv + (nh if self.head_gate else 0)
+            heads = out.view(R, nh, hd)
+            if self.head_gate:
+                heads = native.head_gate(out, proj[:, self.n_qkv:at], torch.empty_like(y), nh, self.vd, hd).view(R, nh, self.vd)
+            out = native.element_gate(heads, proj[:, at:at + nh * self.vd], y, nh, self.vd)
+        elif self.extras and (self.head_gate or self.vd != hd):
             y = torch.empty((R, nh * self.vd), dtype=out.dtype, device=out.device)
             gate = proj[:, self.n_qkv:self.n_qkv + nh] if self.head_gate else None
             out = native.head_gate(out, gate, y, nh, self.vd, hd)
@@ -688,7 +781,12 @@ class LatentAttention:
     exponential joins the softmax's denominator), ``head_gate`` (sigmoid(g_proj x) per head
     on the head's output), ``q_rank`` (r > 0: the queries pass a latent of their own,
     q = uq_proj (rms_norm(dq_proj x) * dq_norm.weight) with r the latent's width, instead of
-    q = q_proj x; the norm is 32-bit and takes ``norm_eps``).
+    q = q_proj x; the norm is 32-bit and takes ``norm_eps``), ``output_gate`` (the concatenated
+    values are multiplied element by element by sigmoid(gate_proj x)), ``borrows_cache`` (the layer
+    has no down projection: its schedule entry names the run whose cached rows, latent and
+    rotated part, it reads with its own queries, U and V), ``lends_cache`` (a later run reads this
+    layer's rows; in a step of prompts they are left for it packed).
+    The rotation may be in neighbouring or in half-split pairs and may have a magnitude (YaRN).
 
         q_h = [a_h | r_h] = q_proj x (per head);  k_h = [U_h c | rot(k_r)],  v_h = V_h c
         score_h(t, j) = (<a_h(t), U_h c(j)> + <rot(r_h(t)), rot(k_r(j))>) * score_scale
@@ -703,6 +801,7 @@ class LatentAttention:
     """
 
     captures_prompts = True      # sequences, slots and counts are read on the device only
+    captures_borrowed = True     # (a borrower takes the lender's packed rows in a step of prompts)
 
     @staticmethod
     def _sizes(params: Mapping):
@@ -735,22 +834,35 @@ class LatentAttention:
             out["sink"] = TensorDecl((nh,), init="norm")
         if params.get("head_gate"):
             out["g_proj.weight"] = TensorDecl((nh, hidden))
+        if params.get("output_gate"):
+            out["gate_proj.weight"] = TensorDecl((nh * vd, hidden))
+        if params.get("borrows_cache"):
+            del out["dkv_proj.weight"], out["dkv_norm.weight"]
         return out
 
     @classmethod
     def resident(cls, params: Mapping, hidden: int) -> Dict[str, Resident]:
-        """The query heads, the down projection and the gates as ONE matrix."""
+        """The query heads, the down projection (of a layer that has one) and the gates as ONE
+        matrix."""
         nh, qd, rd, vd, rank, _ = cls._sizes(params)
         q_rank = int(params.get("q_rank") or 0)
         n_q = q_rank or nh * (qd + rd)      # rows of the first piece: the queries, or their latent
-        pieces = (Piece("dq_proj.weight" if q_rank else "q_proj.weight", 0), Piece("dkv_proj.weight", n_q))
-        n_in = n_q + rank + rd
+        pieces = (Piece("dq_proj.weight" if q_rank else "q_proj.weight", 0),)
+        n_in = n_q
+        borrows = bool(params.get("borrows_cache"))
+        if not borrows:
+            pieces += (Piece("dkv_proj.weight", n_in),)
+            n_in += rank + rd
         if params.get("head_gate"):
             pieces += (Piece("g_proj.weight", n_in),)
             n_in += nh
+        if params.get("output_gate"):
+            pieces += (Piece("gate_proj.weight", n_in),)
+            n_in += nh * vd
         out = {
             "in_proj.weight": Resident((n_in, hidden), pieces=pieces),
-            "dkv_norm.gain": Resident((rank,), torch.float32, (Piece("dkv_norm.weight"),)),
+            **({} if borrows else {
+                "dkv_norm.gain": Resident((rank,), torch.float32, (Piece("dkv_norm.weight"),))}),
             "uk_proj.weight": Resident((nh * qd, rank), pieces=(Piece("uk_proj.weight"),)),
             "uv_proj.weight": Resident((nh * vd, rank), pieces=(Piece("uv_proj.weight"),)),
             "o_proj.weight": Resident((hidden, nh * vd), pieces=(Piece("o_proj.weight"),)),
@@ -777,18 +889,20 @@ class LatentAttention:
         position = part_class("position", pos.kind)(pos.params, max(self.rd, 2), {}, rt) \
             if self.rd else None
         self.inv_freq, self.rot = None, 0
+        self.turn = {"style": native.ROPE_INTERLEAVED, "magnitude": 1.0}
         if position is not None:
             if not hasattr(position, "rotary"):
                 raise ConfigError("latent_attention: the position part must offer rotary()")
-            if getattr(position, "magnitude", 1.0) != 1.0:
-                raise ConfigError("latent_attention: a rotation with a magnitude other than 1 is not built")
-            self.inv_freq, self.rot, style = position.rotary()
-            if self.rot and style != native.ROPE_INTERLEAVED:
-                raise ConfigError("latent_attention: the rotated columns are rotated in neighbouring pairs")
+            self.turn["magnitude"] = float(getattr(position, "magnitude", 1.0))
+            self.inv_freq, self.rot, self.turn["style"] = position.rotary()
+        self.borrows, self.lends = bool(params.get("borrows_cache")), bool(params.get("lends_cache"))
         self.head_gate = bool(params.get("head_gate"))
+        self.output_gate = bool(params.get("output_gate"))
+        if self.head_gate and self.output_gate:
+            raise ConfigError("latent_attention: one gate per head or one per element, not both")
         self.n_q = self.nh * (self.qd + self.rd)
         self.w_in = rt.cast_matrix(weights["in_proj.weight"])
-        self.c_gain = weights["dkv_norm.gain"]
+        self.c_gain = weights.get("dkv_norm.gain")
         # per head: U_h [qd, rank] (q times it) and V_h^T [rank, vd] (the summed latents times it)
         w_uk, w_uv = rt.cast_matrix(weights["uk_proj.weight"]), rt.cast_matrix(weights["uv_proj.weight"])
         self.w_uk = w_uk.view(self.nh, self.qd, self.rank)
@@ -825,21 +939,31 @@ class LatentAttention:
     def _project(self, x: torch.Tensor):
         """(rows that begin with the query heads, the down projection's rows where they do not
         follow the query heads or None, the gates' columns or None)."""
-        rt, tail = self.rt, self.rank + self.rd
+        rt, tail = self.rt, 0 if self.borrows else self.rank + self.rd
+        n_gate = self.nh if self.head_gate else self.nh * self.vd if self.output_gate else 0
         first = rt.linear(x, self.w_in)
         rt.flush()
         if not self.q_rank:
-            gate = first[:, self.n_q + tail:self.n_q + tail + self.nh] if self.head_gate else None
-            return first, None, gate
+            at = self.n_q + tail
+            return first, None, first[:, at:at + n_gate] if n_gate else None
         # the queries' own latent: normed in 32-bit, then up to the heads
         cq = torch.empty((x.shape[0], self.q_rank), dtype=first.dtype, device=first.device)
         native.rms_norm(first[:, :self.q_rank], self.q_gain, self.eps, cq)
         q = rt.linear(cq, self.w_uq)
         rt.flush()
         at = self.q_rank + tail
-        return q, first[:, self.q_rank:at], first[:, at:at + self.nh] if self.head_gate else None
+        return q, first[:, self.q_rank:at] if tail else None, first[:, at:at + n_gate] if n_gate else None
 
-    def _attend_expanded(self, proj: torch.Tensor, down, gate, ctx, view) -> torch.Tensor:
+    def _gated(self, vals: torch.Tensor, gate) -> torch.Tensor:
+        """``vals``: a view [rows, heads, value_dim] of any strides -> [rows, heads * value_dim], times
+        the gate per element if there is one."""
+        R = vals.shape[0]
+        if not self.output_gate:
+            return vals.reshape(R, self.nh * self.vd)
+        y = torch.empty((R, self.nh * self.vd), dtype=vals.dtype, device=vals.device)
+        return native.element_gate(vals, gate, y, self.nh, self.vd)
+
+    def _attend_expanded(self, proj: torch.Tensor, down, gate, ctx, view, cache_entry: int, lent) -> torch.Tensor:
         """Long prompts in bfloat16: the latent rows are normed, rotated and cached as ever, and
         for the step's own rows keys and values are made per head (k_h = U_h c, v_h = V_h c:
         two library products) and attended over by the tcgen05 prompt kernel, with the sink as
@@ -847,10 +971,14 @@ class LatentAttention:
         the latent, on the faster tensor-core path.  Later steps read the cached latent rows."""
         rt, nh, qd, rd, vd, rank, kw, hw = self.rt, self.nh, self.qd, self.rd, self.vd, self.rank, self.kw, self.hw
         R = proj.shape[0]
-        k_rows = torch.empty((R, kw), dtype=proj.dtype, device=proj.device)
-        native.latent_prepare(proj, None, None, k_rows, self.c_gain, self.eps, self.inv_freq, self.rot,
-                              ctx, view.k, view.page_table, view.page_tokens, view.ring_tokens, nh, qd, rd,
-                              rank, kw, down)
+        k_rows = lent
+        if lent is None:
+            k_rows = torch.empty((R, kw), dtype=proj.dtype, device=proj.device)
+            native.latent_prepare(proj, None, None, k_rows, self.c_gain, self.eps, self.inv_freq, self.rot,
+                                  ctx, view.k, view.page_table, view.page_tokens, view.ring_tokens, nh, qd, rd,
+                                  rank, kw, down, **self.turn)
+            if self.lends:
+                ctx.memo[("latent_rows", cache_entry)] = k_rows
         c_rows = k_rows[:, :rank]
         with native.profile_region("library product (latent rows to keys and values)",
                                    (nh * (qd + vd) * rank + R * (rank + nh * (qd + vd))) * proj.element_size(),
@@ -859,7 +987,7 @@ class LatentAttention:
             v_heads = torch.matmul(c_rows, self.w_uv_flat.t())
         qkv = torch.empty((R, 3 * nh * hw), dtype=proj.dtype, device=proj.device)
         native.latent_expand(proj, k_rows, k_heads, v_heads, qkv, self.inv_freq, self.rot, ctx.row_pos,
-                             nh, qd, rd, vd, rank, kw, hw)
+                             nh, qd, rd, vd, rank, kw, hw, **self.turn)
         out = torch.empty((R, nh * hw), dtype=proj.dtype, device=proj.device)
         lens = None if ctx.graph_capture else ctx.counts
         n_items = 0
@@ -871,14 +999,17 @@ class LatentAttention:
         native.attention_prefill_tc(qkv, out, ctx.seq_row0, ctx.seq_end, ctx.n_seqs, ctx.max_count, nh, nh,
                                     hw, self.scale, 0.0, self.window, rt.scratch(need) if need else None,
                                     rt.tickets(n_tickets) if need else None, lens, sink=self.sink)
+        if self.output_gate:
+            return rt.linear(self._gated(out.view(R, nh, hw), gate), self.w_o)
         vals = torch.empty((R, nh * vd), dtype=out.dtype, device=out.device)
         native.head_gate(out, gate, vals, nh, vd, hw)
         return rt.linear(vals, self.w_o)
 
     def forward(self, x: torch.Tensor, ctx, entry: int, cache_entry: int,
                 owns_cache: bool) -> torch.Tensor:
-        if not owns_cache:
-            raise ValueError("latent_attention: reading another run's cache is not built")
+        if owns_cache == self.borrows:
+            raise ValueError("latent_attention: a layer without a down projection reads another run's rows, "
+                             "one with it its own")
         rt, nh, qd, rd, rank, kw = self.rt, self.nh, self.qd, self.rd, self.rank, self.kw
         R = x.shape[0]
         view = ctx.kv(cache_entry)
@@ -891,11 +1022,15 @@ class LatentAttention:
                         f"a step may add at most {max(room, view.ring_tokens - start)} positions "
                         f"to a sequence of {start} whose layers keep a window of {self.window} "
                         f"in a ring of {view.ring_tokens}; got {n}")
+        # in a step of prompts a borrower takes the rows that the lender has left packed
+        lent = ctx.memo.get(("latent_rows", cache_entry)) if self.borrows and fresh else None
+        if self.borrows and fresh and (lent is None or lent.shape != (R, kw)):
+            raise ValueError("latent_attention: no earlier run has left the rows that this one reads")
         proj, down, gate = self._project(x)
         if (fresh and proj.dtype == torch.bfloat16 and _USE_LATENT_EXPAND and _USE_TCGEN05_PREFILL
                 and self.hw and self.scale > 0 and ctx.max_count > rt.short_prompt_tokens
                 and native.attention_prefill_tc_supports(nh, nh, self.hw, 3 * nh * self.hw)):
-            return self._attend_expanded(proj, down, gate, ctx, view)
+            return self._attend_expanded(proj, down, gate, ctx, view, cache_entry, lent)
         # the unrotated query columns of every head into the latent's space: [heads, rows, rank]
         q_heads = proj[:, :self.n_q].view(R, nh, qd + rd)[:, :, :qd].transpose(0, 1)
         with native.profile_region("library product (queries into the latent space)",
@@ -903,10 +1038,14 @@ class LatentAttention:
                                    2.0 * R * nh * qd * rank):
             q_lat = torch.bmm(q_heads, self.w_uk)
         q_rows = torch.empty((R, nh * kw), dtype=proj.dtype, device=proj.device)
-        k_rows = torch.empty((R, kw), dtype=proj.dtype, device=proj.device)
+        k_rows = None if self.borrows else torch.empty((R, kw), dtype=proj.dtype, device=proj.device)
         native.latent_prepare(proj, q_lat, q_rows, k_rows, self.c_gain, self.eps, self.inv_freq,
-                              self.rot, ctx, view.k, view.page_table, view.page_tokens,
-                              view.ring_tokens, nh, qd, rd, rank, kw, down)
+                              self.rot, ctx, None if self.borrows else view.k, view.page_table, view.page_tokens,
+                              view.ring_tokens, nh, qd, rd, rank, kw, down, **self.turn)
+        if lent is not None:
+            k_rows = lent
+        elif self.lends and fresh:
+            ctx.memo[("latent_rows", cache_entry)] = k_rows
         out = torch.empty((R, nh * kw), dtype=proj.dtype, device=proj.device)
         tensor_cores = (proj.dtype == torch.bfloat16 and _USE_LATENT_MMA
                         and native.attention_latent_supports(nh, kw))
@@ -937,15 +1076,18 @@ class LatentAttention:
                                   ctx.seq_slot, ctx.seq_start, ctx.seq_row0, out, scratch, nh, 1, kw,
                                   self.scale, 0.0, self.window, splits, sink=self.sink,
                                   values_in_keys=True)
-        # the heads' summed latents (gated), then V_h per head
-        lat = torch.empty((R, nh * rank), dtype=out.dtype, device=out.device)
-        native.head_gate(out, gate, lat, nh, rank, kw)
+        # the heads' summed latents (gated per head, or read where they lie), then V_h per head
+        if self.head_gate:
+            lat = torch.empty((R, nh * rank), dtype=out.dtype, device=out.device)
+            native.head_gate(out, gate, lat, nh, rank, kw)
+            lat = lat.view(R, nh, rank)
+        else:
+            lat = out.view(R, nh, kw)[:, :, :rank]
         with native.profile_region("library product (summed latents to values)",
                                    (nh * self.vd * rank + R * nh * (self.vd + rank)) * out.element_size(),
                                    2.0 * R * nh * self.vd * rank):
-            vals = torch.bmm(lat.view(R, nh, rank).transpose(0, 1), self.w_uv_t)     # [heads, rows, vd]
-            vals = vals.transpose(0, 1).reshape(R, nh * self.vd)
-        return rt.linear(vals, self.w_o)
+            vals = torch.bmm(lat.transpose(0, 1), self.w_uv_t)     # [heads, rows, vd]
+        return rt.linear(self._gated(vals.transpose(0, 1), gate), self.w_o)
 
 
 register_mixer("attention", Attention)

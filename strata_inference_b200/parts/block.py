@@ -17,8 +17,8 @@ that norms a sub-layer's output only: h += post(sublayer(h)).  The
 residual stream h is kept and summed in 32-bit.  When the norms around an
 add are RMS norms the block runs "norm of the sub-layer's output, add, norm
 for the next sub-layer" as one kernel (csrc/norm.cu add_rms_norm), reaching
-over to the next block's first norm when the model passes it; Dynamic Tanh norms around an
-add are fused in the same way (add_dyt_norm).
+over to the next block's first norm when the model passes it; Dynamic Tanh norms and layer norms
+around an add are fused in the same way (add_dyt_norm, add_layer_norm).
 
 A sandwich or pre-norm block may carry a *mixer input* (a registered "mixer_input" part, such as
 ``short_conv``): it works on the pre-mixer norm's rows before the mixer reads them,
@@ -52,6 +52,15 @@ def _fusable(norm) -> bool:
 
 def _fusable_dyt(norm) -> bool:
     return norm is None or getattr(norm, "fusable_dyt", False)
+
+
+def _passes_rows(norm) -> bool:
+    """The identity norm: the stream's rows as activations."""
+    return norm is not None and getattr(norm, "fusable_rms", False) and norm.gain is None
+
+
+def _fusable_ln(norm) -> bool:
+    return norm is None or getattr(norm, "fusable_ln", False)
 
 
 class SandwichBlock:
@@ -115,6 +124,13 @@ class SandwichBlock:
             out = torch.empty_like(y) if nxt is not None else None
             native.add_dyt_norm(y, post.triple if post is not None else None, h,
                                 nxt.triple if nxt is not None else None, out, self.residual_scale)
+            return out
+        if _fusable_ln(post) and (_fusable_ln(nxt) or _passes_rows(nxt)) and self.residual_scale == 1.0:
+            # layer norms around the add (or the plain rows behind it)
+            self.rt.flush()
+            out = torch.empty_like(y) if nxt is not None else None
+            native.add_layer_norm(y, post.triple if post is not None else None, h,
+                                  nxt.triple if nxt is not None and not _passes_rows(nxt) else None, out)
             return out
         self.rt.flush()         # the steps below read y and h outside the chain
         if post is not None:

@@ -15,6 +15,9 @@ that the block arrangements and their fused "norm, add, norm" step serve it as t
 element in 32-bit, with one stored number ``alpha`` and one ``weight`` and ``b`` per
 column.  Blocks fuse it into the residual add as they fuse the RMS norm (``fusable_dyt``,
 csrc/norm.cu add_dyt_norm).
+
+``layer_norm``: (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + b, 32-bit.  Blocks fuse it
+into the residual add too (``fusable_ln``, csrc/norm.cu add_layer_norm).
 """
 
 from __future__ import annotations
@@ -122,6 +125,42 @@ class DynamicTanh:
         return native.dyt_norm(x, self.weight, self.b, self.alpha, out, rows)
 
 
+class LayerNorm:
+    fusable_rms = False
+    fusable_ln = True
+
+    @staticmethod
+    def tensors(params: Mapping, hidden: int) -> Dict[str, TensorDecl]:
+        return {"weight": TensorDecl((hidden,), init="norm"), "b": TensorDecl((hidden,), init="norm")}
+
+    @staticmethod
+    def resident(params: Mapping, hidden: int) -> Dict[str, Resident]:
+        return {"weight": Resident((hidden,), torch.float32, (Piece("weight"),)),
+                "b": Resident((hidden,), torch.float32, (Piece("b"),))}
+
+    def __init__(self, params: Mapping, hidden: int, weights: Mapping[str, torch.Tensor], rt):
+        self.hidden = hidden
+        self.rt = rt
+        self.eps = float(params["eps"])
+        self.weight, self.b = weights["weight"], weights["b"]
+
+    def scale_output(self, factor: float) -> None:
+        """The norm's output times a constant, in 32-bit (a head's scale on its logits)."""
+        self.weight, self.b = self.weight * factor, self.b * factor
+
+    @property
+    def triple(self):
+        """(weight, bias, eps) as the fused residual kernel takes them."""
+        return self.weight, self.b, self.eps
+
+    def forward(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
+                rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        n = x.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.hidden), dtype=out_dtype or self.rt.dtype, device=x.device)
+        return native.layer_norm(x, self.weight, self.b, self.eps, out, rows)
+
+
 register_norm("rms_norm", RMSNorm)
+register_norm("layer_norm", LayerNorm)
 register_norm("dynamic_tanh", DynamicTanh)
 register_norm("identity", IdentityNorm)

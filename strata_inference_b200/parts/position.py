@@ -10,6 +10,9 @@ cosine are taken in 32-bit inside the kernel (csrc/rope_cache.cu).
 their frequency, pairs that turn rarely are slowed down by ``factor``, with a ramp over the
 pair's index between the indices that make ``fast`` and ``slow`` turns; cosines and sines are
 multiplied by 0.1 ln(factor) + 1 (``magnitude``).
+``llama3`` {factor, low, high, original} (the frequency scaling of Llama 3.1): with L = 2 pi / f a
+pair's wavelength, f stays where L < original / high, becomes f / factor where L > original / low,
+and between the two a mean of both, weighed by how many turns it makes in ``original`` positions.
 ``frequencies: "float64"`` evaluates theta^(-2i/rot) in 64-bit and rounds once to 32-bit.
 ``none``: no encoding.
 
@@ -47,6 +50,18 @@ def yarn(freqs: torch.Tensor, rotary_dim: int, theta: float, scaling: Mapping) -
     return freqs / factor * ramp + freqs * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
+def llama3(freqs: torch.Tensor, scaling: Mapping) -> torch.Tensor:
+    """Frequencies (64-bit) with the long wavelengths slowed down by ``factor``."""
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+    low, high = float(scaling["low"]), float(scaling["high"])
+    length = 2.0 * math.pi / freqs
+    turns = original / length
+    share = (turns - low) / (high - low) if high != low else torch.zeros_like(freqs)
+    between = (1.0 - share) * freqs / factor + share * freqs
+    return torch.where(length < original / high, freqs,
+                       torch.where(length > original / low, freqs / factor, between))
+
+
 class Rope:
     style = native.ROPE_HALF_SPLIT
     magnitude = 1.0
@@ -61,11 +76,15 @@ class Rope:
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= head_dim:
             raise ConfigError(f"rotary_dim {self.rotary_dim} must be even and at most "
                               f"head_dim {head_dim}")
-        if params.get("frequencies") == "float64" or params.get("yarn"):
+        if params.get("yarn") and params.get("llama3"):
+            raise ConfigError("rope: 'yarn' and 'llama3' scale the same frequencies; one of them at most")
+        if params.get("frequencies") == "float64" or params.get("yarn") or params.get("llama3"):
             two_i = torch.arange(self.rotary_dim // 2, dtype=torch.float64) * 2.0
             freqs = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -two_i / self.rotary_dim)
             if params.get("yarn"):
                 freqs, self.magnitude = yarn(freqs, self.rotary_dim, self.theta, params["yarn"])
+            if params.get("llama3"):
+                freqs = llama3(freqs, params["llama3"])
             freqs = freqs.to(torch.float32)
         else:
             inv_ndims = torch.tensor(-1.0 / self.rotary_dim, dtype=torch.float32)
