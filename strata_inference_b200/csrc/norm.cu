@@ -218,11 +218,12 @@ add_rms_norm_bf16_warp_kernel(const __nv_bfloat16* __restrict__ a, const float* 
 // One block per row, one 8-element group per thread, the row in registers: every load of a
 // row is issued before anything is computed (the gains even before the kernel ahead of this
 // one has finished), so a row costs two block-wide sums and no pass over shared memory.
+// (a, h and out are not marked __restrict__: the compiler may move a load through such a pointer
+// ahead of the wait for the kernel that writes there.)
 __global__ void __launch_bounds__(1024)
-add_rms_norm_bf16_group_kernel(const __nv_bfloat16* __restrict__ a, const float* __restrict__ post_gain,
-                               float post_eps, float* __restrict__ h,
-                               const float* __restrict__ pre_gain, float pre_eps,
-                               __nv_bfloat16* __restrict__ out, int hidden) {
+add_rms_norm_bf16_group_kernel(const __nv_bfloat16* a, const float* __restrict__ post_gain,
+                               float post_eps, float* h, const float* __restrict__ pre_gain, float pre_eps,
+                               __nv_bfloat16* out, int hidden) {
     __shared__ float scratch[33];
     pdl_trigger();
     const int c = 8 * threadIdx.x;

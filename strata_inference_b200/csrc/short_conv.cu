@@ -166,11 +166,13 @@ __global__ void __launch_bounds__(256) short_conv_state_kernel(const T* __restri
 // One block per row, 8 channels a thread.  HELD: how many of the state's rows are asked for at
 // the start (taps - 1 when it is that small and the block leaves the registers for it, else 0:
 // each is read where it is used).
+// (a, h and y are not marked __restrict__: the compiler may move a load through such a pointer
+// ahead of the wait for the kernel that writes there.)
 template <int HELD, int THREADS>
 __global__ void __launch_bounds__(THREADS)
-add_norm_conv_kernel(const __nv_bfloat16* __restrict__ a, const float* __restrict__ post_gain, float post_eps,
-                     float* __restrict__ h, const float* __restrict__ pre_gain, float pre_eps,
-                     __nv_bfloat16* __restrict__ y, ConvArgs p) {
+add_norm_conv_kernel(const __nv_bfloat16* a, const float* __restrict__ post_gain, float post_eps,
+                     float* h, const float* __restrict__ pre_gain, float pre_eps,
+                     __nv_bfloat16* y, ConvArgs p) {
     __shared__ float scratch[33];
     pdl_trigger();
     const int hidden = p.channels, taps = p.taps, r = blockIdx.x;
