@@ -1,0 +1,116 @@
+"""Small Simetar configurations for the tests, random weights for them, and the comparison with
+the plain model (tests/plain_simetar.py)."""
+
+from __future__ import annotations
+
+import copy
+import math
+import random
+from typing import Dict, List, Sequence
+
+import numpy as np
+import torch
+
+import plain_simetar as plain
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def llama3(factor=6.0, low=1.0, high=3.0, original=100):
+    return {"factor": factor, "low": low, "high": high, "original": original}
+
+
+def yarn(factor=4.0, original=96, fast=8.0, slow=1.0):
+    return {"factor": factor, "original": original, "fast": fast, "slow": slow}
+
+
+def _rot(dims, base, scaling):
+    rot = {"base": base, "dims": dims}
+    if scaling:
+        rot["scaling"] = scaling
+    return rot
+
+
+def attention(heads, kv_heads, dim, size, conv=3, scale=0.2, softcap=15.0, rot_dims=None, base=10000.0, scaling=None,
+              mlp=None):
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv, "scale": scale}
+    if softcap:
+        mixer["softcap"] = softcap
+    if rot_dims != 0:
+        mixer["rot"] = _rot(dim if rot_dims is None else rot_dims, base, scaling)
+    if size:
+        mixer["mask"] = {"size": size}
+    return {"type": "attention", "mixer": mixer, "mlp": mlp}
+
+
+def latent(heads, dim, rot_dim, vdim, rank, scale=0.3, base=10000.0, scaling=None, kv_from=None, mlp=None):
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "scale": scale,
+             "rot": _rot(rot_dim, base, scaling)}
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+
+
+def model(width, vocab, layers, eps=1e-5):
+    return {"architecture": "Simetar", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": list(layers)}
+
+
+# one mechanism at a time
+ALONE = {
+    "open": model(64, 200, [attention(4, 2, 16, 0, conv=1, softcap=0, rot_dims=0)]),
+    "conv": model(64, 200, [attention(2, 2, 16, 0, conv=5, rot_dims=0)]),
+    "two_taps": model(64, 200, [attention(2, 1, 16, 30, conv=2)]),
+    "cap": model(64, 200, [attention(4, 1, 16, 0, conv=1, scale=0.6, softcap=1.5, rot_dims=0)]),
+    "rotation": model(64, 200, [attention(4, 4, 16, 0, rot_dims=8, base=500.0)]),
+    "llama3": model(64, 200, [attention(4, 2, 24, 0, scaling=llama3())]),
+    "llama3_partial": model(64, 200, [attention(3, 1, 32, 0, rot_dims=12, base=300.0, scaling=llama3(9.0, 0.5, 6.0, 60))]),
+    "window": model(64, 200, [attention(4, 2, 16, 24)]),
+    "dense": model(64, 200, [attention(2, 2, 16, 40, mlp=dense(72))]),
+    "latent": model(64, 200, [latent(4, 16, 8, 16, 32)]),
+    "latent_yarn": model(64, 200, [latent(3, 20, 12, 10, 24, scaling=yarn(), mlp=dense(40))]),
+    "lent": model(64, 200, [latent(2, 16, 8, 16, 24, scaling=yarn()), latent(2, 16, 8, 16, 24, scaling=yarn(), kv_from=0)]),
+}
+
+# windows shorter and longer than a page of 64 and none; a lender with two readers whose heads, widths
+# and scales differ from its own, another lender between them, layers with and without a feed-forward
+MIXED = model(64, 200, [
+    attention(4, 2, 16, 37, rot_dims=8, scaling=llama3(), mlp=dense(96)),
+    latent(4, 16, 8, 24, 40, scaling=yarn(), mlp=dense(64)),
+    attention(3, 1, 32, 90, conv=2, scale=0.15, softcap=8.0),
+    latent(2, 24, 8, 16, 40, scale=0.2, scaling=yarn(), kv_from=1),
+    latent(3, 16, 4, 8, 24, base=500.0, mlp=dense(40)),
+    attention(2, 2, 24, 0, conv=4, base=300.0, softcap=0, mlp=dense(48)),
+    latent(5, 12, 8, 20, 40, scale=0.4, scaling=yarn(), kv_from=1, mlp=dense(80)),
+    latent(1, 32, 4, 12, 24, base=500.0, kv_from=4),
+])
+
+# sizes that are no multiples of 16, 8 or 4; one head; a window of one position
+ODD = model(70, 131, [
+    attention(3, 3, 10, 7, conv=7, rot_dims=6, scaling=llama3(3.0, 0.7, 4.0, 50), mlp=dense(33)),
+    latent(3, 9, 6, 5, 17, scaling=yarn(3.0, 50, 4.0, 0.7), mlp=dense(20)),
+    attention(1, 1, 20, 33, conv=1, base=50.0, softcap=4.0),
+    attention(5, 1, 6, 1, conv=2, scale=0.5),
+    latent(1, 13, 6, 21, 17, scale=0.5, scaling=yarn(3.0, 50, 4.0, 0.7), kv_from=1, mlp=dense(7)),
+    attention(3, 1, 13, 50, conv=3, rot_dims=2),
+], eps=1e-6)
+
+# heads of the fast kernels' widths (64, 128, 256), groups of 1, 2, 4 and 8, more than 16 latent heads, a
+# window of one position and one longer than any request
+WIDE = model(128, 300, [
+    attention(4, 2, 64, 48, base=500000.0, scale=0.12, scaling=llama3(16.0, 1.0, 4.0, 128), mlp=dense(256)),
+    latent(4, 64, 32, 64, 96, scale=0.1, scaling=yarn(16.0, 128, 32.0, 1.0)),
+    attention(8, 1, 128, 130, rot_dims=64, scale=0.08, mlp=dense(136)),
+    attention(2, 1, 256, 1, conv=2, rot_dims=64, scale=0.06),
+    latent(18, 32, 32, 32, 96, scale=0.15, scaling=yarn(16.0, 128, 32.0, 1.0), kv_from=1, mlp=dense(64)),
+    attention(4, 1, 64, 5000, conv=4, scale=0.12, softcap=30.0, mlp=dense(128)),
+    attention(2, 2, 128, 100, conv=1, scale=0.08, softcap=0, scaling=llama3()),
+])
+
+# a scale that makes the softmax pick a few keys among those in sight
+SHARP = model(64, 200, [
+    attention(4, 2, 16, 50, conv=2, scale=1.0, softcap=40.0, rot_dims=4),
+    attention(2, 2, 16, 66, scale=0.9, softcap=40.0, rot_dims=4, mlp=dense(32)),
+    latent(2, 16, 4, 16, 24, scale=1.5),
+])
