@@ -114,3 +114,123 @@ SHARP = model(64, 200, [
     attention(2, 2, 16, 66, scale=0.9, softcap=40.0, rot_dims=4, mlp=dense(32)),
     latent(2, 16, 4, 16, 24, scale=1.5),
 ])
+
+REL_TOL = {"float32": 1e-4, "bfloat16": 4e-2}
+BF16_MEDIAN, BF16_ROWS_OVER, BF16_WORST = 2e-2, 0.1, 0.12
+
+
+def prompts(cfg: dict, lengths: Sequence[int], seed: int) -> List[List[int]]:
+    g = torch.Generator().manual_seed(seed)
+    return [torch.randint(0, cfg["vocab"], (n,), generator=g).tolist() for n in lengths]
+
+
+def random_weights(config: dict, seed: int) -> Dict[str, torch.Tensor]:
+    """Random tensors of every name the configuration asks for, rounded to bfloat16 values; biases,
+    taps and gains large enough that leaving one out, or taking another's, shows."""
+    g = torch.Generator().manual_seed(seed)
+    W = config["width"]
+
+    def mat(o, i, s=1.0):
+        return torch.randn((o, i), generator=g) * (s / math.sqrt(i))
+
+    def vec(n, s=0.3, at=1.0):
+        return torch.randn((n,), generator=g) * s + at
+
+    def norm(name):
+        out[name], out[name + ".b"] = vec(W), vec(W, 0.3, 0.0)
+    out: Dict[str, torch.Tensor] = {"embed": torch.randn((config["vocab"], W), generator=g)}
+    for i, layer in enumerate(config["layers"]):
+        m, pre = layer["mixer"], f"l{i}.mix."
+        H, D = m["heads"], m["dim"]
+        norm(f"l{i}.norm1")
+        if layer["type"] == "attention":
+            for name, n in (("q", H * D), ("k", (m.get("kv_heads") or H) * D)):
+                out[pre + name], out[pre + name + ".b"] = mat(n, W), vec(n, 0.4, 0.0)
+                out[pre + name + ".conv"] = torch.randn((n, m["conv"]), generator=g) * 0.6
+                out[pre + name + ".norm"] = vec(n)
+            V = D
+        else:
+            V, R = m["vdim"], m["kv_rank"]
+            out[pre + "q"] = mat(H * (D + m["rot_dim"]), W)
+            if m.get("kv_from") is None:
+                out[pre + "dkv"], out[pre + "dkv.norm"] = mat(R + m["rot_dim"], W), vec(R)
+            out[pre + "uk"], out[pre + "uv"] = mat(H * D, R), mat(H * V, R)
+        out[pre + "g"], out[pre + "o"] = mat(H * V, W, 1.5), mat(W, H * V)
+        if layer.get("mlp"):
+            F, pre = layer["mlp"]["ff"], f"l{i}.mlp."
+            norm(f"l{i}.norm2")
+            out[pre + "gate"], out[pre + "up"], out[pre + "down"] = mat(F, W), mat(F, W), mat(W, F)
+    norm("final.norm")
+    out["head"] = mat(config["vocab"], W, 2.0)
+    return {n: t.to(torch.bfloat16).to(torch.float32) for n, t in out.items()}
+
+
+def plain_logits(cfg: dict, weights: Dict[str, torch.Tensor], tokens: Sequence[int]) -> torch.Tensor:
+    return torch.from_numpy(np.ascontiguousarray(plain.logits(cfg, weights, list(tokens))))
+
+
+def assert_close(got: torch.Tensor, ref: torch.Tensor, dtype: str, what: str) -> None:
+    """Rows of logits against the plain model's: the largest difference as a fraction of the
+    largest plain logit of the compared rows."""
+    got = got.detach().to("cpu", torch.float64)
+    ref = ref.to(torch.float64)
+    assert got.shape == ref.shape, f"{what}: shape {tuple(got.shape)} vs {tuple(ref.shape)}"
+    assert torch.isfinite(got).all(), f"{what}: non-finite logits"
+    scale = ref.abs().max().item()
+    diff = (got - ref).abs().amax(dim=-1)
+    bad = (diff > REL_TOL[dtype] * scale).nonzero()
+    text = (f"{what}: max |diff| {diff.max().item():.3e}, median {diff.median().item():.3e}, "
+            f"{bad.numel()} of {got.shape[0]} rows over {REL_TOL[dtype]:.0e} x max|ref| {scale:.3e}"
+            + (f"; first of them row {int(bad[0])}" if bad.numel() else ""))
+    if dtype == "float32":
+        assert bad.numel() == 0, text
+    elif got.shape[0] < 8:
+        assert diff.max().item() <= BF16_WORST * scale, text
+    else:
+        assert diff.median().item() <= BF16_MEDIAN * scale, text
+        assert bad.numel() <= max(1, BF16_ROWS_OVER * got.shape[0]), text
+        assert diff.max().item() <= BF16_WORST * scale, text
+
+
+def rows_that_differ(a: torch.Tensor, b: torch.Tensor, factor: float = 100.0) -> int:
+    """How many rows of two plain results differ by more than ``factor`` times the 32-bit
+    tolerance: what a test needs to be able to tell the two apart."""
+    scale = a.abs().max().item()
+    return int(((a - b).abs().amax(dim=-1) > factor * REL_TOL["float32"] * scale).sum())
+
+
+def changed(cfg: dict, edit) -> dict:
+    other = copy.deepcopy(cfg)
+    edit(other)
+    return other
+
+
+def random_model(seed: int) -> dict:
+    """A configuration drawn from the design's whole range: both mixers in any order, grouped and
+    ungrouped heads of the fast kernels' widths and of others, windows of any length or none, caps or
+    none, any number of taps, rotations with and without scaling, readers of earlier layers' rows."""
+    r = random.Random(seed)
+    width, vocab = r.choice([64, 96, 128, 100, 36]), r.randrange(90, 300)
+    layers: list = []
+    for i in range(r.randrange(2, 7)):
+        mlp = dense(r.choice([8, 24, 40, 130, 33])) if r.random() < 0.75 else None
+        lenders = [k for k, l in enumerate(layers) if l["type"] == "latent_attention" and "kv_from" not in l["mixer"]]
+        if r.random() < 0.5:
+            kv, dim = r.choice([1, 2, 4]), r.choice([16, 32, 64, 64, 128, 24, 10])
+            layers.append(attention(
+                kv * r.choice([1, 2, 3, 4]), kv, dim, r.choice([0, 1, 5, 16, 37, 64, 100]), conv=r.choice([1, 2, 3, 4, 5, 9]),
+                scale=r.choice([0.1, 0.3]), softcap=r.choice([0, 2.0, 20.0, 50.0]), rot_dims=r.choice([0, 2, dim // 4 * 2, dim]),
+                base=r.choice([100.0, 10000.0, 500000.0]),
+                scaling=r.choice([None, llama3(), llama3(16.0, 1.0, 4.0, 40), llama3(2.0, 2.0, 30.0, 4096)]), mlp=mlp))
+            continue
+        heads, dim, vdim = r.choice([1, 2, 3, 6, 17]), r.choice([16, 32, 64, 10]), r.choice([16, 48, 64, 7])
+        if lenders and r.random() < 0.6:
+            k = r.choice(lenders)
+            m = layers[k]["mixer"]
+            layers.append(latent(heads, dim, m["rot_dim"], vdim, m["kv_rank"], scale=r.choice([0.1, 0.25]), kv_from=k, mlp=mlp))
+            layers[-1]["mixer"]["rot"] = dict(m["rot"])
+        else:
+            layers.append(latent(heads, dim, r.choice([2, 8, 16, 32]), vdim, r.choice([16, 40, 96, 21]), scale=r.choice([0.1, 0.25]),
+                                 base=r.choice([100.0, 10000.0]),
+                                 scaling=r.choice([None, yarn(), yarn(16.0, 40, 4.0, 0.5), yarn(2.0, 4096, 32.0, 1.0)]), mlp=mlp))
+    return model(width, vocab, layers, eps=r.choice([1e-5, 1e-6]))
