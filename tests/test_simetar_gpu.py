@@ -221,3 +221,266 @@ def test_edges_of_windows_with_a_sharp_softmax(page_tokens):
     for k in range(55):
         out = eng.step([(sa, [a[195 + k]]), (sb, [b[40 + k]])], [[0], [0]])
         assert_close(out, torch.stack([ref[195 + k], rb[40 + k]]), dtype, f"two requests, token {k}")
+
+
+ASKS, ASKED = 47, 46
+
+
+def _asking(cfg, seed):
+    """Weights with which token ASKS has token ASKED's key as its query in the last layer: its weight
+    goes to where that token occurs.  Earlier layers add nothing to the stream."""
+    w = random_weights(cfg, seed)
+    last, pre = cfg["layers"][-1], f"l{len(cfg['layers']) - 1}.mix."
+    for i in range(len(cfg["layers"]) - 1):
+        w[f"l{i}.norm1"].zero_()
+        w[f"l{i}.norm1.b"].zero_()
+    asks, asked = w["embed"][ASKS], w["embed"][ASKED]
+    m = last["mixer"]
+    if last["type"] == "attention":
+        for n in ("q", "k"):
+            w[pre + n + ".b"].zero_()
+            w[pre + n + ".conv"].zero_()
+            w[pre + n + ".conv"][:, -1] = 1.0
+            w[pre + n + ".norm"].fill_(1.0)
+        key = w[pre + "k"] @ asked
+        w[pre + "q"] = torch.outer(key, asks) / asks.dot(asks)
+    else:
+        src = "l%d.mix." % m.get("kv_from", len(cfg["layers"]) - 1)
+        c, _ = plain.latent_rows(plain.f64(asked)[None], plain.sub(w, src), dict(m, rot=None), cfg["norm"]["eps"])
+        key = w[pre + "uk"].double() @ torch.from_numpy(c[0])
+        q = torch.zeros_like(w[pre + "q"])
+        q[:m["dim"]] = (torch.outer(key, asks.double()) / asks.double().dot(asks.double())).float()
+        w[pre + "q"] = q
+    return {n: t.to(torch.bfloat16).float() for n, t in w.items()}
+
+
+@pytest.mark.parametrize("mode", ["prompt", "tokens", "portions"])
+@pytest.mark.parametrize("size", [30, 64, 65, 128, 300])
+def test_a_key_just_in_and_just_out_of_sight(size, mode):
+    """The last token asks for another that occurs once.  At size - 1 positions back that is seen;
+    one further it is not; the row's logits differ widely between the two (checked on the plain
+    model first), in a prompt, when the asking token is decoded alone, and at the end of a portion."""
+    cfg = model(32, 50, [attention(1, 1, 16, size, conv=2, scale=1.0, softcap=40.0, rot_dims=0)])
+    w = _asking(cfg, 40)
+    eng = make_engine(cfg, w, "float32")
+    far = max(size + 150, 260)
+    for start, seen in ((far - 1 - (size - 1), True), (far - 1 - size, False)):
+        toks = [3 + (i % 40) for i in range(far)]
+        toks[start], toks[far - 1] = ASKED, ASKS
+        ref = plain_logits(cfg, w, toks)
+        blind = list(toks)
+        blind[start] = 45
+        moved = rows_that_differ(ref[-1:], plain_logits(cfg, w, blind)[-1:], 50.0)
+        assert moved == (1 if seen else 0), (start, seen)
+        sizes = {"prompt": [far], "tokens": [far - 25] + [1] * 25, "portions": [far - 100] + [20] * 5}[mode]
+        assert_close(run_portions(eng, toks, sizes), ref, "float32", f"window {size}, key at {start} ({mode})")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("lent", [False, True])
+def test_a_far_key_of_the_latent_attention(lent, dtype):
+    """One key among several hundred, at the first position, at both sides of page borders and just
+    before the asking token, read from the layer's own rows or from a lender's."""
+    layers = [latent(1, 16, 4, 16, 20, scale=2.0)]
+    if lent:
+        layers = [latent(2, 8, 4, 8, 20), latent(1, 16, 4, 16, 20, scale=2.0, kv_from=0)]
+    cfg = model(32, 50, layers)
+    w = _asking(cfg, 41)
+    eng = make_engine(cfg, w, dtype)
+    for start in (0, 63, 64, 127, 128, 300, 458):
+        toks = [3 + (i % 40) for i in range(460)]
+        toks[start], toks[-1] = ASKED, ASKS
+        ref = plain_logits(cfg, w, toks)
+        blind = list(toks)
+        blind[start] = 45
+        assert rows_that_differ(ref[-1:], plain_logits(cfg, w, blind)[-1:], 500.0) == 1
+        for sizes in ([460], [459, 1], [300, 100, 58, 2], [435] + [1] * 25):
+            assert_close(run_portions(eng, toks, sizes)[-1:], ref[-1:], dtype, f"key at {start}, steps {sizes[:4]}")
+
+
+def test_the_added_one_the_cap_and_the_gate_show():
+    """Plain models without the added one, without the cap, with a norm per head, or without the gate
+    or the slowed-down frequencies give other logits in nearly every row; the engine agrees with the
+    right one, a sequence's first rows (where the added one weighs most) included."""
+    cfg, dtype = model(64, 200, [attention(4, 2, 16, 60, conv=2, scale=0.5, softcap=2.0, rot_dims=6, scaling=llama3())]), "float32"
+    w = random_weights(cfg, seed=26)
+    toks = prompts(cfg, [150], seed=27)[0]
+    ref = plain_logits(cfg, w, toks)
+
+    def differs(name, other):
+        keep = getattr(plain, name)
+        setattr(plain, name, other)
+        try:
+            return rows_that_differ(ref, plain_logits(cfg, w, toks), 10.0)
+        finally:
+            setattr(plain, name, keep)
+    assert differs("weights_beside_one", plain.softmax) > 140
+    assert differs("softcap", lambda s, cap: s) > 130
+    assert differs("sigmoid", lambda z: np.ones_like(z)) > 140
+    assert differs("llama3_frequencies", lambda d, b, s: plain.plain_frequencies(d, b)) > 100
+    norm = plain.rms_norm
+    assert differs("rms_norm", lambda x, g, eps: (norm(x.reshape(len(x), -1, 16), 1.0, eps)).reshape(x.shape) * g) > 140
+    eng = make_engine(cfg, w, dtype)
+    assert_close(run_whole(eng, toks), ref, dtype, "whole prompt")
+    assert_close(run_portions(eng, toks, [1] * 10 + [60, 2] + [1] * 78), ref, dtype, "portions and single tokens")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("dim", [16, 64])
+def test_a_sink_above_all_scores(dim, dtype):
+    """Where every score is far below 0 the added one takes nearly all of the weight (here scores lie
+    near -11): what is left is summed against it in every kernel."""
+    cfg = model(64, 100, [attention(2, 1, dim, 50, conv=1, scale=12.0 / dim, softcap=30.0, rot_dims=0)])
+    w = random_weights(cfg, seed=30)
+    w["l0.mix.q"], w["l0.mix.k"] = 0.3 * w["l0.mix.q"], 0.3 * w["l0.mix.k"]
+    w["l0.mix.q.b"], w["l0.mix.k.b"] = torch.ones(2 * dim), -torch.ones(dim)        # (opposite directions)
+    for n in ("q", "k"):
+        w[f"l0.mix.{n}.conv"].fill_(1.0)
+        w[f"l0.mix.{n}.norm"].fill_(1.0)
+    w["l0.mix.k.conv"].fill_(64.0)        # (values that are large, so that what is left shows)
+    w = {n: t.to(torch.bfloat16).float() for n, t in w.items()}
+    toks = prompts(cfg, [200], seed=31)[0]
+    ref = plain_logits(cfg, w, toks)
+    keep = plain.weights_beside_one
+    plain.weights_beside_one = lambda s: np.exp(s)           # the added one alone
+    try:
+        alone = plain_logits(cfg, w, toks)
+    finally:
+        plain.weights_beside_one = keep
+    assert (alone - ref).abs().max() < 0.2 * ref.abs().max()
+    eng = make_engine(cfg, w, dtype)
+    for sizes in ([200], [100, 40, 60], [190] + [1] * 10):
+        assert_close(run_portions(eng, toks, sizes), ref, dtype, f"heads of {dim}, {sizes[:3]}")
+
+
+def test_lent_rows():
+    """A reader of another layer's rows differs from one that makes its own; lenders are told apart
+    (the plain model with the readers exchanged gives other logits)."""
+    cfg = model(64, 120, [latent(2, 16, 8, 16, 24, scaling=yarn(), mlp=dense(32)), latent(3, 16, 8, 8, 24, scaling=yarn()),
+                          latent(4, 8, 8, 24, 24, scaling=yarn(), kv_from=0), latent(1, 16, 8, 8, 24, scaling=yarn(), kv_from=1),
+                          latent(2, 24, 8, 16, 24, scaling=yarn(), kv_from=0)])
+    w = random_weights(cfg, seed=28)
+    toks = prompts(cfg, [170], seed=29)[0]
+    ref = plain_logits(cfg, w, toks)
+
+    def swap(c):
+        c["layers"][2]["mixer"]["kv_from"], c["layers"][3]["mixer"]["kv_from"] = 1, 0
+    assert rows_that_differ(ref, plain_logits(changed(cfg, swap), w, toks), 50.0) > 160
+    for dtype in DTYPES:
+        eng = make_engine(cfg, w, dtype)
+        assert len(eng.cache.groups) == 1 and len(eng.cache.groups[0].entries) == 2, "readers keep no rows of their own"
+        for sizes in ([170], [100, 2, 30, 20] + [1] * 18, [1] * 40 + [130]):
+            assert_close(run_portions(eng, toks, sizes), ref, dtype, f"portions {sizes[:5]}")
+
+
+def test_the_convolutions_reach():
+    """The last taps - 1 projected rows of a sequence are carried from step to step in every attention
+    layer: a plain model that forgets them differs in the rows behind."""
+    def taps(c):
+        for layer in c["layers"]:
+            if layer["type"] == "attention":
+                layer["mixer"]["conv"] = 6
+    cfg = changed(MIXED, taps)
+    w = random_weights(cfg, seed=28)
+    toks = prompts(cfg, [60], seed=29)[0]
+    ref = plain_logits(cfg, w, toks)
+    silent = {n: (torch.cat([torch.zeros_like(t[:, :-1]), t[:, -1:]], dim=1) if n.endswith(".conv") else t) for n, t in w.items()}
+    assert rows_that_differ(ref[1:], plain_logits(cfg, silent, toks)[1:], 50.0) == 59
+    for dtype in DTYPES:
+        eng = make_engine(cfg, w, dtype)
+        for sizes in ([30, 1, 1, 1, 1, 1, 1, 24], [2] * 30, [3, 4, 5, 6, 7, 1, 34], [1] * 60):
+            assert_close(run_portions(eng, toks, sizes), ref, dtype, f"portions {sizes[:6]}")
+
+
+def test_first_tokens_of_a_sequence():
+    cfg, dtype = MIXED, "float32"
+    w = random_weights(cfg, seed=24)
+    toks = prompts(cfg, [40], seed=25)[0]
+    ref = plain_logits(cfg, w, toks)
+    eng = make_engine(cfg, w, dtype, max_slots=1)
+    assert_close(run_portions(eng, toks, [1, 1, 1, 2, 2, 5]), ref, dtype, "first tokens one by one")
+    assert_close(run_portions(eng, toks[::-1], [3, 1]), plain_logits(cfg, w, toks[::-1]), dtype, "the slot again")
+    assert_close(run_whole(eng, toks[:1]), ref[:1], dtype, "one token alone")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["odd", "wide"])
+def test_other_sizes(name, dtype):
+    """(wide: heads of the fast kernels; bfloat16 prompts of more than 128 tokens take the tcgen05
+    kernel, shorter ones the mma.sync kernel, portions of 32 rows and more the prompt kernel over
+    gathered keys, single rows the decode kernel)"""
+    cfg = {"odd": ODD, "wide": WIDE}[name]
+    w = random_weights(cfg, 17)
+    eng = make_engine(cfg, w, dtype, max_continuation=96)
+    toks = prompts(cfg, [420], seed=18)[0]
+    ref = plain_logits(cfg, w, toks)
+    assert_close(run_whole(eng, toks), ref, dtype, f"{name}: whole prompt")
+    assert_close(run_whole(eng, toks[:100]), ref[:100], dtype, f"{name}: a short prompt")
+    assert_close(run_portions(eng, toks, [33, 2, 60, 64, 90, 50] + [1] * 41), ref, dtype, f"{name}: portions and tokens")
+    assert_close(run_portions(eng, toks, [260, 90, 40]), ref, dtype, f"{name}: large portions")
+    a, b = toks[:250], prompts(cfg, [60], seed=19)[0]
+    rb = plain_logits(cfg, w, b)
+    sa, sb = eng.new_sequence(), eng.new_sequence()
+    out = eng.step([(sa, a[:240]), (sb, b[:50])], [all_rows(240), all_rows(50)])
+    assert_close(out, torch.cat([ref[:240], rb[:50]]), dtype, f"{name}: two prompts")
+    for k in range(10):
+        out = eng.step([(sa, [a[240 + k]]), (sb, [b[50 + k]])], [[0], [0]])
+        assert_close(out, torch.stack([ref[240 + k], rb[50 + k]]), dtype, f"{name}: two requests, token {k}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("seed", list(range(16)))
+def test_configurations_drawn_at_random(seed, dtype):
+    """Any of the sizes and constants: a prompt, portions down to two tokens with single tokens
+    behind them, and two unequal requests together."""
+    cfg = random_model(seed)
+    w = random_weights(cfg, 70 + seed)
+    eng = make_engine(cfg, w, dtype)
+    toks = prompts(cfg, [190], seed=seed)[0]
+    ref = plain_logits(cfg, w, toks)
+    assert_close(run_whole(eng, toks), ref, dtype, f"drawn model {seed}: whole prompt")
+    assert_close(run_portions(eng, toks, [70, 2, 30, 18] + [1] * 70), ref, dtype, f"drawn model {seed}: portions and tokens")
+    a, b = toks[:120], prompts(cfg, [60], seed=seed + 100)[0]
+    rb = plain_logits(cfg, w, b)
+    sa, sb = eng.new_sequence(), eng.new_sequence()
+    out = eng.step([(sa, a[:101]), (sb, b[:33])], [all_rows(101), all_rows(33)])
+    assert_close(out, torch.cat([ref[:101], rb[:33]]), dtype, f"drawn model {seed}: two prompts")
+    for k in range(19):
+        out = eng.step([(sa, [a[101 + k]]), (sb, [b[33 + k]])], [[0], [0]])
+        assert_close(out, torch.stack([ref[101 + k], rb[33 + k]]), dtype, f"drawn model {seed}: two requests, token {k}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_recorded_steps_of_many_rows(dtype):
+    """48 requests decoded together: their single-token steps are recorded and replayed."""
+    cfg = model(64, 120, [attention(2, 1, 64, 10, mlp=dense(24)), latent(3, 16, 8, 16, 24, scaling=yarn()),
+                          attention(2, 1, 16, 20, conv=2), latent(2, 16, 8, 32, 24, scaling=yarn(), kv_from=1, mlp=dense(40))])
+    w = random_weights(cfg, 52)
+    eng = make_engine(cfg, w, dtype, max_tokens=8192, max_slots=48)
+    reqs = prompts(cfg, [19 + (i * 7) % 23 for i in range(48)], seed=53)
+    refs = [plain_logits(cfg, w, t) for t in reqs]
+    slots = [eng.new_sequence() for _ in reqs]
+    eng.step([(s, t[:4]) for s, t in zip(slots, reqs)], [[3]] * 48)
+    for k in range(4, 19):
+        out = eng.step([(s, [t[k]]) for s, t in zip(slots, reqs)], [[0]] * 48)
+        assert_close(out, torch.stack([r[k] for r in refs]), dtype, f"48 requests, token {k}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_recorded_prompts(dtype):
+    """Steps of prompts with one wanted row each are recorded at the second of a shape and replayed
+    for others, filled up with rows of no sequence (a reader of another layer's rows takes them as
+    that layer has just made them); the tokens that follow continue from them."""
+    for cfg in (MIXED, WIDE):
+        w = random_weights(cfg, 54)
+        eng = make_engine(cfg, w, dtype)
+        assert eng.model.captures_prompts
+        for seed, n in ((1, 100), (2, 97), (3, 120), (4, 66), (5, 200), (6, 203), (7, 230)):
+            toks = prompts(cfg, [n], seed=seed)[0]
+            ref = plain_logits(cfg, w, toks)
+            s = eng.new_sequence()
+            assert_close(eng.step([(s, toks[:-6])]), ref[-7:-6], dtype, f"prompt of {n - 6}")
+            for k in range(6):
+                assert_close(eng.step([(s, [toks[n - 6 + k]])]), ref[n - 6 + k:n - 5 + k], dtype, f"prompt {n}, token {k}")
+            eng.end_sequence(s)
+        assert any(g.graph is not None for g in eng._prompt_graphs.values())
