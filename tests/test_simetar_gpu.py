@@ -681,3 +681,207 @@ def test_gate_per_element(heads, vd, pad, dtype):
         native.element_gate(o, gate, y, heads, vd)
         want = o[:, :, :vd].double().reshape(R, -1) * torch.sigmoid(gate.double())
         assert (y.double() - want).abs().max() <= (1e-6 if dtype == torch.float32 else 1e-2) * want.abs().max()
+
+
+def _capped_reference(q, k, v, scale, cap, window, one):
+    """64-bit: q[T, H, d], k, v[T, G, d] -> [T, H, d]."""
+    T, H, _ = q.shape
+    G = k.shape[1]
+    out = np.zeros(q.shape)
+    qd, kd, vd = plain.f64(q), plain.f64(k), plain.f64(v)
+    for t in range(T):
+        lo = plain.first_visible(t, window)
+        for a in range(H):
+            s = plain.softcap(kd[lo:t + 1, a // (H // G)] @ qd[t, a] * scale, cap)
+            out[t, a] = (plain.weights_beside_one if one else plain.softmax)(s) @ vd[lo:t + 1, a // (H // G)]
+    return out
+
+
+@pytest.mark.parametrize("cap, one", [(20.0, True), (3.0, True), (20.0, False), (0.0, True)])
+@pytest.mark.parametrize("heads, kv, hd, window, lens", [
+    (4, 2, 128, 96, [398, 23, 97]), (4, 4, 64, 0, [300, 5, 64, 131]), (2, 1, 256, 200, [500, 130]), (8, 2, 64, 70, [260, 40])])
+def test_prompt_kernels_with_a_cap_and_a_sink(heads, kv, hd, window, lens, cap, one):
+    """The tcgen05 prompt kernel (as a grid and as a balanced list; then the last rows of every
+    sequence with the rows before them as keys only) and the mma.sync one against the 64-bit
+    softmax; with the closer tanh the result is nearer to it than with the hardware's."""
+    from strata_inference_b200.kernels import native
+    g = torch.Generator().manual_seed(heads + hd + window)
+    scale = 3.0 / math.sqrt(hd)
+    rows, refs, row0, at = [], [], [], 0
+    for T in lens:
+        q = torch.randn((T, heads, hd), generator=g).to(torch.bfloat16)
+        k, v = (torch.randn((T, kv, hd), generator=g).to(torch.bfloat16) for _ in range(2))
+        refs.append(_capped_reference(q, k, v, scale, cap, window, one))
+        rows.append(torch.cat([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1)], dim=1))
+        row0.append(at)
+        at += T
+    packed, sink = torch.cat(rows).contiguous().cuda(), torch.zeros(heads, device="cuda") if one else None
+    ref = np.concatenate(refs).reshape(at, -1)
+    errors = {}
+
+    def check(out, what, close, start=None):
+        got = out.float().cpu().numpy()
+        for b, T in enumerate(lens):
+            lo = row0[b] + (start[b] if start else 0)
+            err = np.abs(got[lo:row0[b] + T] - ref[lo:row0[b] + T])
+            errors.setdefault((what, close), []).append(float(np.sqrt((err ** 2).mean())))
+            assert err.max() <= 2e-2 * np.abs(ref).max(), f"{what}, sequence {b}: {err.max():.3e}"
+
+    def tc(host, close, start=None):
+        out = torch.full((at, heads * hd), float("nan"), dtype=torch.bfloat16, device="cuda")
+        if host:
+            items, need, n_tickets = native.attention_prefill_tc_plan(lens, heads, kv, hd, window, start)
+            assert items > 0
+        else:
+            need, n_tickets = native.attention_prefill_tc_split(len(lens), max(lens), heads, kv, hd)
+        native.attention_prefill_tc(packed, out, i32(row0), i32(lens), len(lens), max(lens), heads, kv, hd, scale, cap, window,
+                                    torch.empty(max(need, 16), dtype=torch.uint8, device="cuda"),
+                                    torch.zeros(max(n_tickets, 1), dtype=torch.int32, device="cuda"),
+                                    lens if host else None, i32(start) if start else None, start if host else None,
+                                    sink=sink, close_cap=close)
+        assert native.attention_prefill_tc_error() == 0
+        check(out, "tcgen05", close, start)
+    for close in (False, True):
+        if native.attention_prefill_tc_supports(heads, kv, hd, (heads + 2 * kv) * hd):
+            for host in (False, True):
+                tc(host, close)
+                tc(host, close, [max(0, T - 40) for T in lens])
+        if native.attention_prefill_supports(heads, kv, hd):
+            out = torch.full((at, heads * hd), float("nan"), dtype=torch.bfloat16, device="cuda")
+            native.attention_prefill(packed, out, i32(row0), i32(lens), len(lens), max(lens), heads, kv, hd, scale, cap, window,
+                                     sink=sink, close_cap=close)
+            check(out, "mma.sync", close)
+    assert errors
+    for what in {k for k, _ in errors}:
+        if cap >= 20.0:
+            assert np.mean(errors[what, True]) <= np.mean(errors[what, False]), errors
+
+
+@pytest.mark.parametrize("style", [0, 1])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_latent_rows_in_both_rotations(style, dtype):
+    """latent_prepare and latent_expand with half-split and neighbouring pairs and a magnitude; query
+    rows alone for a layer that reads another's rows."""
+    from strata_inference_b200.kernels import native
+    heads, qd, rd, vd, rank, kw, hw, R = 3, 16, 12, 24, 20, 32, 64, 6
+    g = torch.Generator().manual_seed(3)
+    proj = torch.randn((R, heads * (qd + rd) + rank + rd), generator=g).to(dtype).cuda()
+    lat = torch.randn((heads, R, rank), generator=g).to(dtype).cuda()
+    gain, freqs, mag = torch.rand(rank, generator=g) + 0.5, torch.rand(4, generator=g), 1.25
+    ctx = _Step([(0, 5, R)])
+    code = native.ROPE_HALF_SPLIT if style == 0 else native.ROPE_INTERLEAVED
+    pair = (lambda i: (i, i + 4)) if style == 0 else (lambda i: (2 * i, 2 * i + 1))
+    shift = lambda t: plain.rotate(np.concatenate([np.zeros((5,) + t.shape[1:]), t]), 8, plain.f64(freqs), pair, mag)[5:]  # noqa: E731
+    p = plain.f64(proj)
+    heads_of = p[:, :heads * (qd + rd)].reshape(R, heads, qd + rd)
+    want_q = np.zeros((R, heads, kw))
+    want_q[:, :, :rank], want_q[:, :, rank:rank + rd] = plain.f64(lat).transpose(1, 0, 2), shift(heads_of[:, :, qd:])
+    want_k = np.zeros((R, kw))
+    down = p[:, heads * (qd + rd):]
+    want_k[:, :rank] = plain.rms_norm(down[:, :rank], plain.f64(gain), 1e-6)
+    want_k[:, rank:rank + rd] = shift(down[:, None, rank:])[:, 0]
+    tol = 2e-5 if dtype == torch.float32 else 2e-2
+    for own in (True, False):
+        q_rows = torch.full((R, heads * kw), float("nan"), dtype=dtype, device="cuda")
+        k_rows = torch.full((R, kw), float("nan"), dtype=dtype, device="cuda") if own else None
+        src = proj if own else proj[:, :heads * (qd + rd)].contiguous()
+        native.latent_prepare(src, lat, q_rows, k_rows, _dev(gain) if own else None, 1e-6, _dev(freqs), 8, ctx, None, None, 0, 0,
+                              heads, qd, rd, rank, kw, style=code, magnitude=mag)
+        assert np.abs(plain.f64(q_rows).reshape(R, heads, kw) - want_q).max() <= tol
+        if own:
+            assert np.abs(plain.f64(k_rows) - want_k).max() <= tol * np.abs(want_k).max()
+            kept = k_rows
+    kh, vh = (torch.randn((R, heads * n), generator=g).to(dtype).cuda() for n in (qd, vd))
+    qkv = torch.empty((R, 3 * heads * hw), dtype=dtype, device="cuda")
+    native.latent_expand(proj, kept, kh, vh, qkv, _dev(freqs), 8, ctx.row_pos, heads, qd, rd, vd, rank, kw, hw, style=code,
+                         magnitude=mag)
+    want = np.zeros((R, 3, heads, hw))
+    want[:, 0, :, :qd], want[:, 0, :, qd:qd + rd] = heads_of[:, :, :qd], shift(heads_of[:, :, qd:])
+    want[:, 1, :, :qd], want[:, 1, :, qd:qd + rd] = plain.f64(kh).reshape(R, heads, qd), want_k[:, None, rank:rank + rd]
+    want[:, 2, :, :vd] = plain.f64(vh).reshape(R, heads, vd)
+    assert np.abs(plain.f64(qkv).reshape(want.shape) - want).max() <= tol * np.abs(want).max()
+
+
+# --------------------------------------------------------------------------
+# the engine's own entry points
+
+
+def _write_model(path, cfg, weights):
+    from strata_inference_b200.weights.safetensors_io import write_safetensors
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(path, "model.safetensors"),
+                      {n: t.to(torch.bfloat16) for n, t in weights.items()})
+    return path
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_greedy_generation_through_the_generation_engine(tmp_path, dtype):
+    """Several prompts through GenerationEngine.generate (its scheduler batches them): every
+    chosen token is the plain model's best, or so near it that rounding decides, given the run's
+    own history."""
+    from strata_inference_b200 import GenerationConfig, GenerationEngine, SamplingConfig
+    cfg = MIXED
+    w = random_weights(cfg, 21)
+    path = _write_model(str(tmp_path / "m"), cfg, w)
+    engine = GenerationEngine.from_dir(path, dtype=dtype, max_tokens=1024)
+    reqs = prompts(cfg, [5, 47, 90, 13], seed=22)
+    outs = engine.generate(reqs, GenerationConfig(max_tokens=40, sampling=SamplingConfig(temperature=0.0)))
+    tol = {"float32": 1e-4, "bfloat16": 0.15}[dtype]
+    far = total = 0
+    for p, o in zip(reqs, outs):
+        assert len(o.token_ids) == 40 and o.stop_reason == "max_tokens"
+        ref = plain_logits(cfg, w, list(p) + list(o.token_ids))
+        for k, tok in enumerate(o.token_ids):
+            row = ref[len(p) + k - 1]
+            far += (row.max() - row[tok]).item() > tol * row.abs().max().item()
+            total += 1
+    assert far == 0, f"{far} of {total} tokens lie far below the best"
+
+
+def test_trace_replay_of_a_model_folder(tmp_path):
+    """bin/trace_run on a folder: prompts of unequal length in one step, then single tokens
+    together, the shorter request ending first; the files hold the wanted rows' logits."""
+    cfg = MIXED
+    w = random_weights(cfg, seed=23)
+    path = _write_model(str(tmp_path / "m"), cfg, w)
+    a, b = prompts(cfg, [90, 45], seed=24)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:50], "want": [0, 39, 40, 49]},
+                                     {"id": "b", "tokens": b[:42], "want": [41]}], "end": []}]
+    for k in range(40):
+        entries = [{"id": "a", "tokens": [a[50 + k]], "want": [0]}]
+        if k < 3:
+            entries.append({"id": "b", "tokens": [b[42 + k]], "want": [0] if k != 1 else []})
+        steps.append({"step": k + 1, "entries": entries, "end": ["b"] if k == 2 else []})
+    out_dir = str(tmp_path / "out")
+    proc = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", path, "--dtype", "float32",
+                           "--out", out_dir, "--max-tokens", "256"], input="\n".join(json.dumps(s) for s in steps) + "\n",
+                          capture_output=True, text=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done")] == [f"done {k}" for k in range(41)]
+    ra, rb = plain_logits(cfg, w, a), plain_logits(cfg, w, b)
+    got = torch.from_numpy(np.fromfile(os.path.join(out_dir, "0.f32"), dtype="<f4").reshape(5, -1))
+    assert_close(got, torch.stack([ra[0], ra[39], ra[40], ra[49], rb[41]]), "float32", "the prompts' rows")
+    for k in range(40):
+        want = [ra[50 + k]] + ([rb[42 + k]] if k < 3 and k != 1 else [])
+        got = torch.from_numpy(np.fromfile(os.path.join(out_dir, f"{k + 1}.f32"), dtype="<f4").reshape(len(want), -1))
+        assert_close(got, torch.stack(want), "float32", f"step {k + 1}")
+
+
+def test_command_line_generates_from_a_model_folder(tmp_path):
+    cfg = ALONE["lent"]
+    w = random_weights(cfg, seed=2)
+    path = _write_model(str(tmp_path / "m"), cfg, w)
+    prompt = prompts(cfg, [9], seed=3)[0]
+    p = subprocess.run([sys.executable, "-m", "strata_inference_b200.cli", "-m", path, "--token-ids",
+                        ",".join(map(str, prompt)), "-n", "6", "--temp", "0", "--output-format", "json",
+                        "--dtype", "float32"], capture_output=True, text=True, timeout=900, cwd=ROOT)
+    assert p.returncode == 0, p.stderr[-2000:]
+    out = json.loads(p.stdout)
+    tokens = out["output_token_ids"]
+    assert len(tokens) == 6 and out["stop_reason"] == "max_tokens"
+    logits = plain_logits(cfg, w, list(prompt) + list(tokens))
+    for k, tok in enumerate(tokens):
+        row = logits[len(prompt) + k - 1]
+        assert (row.max() - row[tok]).item() <= 1e-4 * row.abs().max().item()
