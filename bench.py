@@ -560,6 +560,27 @@ def kerolorn_config(size):
             "canon": {"taps": 4}, "logit_scale": 0.5, "layers": [layer] * n_layers}
 
 
+def simetar_config(size):
+    """Simetar at these sizes: attention over a window of 4 096 positions (as Gemma2's) with a cap of 50,
+    a convolution of 4 taps on q and k, every head width rotated; latent attention with Vavupel's latent
+    of 448 + 64 rotated columns and values of 128; in turn, every second latent layer a reader of
+    the one before; the other models' feed-forward width."""
+    width, ff, heads, kv, hd, vocab, n_layers = KARUPEL_SIZES[size]
+    mlp = {"kind": "dense", "ff": ff}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "conv": 4, "scale": hd ** -0.5, "softcap": 50.0,
+        "mask": {"size": 4096},
+        "rot": {"base": 500000.0, "dims": hd, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    lat = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 448, "scale": 192 ** -0.5,
+           "rot": {"base": 10000.0, "dims": 64,
+                   "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    layers = []
+    for i in range(n_layers):
+        reader = dict(lat, kv_from=i - 2) if i % 4 == 3 else lat
+        layers.append({"type": "latent_attention", "mlp": mlp, "mixer": reader} if i % 2 else att)
+    return {"architecture": "Simetar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def gemma2_config_like(size):
     width, ff, heads, kv, hd, vocab, n_layers = KARUPEL_SIZES[size]
     cfg = baseline_config()
@@ -589,7 +610,7 @@ def unread_expert_bytes(engine, rows):
 
 def spread_rows(engine):
     """Norms of a randomly drawn model as the identity's neighbour: RMS gains and heads' factors of 1,
-    Dynamic Tanh norms with weight 1, b 0 and alpha 1, and routers' corrections of 0.  Drawn like
+    Dynamic Tanh norms with weight 1, b 0 and alpha 1, layer norms with weight 1 and b 0, and routers' corrections of 0.  Drawn like
     other norm weights (around 0, spread 0.1) Dynamic Tanh turns every row into nearly the same
     vector b, and corrections outweigh the scores: a router then sends all rows of a step to the
     same experts, and the experts' work would be that of the worst imbalance there is."""
@@ -601,9 +622,15 @@ def spread_rows(engine):
             blk.feed_forward.b_router.zero_()
         if getattr(blk.mixer, "temp", None) is not None:
             blk.mixer.temp.fill_(1.0)
+        for gains in (getattr(blk.mixer, "q_gain", None), getattr(blk.mixer, "k_gain", None)):
+            if gains is not None:
+                gains.fill_(1.0)
     for n in norms:
         if n is not None and getattr(n, "gain", None) is not None:
             n.gain.fill_(1.0)
+        if n is not None and hasattr(n, "b") and not hasattr(n, "alpha"):      # (a layer norm)
+            n.weight.fill_(1.0)
+            n.b.zero_()
         if n is not None and hasattr(n, "alpha") and hasattr(n, "b"):
             n.weight.fill_(1.0)
             n.b.zero_()
@@ -632,7 +659,7 @@ def run_karupel(args, pair=None, title="Karupel beside Gemma2"):
                                                max_slots=max(batches))
             engine = gen.engine
             randomize_pools(engine)
-            if name in ("besorax", "kerolorn"):
+            if name in ("besorax", "kerolorn", "simetar"):
                 spread_rows(engine)
             weight_bytes = engine.model.weight_bytes()
             row = {"weights_gb": round(weight_bytes / 1e9, 2)}
@@ -714,8 +741,12 @@ def main():
     ap.add_argument("--kerolorn", action="store_true",
                     help="Kerolorn beside Besorax at equal layer sizes: a prompt step and single-token "
                          "steps (with --kernels the per-kernel tables of both)")
+    ap.add_argument("--simetar", action="store_true",
+                    help="Simetar beside Gemma2 (its windowed, capped attention and feed-forward) and Vavupel "
+                         "(its latent attention) at equal layer sizes: a prompt step and single-token steps "
+                         "(with --kernels the per-kernel tables of all three)")
     ap.add_argument("--size", default="", choices=[""] + sorted(KARUPEL_SIZES),
-                    help="with --karupel, --vavupel, --gegorax, --besorax or --kerolorn: one of the sizes (default: all)")
+                    help="with --karupel, --vavupel, --gegorax, --besorax, --kerolorn or --simetar: one of the sizes (default: all)")
     ap.add_argument("--shape", default="2b", choices=sorted(SHAPES),
                     help="layer sizes: the 2B shape (the recorded line) or the 9B / 27B shapes")
     args = ap.parse_args()
@@ -742,6 +773,9 @@ def main():
     if args.kerolorn:
         return run_karupel(args, (("kerolorn", kerolorn_config), ("besorax", besorax_config)),
                            "Kerolorn beside Besorax")
+    if args.simetar:
+        return run_karupel(args, (("simetar", simetar_config), ("gemma2", gemma2_config_like),
+                                  ("vavupel", vavupel_config)), "Simetar beside Gemma2 and Vavupel")
     if args.karupel:
         return run_karupel(args)
     if args.kernels:

@@ -166,152 +166,169 @@ __device__ __forceinline__ uint4 pack8(const float (&x)[8]) {
 
 // The common case in 16-byte accesses: bfloat16, heads of a multiple of 8 that need no filling
 // up, neighbouring pairs.  A thread owns 8 neighbouring channels of q, k or v and takes RUN
-// neighbouring rows one after the other, the TAPS - 1 rows before them in registers; the rows'
-// cosines and sines are taken once per block, ahead of the wait for the projection (positions
-// and tables are written by the host before the step).  A row costs one barrier.
-// TAPS 0: no convolution.
-template <int TAPS, int RUN, int THREADS>
-__global__ void __launch_bounds__(THREADS) row_prepare_bf16_kernel(RowPrepareArgs p) {
-    constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
+// neighbouring rows at once.  A run inside one sequence whose first row has all its predecessors in
+// this step asks for its rows together and convolves them tap by tap from registers; in any other
+// run each row fetches what lies before it from the step's rows or from the state.  The rows'
+// sums cross the block with one barrier.  Where a row is stored, and its cosines and sines, are
+// worked out once per block ahead of the wait for the projection (positions and tables are
+// written by the host before the step).  TAPS 0: no convolution.
+template <int TAPS, int RUN, int THREADS, int BLOCKS>
+__global__ void __launch_bounds__(THREADS, BLOCKS) row_prepare_bf16_kernel(RowPrepareArgs p) {
+    constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;          // rows before its own that a row reads
     extern __shared__ float2 turns[];          // [RUN][rot / 2]
-    __shared__ float2 sums[2][32];
+    __shared__ float2 sums[RUN][32];
+    __shared__ long long cells[RUN];           // the rows' cells of kv head 0, or -1
+    __shared__ int slots[RUN], backs[RUN], seqs[RUN];
     pdl_trigger();
     const int nq = p.n_heads * p.kd, nk = p.n_kv * p.kd, C = nq + nk;
     const int units = p.n_heads + 2 * p.n_kv;
     const int c = 8 * threadIdx.x;             // the thread's first channel of the projected row
     const bool live = c < C + (p.values_from_keys ? 0 : nk);
     const bool is_q = c < nq, is_v = c >= C;   // (v channels of their own are passed on)
-    const int r0 = blockIdx.x * RUN, r1 = min(r0 + RUN, p.rows);
+    const int r0 = blockIdx.x * RUN, n_rows = min(RUN, p.rows - r0);
     const int half = p.inv_freq ? p.rot / 2 : 0;
-    for (int i = threadIdx.x; i < (r1 - r0) * half; i += blockDim.x) {
+    if ((int)threadIdx.x < n_rows) {
+        const int r = r0 + threadIdx.x, pos = p.row_pos[r], b = p.row_seq[r], slot = p.seq_slot[b];
+        cells[threadIdx.x] = cell_of_row(p, pos, b, slot);
+        slots[threadIdx.x] = slot;
+        backs[threadIdx.x] = pos - p.seq_start[b];
+        seqs[threadIdx.x] = b;
+    }
+    for (int i = threadIdx.x; i < n_rows * half; i += blockDim.x) {
         const int k = i / half;
         const float ang = (float)p.row_pos[r0 + k] * p.inv_freq[i - k * half];
         turns[i] = make_float2(cosf(ang) * p.magnitude, sinf(ang) * p.magnitude);
     }
-    float bias[8], gain[8], w[TAPS > 0 ? TAPS : 1][8];
+    float bias[8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) { bias[e] = 0.f; gain[e] = 1.f; }
-    if (live) {
-        if (p.bias) load8(p.bias + c, bias);
-        if (p.q_gain && !is_v) load8(is_q ? p.q_gain + c : p.k_gain + (c - nq), gain);
-        if (TAPS > 0 && !is_v) {
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) load8(p.conv + (size_t)j * C + c, w[j]);
-        }
-    }
-    const int d0 = c % p.kd;                   // the thread's place in its head
-    const bool rotates = !is_v && d0 < 2 * half;
-    // where the thread's 8 values go in a pool behind the row's cell
-    const size_t head_at = (size_t)((is_v ? c - C : c - nq) / p.kd) * p.page_tokens * p.pad + d0;
+    for (int e = 0; e < 8; ++e) bias[e] = 0.f;
+    if (live && p.bias) load8(p.bias + c, bias);
     __syncthreads();
+    const bool conv = TAPS > 0 && live && !is_v;
+    const bool together = n_rows == RUN && seqs[RUN - 1] == seqs[0] && backs[0] >= BACK;
     pdl_wait();
-    const __nv_bfloat16* proj = (const __nv_bfloat16*)p.proj + c;
-    uint4 raw[RUN];                            // every row is asked for before the first is worked on
+    const __nv_bfloat16* proj = (const __nv_bfloat16*)p.proj + (size_t)r0 * p.proj_stride + c;
+    auto fetch = [&](int row) {                // `row`: from the run's first
+        return *reinterpret_cast<const uint4*>(proj + (long long)row * p.proj_stride);
+    };
+    auto input = [&](const uint4& raw, float (&u)[8]) {
+        unpack8(raw, u);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) u[e] += bias[e];
+    };
+    float acc[RUN][8];
 #pragma unroll
     for (int k = 0; k < RUN; ++k)
-        raw[k] = live && r0 + k < r1 ? *reinterpret_cast<const uint4*>(proj + (size_t)(r0 + k) * p.proj_stride)
-                                     : make_uint4(0, 0, 0, 0);
-    float past[H][8];                          // past[d - 1]: the input d positions back
-    int before = -1;                           // the sequence of the row before
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[k][e] = 0.f;
+    if (conv && together && RUN > 1) {
+        uint4 raw[RUN + BACK];
+#pragma unroll
+        for (int k = 0; k < RUN + BACK; ++k) raw[k] = fetch(k - BACK);
+#pragma unroll
+        for (int j = TAPS - 1; j >= 0; --j) {
+            float w[8];
+            load8(p.conv + (size_t)j * C + c, w);
+#pragma unroll
+            for (int k = 0; k < RUN; ++k) {
+                float u[8];
+                input(raw[k + j], u);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[k][e] += w[e] * u[e];
+            }
+        }
+    } else if (conv) {
+#pragma unroll
+        for (int k = 0; k < RUN; ++k) {
+            if (k >= n_rows) break;
+            float u[BACK + 1][8];              // u[d]: the input d positions back
+            input(fetch(k), u[0]);
+            float* hist = BACK > 0 && slots[k] >= 0 ? p.state + (size_t)slots[k] * p.state_stride + c : nullptr;
+#pragma unroll
+            for (int d = 1; d <= BACK; ++d) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) u[d][e] = 0.f;
+                if (d <= backs[k]) input(fetch(k - d), u[d]);
+                else if (hist) load8(hist + (size_t)(BACK + backs[k] - d) * C, u[d]);
+            }
+#pragma unroll
+            for (int d = 0; d <= BACK; ++d) {
+                float w[8];
+                load8(p.conv + (size_t)(TAPS > 0 ? TAPS - 1 - d : 0) * C + c, w);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[k][e] += w[e] * u[d][e];
+            }
+            if (p.single && hist) {            // one position on
+#pragma unroll
+                for (int d = 0; d < BACK; ++d) store8(hist + (size_t)(BACK - 1 - d) * C, u[d]);
+            }
+        }
+    } else if (live) {
+#pragma unroll
+        for (int k = 0; k < RUN; ++k)
+            if (k < n_rows) input(fetch(k), acc[k]);
+    }
+    __nv_bfloat16* dst = (__nv_bfloat16*)p.qkv + (size_t)r0 * units * p.pad + c;
+    const int d0 = c % p.kd;                   // the thread's place in its head
+    // where the thread's 8 values go in a pool behind a row's cell
+    const size_t head_at = (size_t)((is_v ? c - C : c - nq) / p.kd) * p.page_tokens * p.pad + d0;
+    if (live && (is_v || (!is_q && p.values_from_keys))) {
+#pragma unroll
+        for (int k = 0; k < RUN; ++k) {
+            if (k >= n_rows) break;
+            const uint4 v = pack8(acc[k]);
+            *reinterpret_cast<uint4*>(dst + (size_t)k * units * p.pad + (is_v ? 0 : nk)) = v;
+            if (cells[k] >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.v_pool + cells[k] + head_at) = v;
+        }
+    }
+    const int lane = threadIdx.x & 31, n_warps = (blockDim.x + 31) >> 5;
+    float gain[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) gain[e] = 1.f;
+    if (p.q_gain) {
+        // (a warp of q channels alone, or of others alone, sums one number a row)
+        const bool any_q = __any_sync(0xffffffffu, is_q), any_k = __any_sync(0xffffffffu, !is_q);
+#pragma unroll
+        for (int k = 0; k < RUN; ++k) {
+            float t = 0.f;
+            if (live && !is_v) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) t += acc[k][e] * acc[k][e];
+            }
+            float2 s = make_float2(0.f, 0.f);
+            if (any_q) s.x = warp_sum(is_q ? t : 0.f);
+            if (any_k) s.y = warp_sum(is_q ? 0.f : t);
+            if (lane == 0) sums[k][threadIdx.x >> 5] = s;
+        }
+        if (live && !is_v) load8(is_q ? p.q_gain + c : p.k_gain + (c - nq), gain);
+        __syncthreads();
+    }
+    if (is_v || !live) return;                 // (neither a barrier nor a shuffle is left)
+    const bool rotates = d0 < 2 * half;
 #pragma unroll
     for (int k = 0; k < RUN; ++k) {
-        const int r = r0 + k;
-        if (r >= r1) break;                    // (the same for the whole block)
-        const int b = p.row_seq[r], slot = p.seq_slot[b], pos = p.row_pos[r];
-        const long long cell = is_q ? -1 : cell_of_row(p, pos, b, slot);
-        float x[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = 0.f;
-        if (live) {
-            unpack8(raw[k], x);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] += bias[e];
-        }
-        float* hist = nullptr;
-        if (TAPS > 0 && live && !is_v) {
-            if (TAPS > 1) {
-                hist = slot >= 0 ? p.state + (size_t)slot * p.state_stride + c : nullptr;
-                if (b != before) {             // the run's first row of a sequence
-                    const int back = pos - p.seq_start[b];
-#pragma unroll
-                    for (int d = 1; d < TAPS; ++d) {
-#pragma unroll
-                        for (int e = 0; e < 8; ++e) past[d - 1][e] = 0.f;
-                        if (d <= back) {
-                            unpack8(*reinterpret_cast<const uint4*>(proj + (size_t)(r - d) * p.proj_stride), past[d - 1]);
-#pragma unroll
-                            for (int e = 0; e < 8; ++e) past[d - 1][e] += bias[e];
-                        } else if (hist) {
-                            load8(hist + (size_t)(TAPS - 1 + back - d) * C, past[d - 1]);
-                        }
-                    }
-                }
-            }
-            float y[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                y[e] = w[TAPS > 0 ? TAPS - 1 : 0][e] * x[e];
-#pragma unroll
-                for (int d = 1; d < TAPS; ++d) y[e] += w[TAPS - 1 - d][e] * past[d - 1][e];
-            }
-            if (TAPS > 1) {                    // one position on
-#pragma unroll
-                for (int d = TAPS - 1; d > 1; --d)
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) past[d - 1][e] = past[d - 2][e];
-#pragma unroll
-                for (int e = 0; e < 8; ++e) past[0][e] = x[e];
-                if (p.single && hist) {
-#pragma unroll
-                    for (int d = 1; d < TAPS; ++d) store8(hist + (size_t)(TAPS - 1 - d) * C, past[d - 1]);
-                }
-            }
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = y[e];
-        }
-        before = b;
-        __nv_bfloat16* dst = (__nv_bfloat16*)p.qkv + (size_t)r * units * p.pad + c;
-        if (live && (is_v || (!is_q && p.values_from_keys))) {
-            const uint4 v = pack8(x);
-            *reinterpret_cast<uint4*>(dst + (is_v ? 0 : nk)) = v;
-            if (cell >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.v_pool + cell + head_at) = v;
-        }
+        if (k >= n_rows) break;
         if (p.q_gain) {
-            float2 s = make_float2(0.f, 0.f);
-            if (live && !is_v) {
-                float t = 0.f;
+            float total = 0.f;
+            for (int w = 0; w < n_warps; ++w) total += is_q ? sums[k][w].x : sums[k][w].y;
+            const float inv = 1.0f / sqrtf(total / (float)(is_q ? nq : nk) + p.eps);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) t += x[e] * x[e];
-                if (is_q) s.x = t;
-                else s.y = t;
-            }
-            s.x = warp_sum(s.x);
-            s.y = warp_sum(s.y);
-            const int lane = threadIdx.x & 31;
-            if (lane == 0) sums[k & 1][threadIdx.x >> 5] = s;
-            __syncthreads();                   // (two rows' sums in turn: one barrier a row is enough)
-            s = lane < (int)((blockDim.x + 31) >> 5) ? sums[k & 1][lane] : make_float2(0.f, 0.f);
-            const float aq = warp_sum(s.x), ak = warp_sum(s.y);
-            const float inv = 1.0f / sqrtf((is_q ? aq / (float)nq : ak / (float)nk) + p.eps);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = x[e] * inv * gain[e];
+            for (int e = 0; e < 8; ++e) acc[k][e] = acc[k][e] * inv * gain[e];
         }
-        if (live && !is_v) {
-            if (rotates) {
-                const float2* cs = turns + (size_t)k * half + d0 / 2;
+        if (rotates) {
+            const float2* cs = turns + (size_t)k * half + d0 / 2;
 #pragma unroll
-                for (int i = 0; i < 4; ++i)
-                    if (d0 / 2 + i < half) {
-                        const float2 t = cs[i];
-                        const float u = x[2 * i], v = x[2 * i + 1];
-                        x[2 * i] = u * t.x - v * t.y;
-                        x[2 * i + 1] = v * t.x + u * t.y;
-                    }
-            }
-            const uint4 y = pack8(x);
-            *reinterpret_cast<uint4*>(dst) = y;
-            if (cell >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.k_pool + cell + head_at) = y;
+            for (int i = 0; i < 4; ++i)
+                if (d0 / 2 + i < half) {
+                    const float2 t = cs[i];
+                    const float u = acc[k][2 * i], v = acc[k][2 * i + 1];
+                    acc[k][2 * i] = u * t.x - v * t.y;
+                    acc[k][2 * i + 1] = v * t.x + u * t.y;
+                }
         }
+        const uint4 y = pack8(acc[k]);
+        *reinterpret_cast<uint4*>(dst + (size_t)k * units * p.pad) = y;
+        if (!is_q && cells[k] >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.k_pool + cells[k] + head_at) = y;
     }
 }
 
@@ -376,20 +393,21 @@ SIB_EXPORT int sib_row_prepare(
         (rot == 0 || neighbours) && proj_stride % 8 == 0 && wide(proj) && wide(qkv) && wide(k_pool) && wide(v_pool) &&
         wide(bias) && wide(conv) && wide(q_gain) && wide(k_gain) && wide(state) && state_stride % 4 == 0) {
         const int threads = (channels / 8 + 31) / 32 * 32;
-        // few rows: a block each; many: runs of 4, which read the rows before them from registers
-        const int run = single || rows < 592 ? 1 : 4;
+        // few rows: a block each; many: runs of 2, whose rows share what they read
+        const int run = single || rows < 592 ? 1 : 2;
         const dim3 grid((rows + run - 1) / run);
         const size_t smem = (size_t)run * (rot / 2) * sizeof(float2) + 16;
 #define GO(TAPS, RUN)                                                                                              \
     do {                                                                                                           \
-        if (threads <= 512) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 512>, grid, dim3(threads), smem, s, p); \
-        else if (threads <= 768) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 768>, grid, dim3(threads), smem, s, p); \
-        else sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 1024>, grid, dim3(threads), smem, s, p);        \
+        if (threads <= 256) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 256, 3>, grid, dim3(threads), smem, s, p); \
+        else if (threads <= 384) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 384, 2>, grid, dim3(threads), smem, s, p); \
+        else if (threads <= 768) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 768, 1>, grid, dim3(threads), smem, s, p); \
+        else sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 1024, 1>, grid, dim3(threads), smem, s, p);     \
     } while (0)
 #define BY_RUN(TAPS)              \
     do {                          \
         if (run == 1) GO(TAPS, 1); \
-        else GO(TAPS, 4);         \
+        else GO(TAPS, 2);         \
     } while (0)
         if (taps == 0) BY_RUN(0);
         else if (taps == 1) BY_RUN(1);
