@@ -14,8 +14,9 @@
 // sequence are per-slot state, 32-bit, oldest first: state[slot] = [taps - 1][q and k channels].
 // Everything is 32-bit between the product's output and the packed rows.
 //
-//   row_prepare          a block per row (or per few rows), the row in shared memory or in registers;
+//   row_prepare          a block per row (or per run of rows), the row in shared memory or in registers;
 //                        steps of one row per sequence move the state on in the same launch
+//                        steps of prompts leave it as their last rows pass
 //   row_prepare_state    the state after any other step, in a launch of its own behind it
 //
 // Rows of a sequence that holds no slot (slot -1, fillers of a recorded step) see zeros before
@@ -24,6 +25,8 @@
 #include "common.cuh"
 
 namespace {
+
+constexpr int MAX_RUN = 32;        // the most rows of a block
 
 struct RowPrepareArgs {
     const void* proj;          // [rows, proj_stride]: q heads | k heads | (v heads) | ...
@@ -46,6 +49,8 @@ struct RowPrepareArgs {
     long long proj_stride, state_stride;
     int rows, n_heads, n_kv, kd, vd, pad, rot, taps;
     int values_from_keys, neighbours, single;
+    int fresh;                 // every sequence begins in this step: no history is read, and the last rows
+                               // of each leave theirs (else, unless `single`, row_prepare_state does)
     int max_pages, page_tokens, ring_tokens, fixed_tokens;
     float eps, magnitude;
 };
@@ -68,10 +73,12 @@ __global__ void __launch_bounds__(256) row_prepare_kernel(RowPrepareArgs p) {
     const int nq = p.n_heads * p.kd, nk = p.n_kv * p.kd, C = nq + nk;
     const int pos = p.row_pos[r], b = p.row_seq[r], slot = p.seq_slot[b];
     const int back = pos - p.seq_start[b];                   // rows of this step before this one
+    const int left = p.seq_end[b] - 1 - pos;                 // rows of the sequence behind this one
     const long long cell = cell_of_row(p, pos, b, slot);
     pdl_wait();
     const T* src = (const T*)p.proj + (size_t)r * p.proj_stride;
-    float* hist = p.taps > 1 && slot >= 0 ? p.state + (size_t)slot * p.state_stride : nullptr;
+    float* state = p.taps > 1 && slot >= 0 ? p.state + (size_t)slot * p.state_stride : nullptr;
+    const float* hist = p.fresh ? nullptr : state;
     float sq = 0.f, sk = 0.f;
     for (int c = threadIdx.x; c < C; c += blockDim.x) {
         const float bias = p.bias ? p.bias[c] : 0.f;
@@ -86,9 +93,12 @@ __global__ void __launch_bounds__(256) row_prepare_kernel(RowPrepareArgs p) {
                 else break;                                  // (zeros from here on)
                 acc += p.conv[(size_t)(p.taps - 1 - d) * C + c] * u;
             }
-            if (p.single && hist)
+            if (p.fresh && state) {
+                if (left < p.taps - 1) state[(size_t)(p.taps - 2 - left) * C + c] = own;
+            } else if (p.single && state) {
                 for (int k = 0; k < p.taps - 1; ++k)
-                    hist[(size_t)k * C + c] = k + 1 < p.taps - 1 ? hist[(size_t)(k + 1) * C + c] : own;
+                    state[(size_t)k * C + c] = k + 1 < p.taps - 1 ? state[(size_t)(k + 1) * C + c] : own;
+            }
         }
         row[c] = acc;
         if (c < nq) sq += acc * acc;
@@ -165,170 +175,190 @@ __device__ __forceinline__ uint4 pack8(const float (&x)[8]) {
 }
 
 // The common case in 16-byte accesses: bfloat16, heads of a multiple of 8 that need no filling
-// up, neighbouring pairs.  A thread owns 8 neighbouring channels of q, k or v and takes RUN
-// neighbouring rows at once.  A run inside one sequence whose first row has all its predecessors in
-// this step asks for its rows together and convolves them tap by tap from registers; in any other
-// run each row fetches what lies before it from the step's rows or from the state.  The rows'
-// sums cross the block with one barrier.  Where a row is stored, and its cosines and sines, are
-// worked out once per block ahead of the wait for the projection (positions and tables are
-// written by the host before the step).  TAPS 0: no convolution.
-template <int TAPS, int RUN, int THREADS, int BLOCKS>
-__global__ void __launch_bounds__(THREADS, BLOCKS) row_prepare_bf16_kernel(RowPrepareArgs p) {
+// up, neighbouring pairs.  q and k are normed apart, so blockIdx.x's first part takes a row's q
+// channels, its second the k channels (and the values that are made of them), its third the v
+// channels that a mixer has beside them.  A thread owns 8 neighbouring channels and walks the `run`
+// rows of its block: the next row is on its way while one is worked on, a row's shares of the next
+// TAPS - 1 rows' sums are added up in registers as it passes, so that it is unpacked once, and a row
+// costs one barrier.  Where the rows are stored, their cosines and sines, the taps and (SINGLE: one
+// row of each sequence) the history are fetched ahead of the wait for the projection: positions
+// and tables are written by the host before the step, the history by an earlier step.
+// TAPS 0: no convolution.
+template <int TAPS, bool SINGLE, int THREADS, int BLOCKS>
+__global__ void __launch_bounds__(THREADS, BLOCKS) row_prepare_bf16_kernel(RowPrepareArgs p, int run, int roles) {
     constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;          // rows before its own that a row reads
-    extern __shared__ float2 turns[];          // [RUN][rot / 2]
-    __shared__ float2 sums[RUN][32];
-    __shared__ long long cells[RUN];           // the rows' cells of kv head 0, or -1
-    __shared__ int slots[RUN], backs[RUN], seqs[RUN];
+    constexpr int HELD = BACK > 0 ? BACK : 1;
+    __shared__ __align__(16) float sums[2][32];            // [row & 1][warp]
+    __shared__ long long cells[MAX_RUN];       // the rows' cells of kv head 0, or -1
+    __shared__ int slots[MAX_RUN], backs[MAX_RUN], seqs[MAX_RUN], lefts[MAX_RUN];
+    extern __shared__ float4 turns[];          // [run][2][groups]: (cos, sin) of a thread's 4 pairs, 2 and 2
     pdl_trigger();
     const int nq = p.n_heads * p.kd, nk = p.n_kv * p.kd, C = nq + nk;
     const int units = p.n_heads + 2 * p.n_kv;
-    const int c = 8 * threadIdx.x;             // the thread's first channel of the projected row
-    const bool live = c < C + (p.values_from_keys ? 0 : nk);
-    const bool is_q = c < nq, is_v = c >= C;   // (v channels of their own are passed on)
-    const int r0 = blockIdx.x * RUN, n_rows = min(RUN, p.rows - r0);
-    const int half = p.inv_freq ? p.rot / 2 : 0;
+    const int role = blockIdx.x % roles;       // 0: q, 1: k, 2: v of its own
+    const bool is_q = role == 0, is_v = role == 2;
+    const int width = is_q ? nq : nk, c0 = is_q ? 0 : is_v ? C : nq;
+    const int lc = 8 * threadIdx.x, c = c0 + lc;           // the thread's first channel of the projected row
+    const bool live = lc < width;
+    const int r0 = (blockIdx.x / roles) * run, n_rows = min(run, p.rows - r0);
+    const int groups = p.inv_freq && !is_v ? (p.rot + 7) / 8 : 0;
     if ((int)threadIdx.x < n_rows) {
         const int r = r0 + threadIdx.x, pos = p.row_pos[r], b = p.row_seq[r], slot = p.seq_slot[b];
-        cells[threadIdx.x] = cell_of_row(p, pos, b, slot);
+        cells[threadIdx.x] = is_q ? -1 : cell_of_row(p, pos, b, slot);
         slots[threadIdx.x] = slot;
         backs[threadIdx.x] = pos - p.seq_start[b];
         seqs[threadIdx.x] = b;
+        lefts[threadIdx.x] = p.seq_end[b] - 1 - pos;       // rows of the sequence behind this one
     }
-    for (int i = threadIdx.x; i < n_rows * half; i += blockDim.x) {
-        const int k = i / half;
-        const float ang = (float)p.row_pos[r0 + k] * p.inv_freq[i - k * half];
-        turns[i] = make_float2(cosf(ang) * p.magnitude, sinf(ang) * p.magnitude);
+    for (int i = threadIdx.x; i < 64; i += blockDim.x) (&sums[0][0])[i] = 0.f;      // (warps that are not there)
+    for (int i = threadIdx.x; i < n_rows * groups * 4; i += blockDim.x) {
+        const int k = i / (groups * 4), pair = i - k * groups * 4;
+        float2 t = make_float2(1.f, 0.f);      // (pairs behind the rotated ones pass)
+        if (2 * pair < p.rot) {
+            const float ang = (float)p.row_pos[r0 + k] * p.inv_freq[pair];
+            t = make_float2(cosf(ang) * p.magnitude, sinf(ang) * p.magnitude);
+        }
+        reinterpret_cast<float2*>(turns + (size_t)(2 * k + ((pair >> 1) & 1)) * groups + (pair >> 2))[pair & 1] = t;
     }
-    float bias[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) bias[e] = 0.f;
-    if (live && p.bias) load8(p.bias + c, bias);
-    __syncthreads();
     const bool conv = TAPS > 0 && live && !is_v;
-    const bool together = n_rows == RUN && seqs[RUN - 1] == seqs[0] && backs[0] >= BACK;
-    pdl_wait();
-    const __nv_bfloat16* proj = (const __nv_bfloat16*)p.proj + (size_t)r0 * p.proj_stride + c;
-    auto fetch = [&](int row) {                // `row`: from the run's first
-        return *reinterpret_cast<const uint4*>(proj + (long long)row * p.proj_stride);
+    float bias[8], gain[8], w[TAPS > 0 ? TAPS : 1][8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { bias[e] = 0.f; gain[e] = 1.f; }
+    if (live && p.bias) load8(p.bias + c, bias);
+    if (live && p.q_gain && !is_v) load8((is_q ? p.q_gain : p.k_gain) + lc, gain);
+    if (conv) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) load8(p.conv + (size_t)j * C + c, w[j]);
+    }
+    const float inv_n = 1.0f / (float)width;
+    const int head = lc / p.kd, d0 = lc - head * p.kd;     // the thread's head and its place there
+    const bool rotates = d0 < 8 * groups;
+    // where the thread's 8 values go in a pool behind a row's cell
+    const size_t head_at = (size_t)head * p.page_tokens * p.pad + d0;
+    __syncthreads();
+    auto state_of = [&](int slot) {
+        return BACK > 0 && slot >= 0 ? p.state + (size_t)slot * p.state_stride + c : nullptr;
     };
+    float past[HELD][8];                       // the input d + 1 positions back
+    // what the rows passed so far add to the next row's sum, the one behind it, ...
+    float ahead[HELD][8];
+    auto look_ahead = [&]() {
+#pragma unroll
+        for (int f = 0; f < BACK; ++f)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                ahead[f][e] = 0.f;
+#pragma unroll
+                for (int d = 0; d + f < BACK; ++d) ahead[f][e] += w[TAPS > 1 ? TAPS - 2 - d - f : 0][e] * past[d][e];
+            }
+    };
+    if (SINGLE && conv) {
+        const float* hist = state_of(slots[0]);
+#pragma unroll
+        for (int d = 0; d < BACK; ++d) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) past[d][e] = 0.f;
+            if (hist) load8(hist + (size_t)(BACK - 1 - d) * C, past[d]);
+        }
+        look_ahead();
+    }
+    pdl_wait();
+    const __nv_bfloat16* src = (const __nv_bfloat16*)p.proj + (size_t)r0 * p.proj_stride + c;
+    uint4 next = live ? *reinterpret_cast<const uint4*>(src) : make_uint4(0, 0, 0, 0);
     auto input = [&](const uint4& raw, float (&u)[8]) {
         unpack8(raw, u);
 #pragma unroll
         for (int e = 0; e < 8; ++e) u[e] += bias[e];
     };
-    float acc[RUN][8];
-#pragma unroll
-    for (int k = 0; k < RUN; ++k)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[k][e] = 0.f;
-    if (conv && together && RUN > 1) {
-        uint4 raw[RUN + BACK];
-#pragma unroll
-        for (int k = 0; k < RUN + BACK; ++k) raw[k] = fetch(k - BACK);
-#pragma unroll
-        for (int j = TAPS - 1; j >= 0; --j) {
-            float w[8];
-            load8(p.conv + (size_t)j * C + c, w);
-#pragma unroll
-            for (int k = 0; k < RUN; ++k) {
-                float u[8];
-                input(raw[k + j], u);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) acc[k][e] += w[e] * u[e];
-            }
-        }
-    } else if (conv) {
-#pragma unroll
-        for (int k = 0; k < RUN; ++k) {
-            if (k >= n_rows) break;
-            float u[BACK + 1][8];              // u[d]: the input d positions back
-            input(fetch(k), u[0]);
-            float* hist = BACK > 0 && slots[k] >= 0 ? p.state + (size_t)slots[k] * p.state_stride + c : nullptr;
-#pragma unroll
-            for (int d = 1; d <= BACK; ++d) {
-#pragma unroll
-                for (int e = 0; e < 8; ++e) u[d][e] = 0.f;
-                if (d <= backs[k]) input(fetch(k - d), u[d]);
-                else if (hist) load8(hist + (size_t)(BACK + backs[k] - d) * C, u[d]);
-            }
-#pragma unroll
-            for (int d = 0; d <= BACK; ++d) {
-                float w[8];
-                load8(p.conv + (size_t)(TAPS > 0 ? TAPS - 1 - d : 0) * C + c, w);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) acc[k][e] += w[e] * u[d][e];
-            }
-            if (p.single && hist) {            // one position on
-#pragma unroll
-                for (int d = 0; d < BACK; ++d) store8(hist + (size_t)(BACK - 1 - d) * C, u[d]);
-            }
-        }
-    } else if (live) {
-#pragma unroll
-        for (int k = 0; k < RUN; ++k)
-            if (k < n_rows) input(fetch(k), acc[k]);
-    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (width / 8 + 31) >> 5;
     __nv_bfloat16* dst = (__nv_bfloat16*)p.qkv + (size_t)r0 * units * p.pad + c;
-    const int d0 = c % p.kd;                   // the thread's place in its head
-    // where the thread's 8 values go in a pool behind a row's cell
-    const size_t head_at = (size_t)((is_v ? c - C : c - nq) / p.kd) * p.page_tokens * p.pad + d0;
-    if (live && (is_v || (!is_q && p.values_from_keys))) {
+#pragma unroll 1
+    for (int k = 0; k < n_rows; ++k, dst += (size_t)units * p.pad) {
+        const uint4 raw = next;
+        if (!SINGLE && live && k + 1 < n_rows)
+            next = *reinterpret_cast<const uint4*>(src + (size_t)(k + 1) * p.proj_stride);
+        float x[8];
+        input(raw, x);
+        if (conv) {
+            if (SINGLE) {
+                float* hist = state_of(slots[0]);
+                if (BACK > 0 && hist) {        // one position on
+                    store8(hist + (size_t)(BACK - 1) * C, x);
 #pragma unroll
-        for (int k = 0; k < RUN; ++k) {
-            if (k >= n_rows) break;
-            const uint4 v = pack8(acc[k]);
-            *reinterpret_cast<uint4*>(dst + (size_t)k * units * p.pad + (is_v ? 0 : nk)) = v;
-            if (cells[k] >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.v_pool + cells[k] + head_at) = v;
-        }
-    }
-    const int lane = threadIdx.x & 31, n_warps = (blockDim.x + 31) >> 5;
-    float gain[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) gain[e] = 1.f;
-    if (p.q_gain) {
-        // (a warp of q channels alone, or of others alone, sums one number a row)
-        const bool any_q = __any_sync(0xffffffffu, is_q), any_k = __any_sync(0xffffffffu, !is_q);
-#pragma unroll
-        for (int k = 0; k < RUN; ++k) {
-            float t = 0.f;
-            if (live && !is_v) {
-#pragma unroll
-                for (int e = 0; e < 8; ++e) t += acc[k][e] * acc[k][e];
-            }
-            float2 s = make_float2(0.f, 0.f);
-            if (any_q) s.x = warp_sum(is_q ? t : 0.f);
-            if (any_k) s.y = warp_sum(is_q ? 0.f : t);
-            if (lane == 0) sums[k][threadIdx.x >> 5] = s;
-        }
-        if (live && !is_v) load8(is_q ? p.q_gain + c : p.k_gain + (c - nq), gain);
-        __syncthreads();
-    }
-    if (is_v || !live) return;                 // (neither a barrier nor a shuffle is left)
-    const bool rotates = d0 < 2 * half;
-#pragma unroll
-    for (int k = 0; k < RUN; ++k) {
-        if (k >= n_rows) break;
-        if (p.q_gain) {
-            float total = 0.f;
-            for (int w = 0; w < n_warps; ++w) total += is_q ? sums[k][w].x : sums[k][w].y;
-            const float inv = 1.0f / sqrtf(total / (float)(is_q ? nq : nk) + p.eps);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) acc[k][e] = acc[k][e] * inv * gain[e];
-        }
-        if (rotates) {
-            const float2* cs = turns + (size_t)k * half + d0 / 2;
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-                if (d0 / 2 + i < half) {
-                    const float2 t = cs[i];
-                    const float u = acc[k][2 * i], v = acc[k][2 * i + 1];
-                    acc[k][2 * i] = u * t.x - v * t.y;
-                    acc[k][2 * i + 1] = v * t.x + u * t.y;
+                    for (int d = 0; d + 1 < BACK; ++d) store8(hist + (size_t)(BACK - 2 - d) * C, past[d]);
                 }
+            } else if (BACK > 0 && (k == 0 || seqs[k] != seqs[k - 1])) {
+                // the block's first row of a sequence: what lies before it, from the step's rows or the state
+                const int back = backs[k];     // rows of this step before this one
+                const float* hist = p.fresh ? nullptr : state_of(slots[k]);
+#pragma unroll
+                for (int d = 0; d < BACK; ++d) {
+                    if (d < back) {
+                        input(*reinterpret_cast<const uint4*>(src + (long long)(k - d - 1) * p.proj_stride), past[d]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) past[d][e] = 0.f;
+                        if (hist) load8(hist + (size_t)(BACK - 1 + back - d) * C, past[d]);
+                    }
+                }
+                look_ahead();
+            }
+            if (!SINGLE && BACK > 0 && p.fresh && lefts[k] < BACK) {
+                float* state = state_of(slots[k]);
+                if (state) store8(state + (size_t)(BACK - 1 - lefts[k]) * C, x);
+            }
+            float y[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                y[e] = w[TAPS > 0 ? TAPS - 1 : 0][e] * x[e];
+                if (BACK > 0) y[e] += ahead[0][e];
+#pragma unroll
+                for (int f = 0; f < BACK; ++f)
+                    ahead[f][e] = w[TAPS > 1 ? TAPS - 2 - f : 0][e] * x[e] + (f + 1 < BACK ? ahead[f + 1 < BACK ? f + 1 : 0][e] : 0.f);
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = y[e];
         }
-        const uint4 y = pack8(acc[k]);
-        *reinterpret_cast<uint4*>(dst + (size_t)k * units * p.pad) = y;
-        if (!is_q && cells[k] >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.k_pool + cells[k] + head_at) = y;
+        const long long cell = cells[k];
+        if (live && (is_v || (!is_q && p.values_from_keys))) {
+            const uint4 v = pack8(x);
+            *reinterpret_cast<uint4*>(dst + (is_v ? 0 : nk)) = v;
+            if (cell >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.v_pool + cell + head_at) = v;
+        }
+        if (is_v) continue;                    // (the same for the whole block)
+        if (p.q_gain) {
+            float t = 0.f;
+            if (live) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) t += x[e] * x[e];
+            }
+            t = warp_sum(t);
+            if (lane == 0) sums[k & 1][warp] = t;
+            __syncthreads();                   // (two rows' sums in turn: one barrier a row is enough)
+            float total = 0.f;
+            for (int i = 0; i < n_warps; i += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(&sums[k & 1][i]);
+                total += (f.x + f.y) + (f.z + f.w);
+            }
+            const float inv = rsqrtf(total * inv_n + p.eps);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = x[e] * inv * gain[e];
+        }
+        if (live) {
+            if (rotates) {
+                const float4 lo = turns[(size_t)2 * k * groups + d0 / 8], hi = turns[(size_t)(2 * k + 1) * groups + d0 / 8];
+                const float cs[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float u = x[2 * i], v = x[2 * i + 1];
+                    x[2 * i] = u * cs[2 * i] - v * cs[2 * i + 1];
+                    x[2 * i + 1] = v * cs[2 * i] + u * cs[2 * i + 1];
+                }
+            }
+            const uint4 y = pack8(x);
+            *reinterpret_cast<uint4*>(dst) = y;
+            if (cell >= 0) *reinterpret_cast<uint4*>((__nv_bfloat16*)p.k_pool + cell + head_at) = y;
+        }
     }
 }
 
@@ -356,14 +386,16 @@ __global__ void __launch_bounds__(256) row_prepare_state_kernel(RowPrepareArgs p
 
 }  // namespace
 
-// `single`: every sequence of the step has exactly one row.  `taps` 0: no convolution.
+// `single`: every sequence of the step has exactly one row.  `fresh`: every sequence begins in this
+// step, with a state of zeros.  `taps` 0: no convolution.
 SIB_EXPORT int sib_row_prepare(
     const void* proj, long long proj_stride, void* qkv, int dtype, const float* bias, const float* conv, int taps,
     float* state, long long state_stride, const float* q_gain, const float* k_gain, float eps,
     const float* inv_freq, int rot, int neighbours, float magnitude, const int* row_pos, const int* row_seq,
     const int* seq_slot, const int* seq_start, const int* seq_end, const int* seq_row0, void* k_pool, void* v_pool,
     const int* page_table, int max_pages, int page_tokens, int ring_tokens, int fixed_tokens, int rows, int n_seqs,
-    int n_heads, int n_kv, int kd, int vd, int pad, int values_from_keys, int single, void* stream) {
+    int n_heads, int n_kv, int kd, int vd, int pad, int values_from_keys, int single,
+    int fresh, void* stream) {
     if (rows == 0) return 0;
     SIB_REQUIRE(rows > 0 && n_seqs > 0 && n_seqs < 65536 && n_heads > 0 && n_kv > 0 && kd > 0 && vd > 0,
                 "row_prepare: rows=%d sequences=%d heads=%d kv_heads=%d key width=%d value width=%d", rows, n_seqs,
@@ -384,37 +416,38 @@ SIB_EXPORT int sib_row_prepare(
                 "row_prepare: incomplete cache description");
     RowPrepareArgs p{proj, qkv, bias, conv, state, q_gain, k_gain, rot ? inv_freq : nullptr, row_pos, row_seq,
                      seq_slot, seq_start, seq_end, seq_row0, k_pool, v_pool, page_table, proj_stride, state_stride,
-                     rows, n_heads, n_kv, kd, vd, pad, rot, taps, values_from_keys, neighbours, single,
+                     rows, n_heads, n_kv, kd, vd, pad, rot, taps, values_from_keys, neighbours, single, fresh,
                      max_pages, page_tokens, ring_tokens, fixed_tokens, eps, magnitude};
     cudaStream_t s = (cudaStream_t)stream;
     auto wide = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
-    const int channels = C + (values_from_keys ? 0 : nk);
-    if (dtype == SIB_BF16 && kd == vd && kd == pad && kd % 8 == 0 && channels <= 8192 && taps <= 4 &&
+    if (dtype == SIB_BF16 && kd == vd && kd == pad && kd % 8 == 0 && nq <= 8192 && nk <= 8192 && taps <= 4 && rows < (1 << 28) &&
         (rot == 0 || neighbours) && proj_stride % 8 == 0 && wide(proj) && wide(qkv) && wide(k_pool) && wide(v_pool) &&
         wide(bias) && wide(conv) && wide(q_gain) && wide(k_gain) && wide(state) && state_stride % 4 == 0) {
-        const int threads = (channels / 8 + 31) / 32 * 32;
-        // few rows: a block each; many: runs of 2, whose rows share what they read
-        const int run = single || rows < 592 ? 1 : 2;
-        const dim3 grid((rows + run - 1) / run);
-        const size_t smem = (size_t)run * (rot / 2) * sizeof(float2) + 16;
-#define GO(TAPS, RUN)                                                                                              \
-    do {                                                                                                           \
-        if (threads <= 256) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 256, 3>, grid, dim3(threads), smem, s, p); \
-        else if (threads <= 384) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 384, 2>, grid, dim3(threads), smem, s, p); \
-        else if (threads <= 768) sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 768, 1>, grid, dim3(threads), smem, s, p); \
-        else sib_launch_chained(row_prepare_bf16_kernel<TAPS, RUN, 1024, 1>, grid, dim3(threads), smem, s, p);     \
+        const int threads = ((nq > nk ? nq : nk) / 8 + 31) / 32 * 32;
+        const int roles = values_from_keys ? 2 : 3;
+        // as many rows a block as spread them over the SMs in one wave (two blocks an SM up to 256 threads)
+        const int blocks = 148 * (threads <= 256 ? 2 : 1) / roles, even = (rows + blocks - 1) / blocks;
+        const size_t row_bytes = (size_t)2 * ((rot + 7) / 8) * sizeof(float4);
+        int run = single ? 1 : even < MAX_RUN ? even : MAX_RUN;
+        while (run > 1 && run * row_bytes > 40 * 1024) --run;
+        const dim3 grid((unsigned)((rows + run - 1) / run) * roles);
+        const size_t smem = run * row_bytes + 16;
+#define GO(TAPS, SINGLE, THREADS, BLOCKS)                                                                          \
+    sib_launch_chained(row_prepare_bf16_kernel<TAPS, SINGLE, THREADS, BLOCKS>, grid, dim3(threads), smem, s, p, run, roles)
+#define BY_STEP(TAPS)                                         \
+    do {                                                      \
+        if (single && threads <= 512) GO(TAPS, true, 512, 1); \
+        else if (single) GO(TAPS, true, 1024, 1);             \
+        else if (threads <= 256) GO(TAPS, false, 256, 2);     \
+        else if (threads <= 512) GO(TAPS, false, 512, 1);     \
+        else GO(TAPS, false, 1024, 1);                        \
     } while (0)
-#define BY_RUN(TAPS)              \
-    do {                          \
-        if (run == 1) GO(TAPS, 1); \
-        else GO(TAPS, 2);         \
-    } while (0)
-        if (taps == 0) BY_RUN(0);
-        else if (taps == 1) BY_RUN(1);
-        else if (taps == 2) BY_RUN(2);
-        else if (taps == 3) BY_RUN(3);
-        else BY_RUN(4);
-#undef BY_RUN
+        if (taps == 0) BY_STEP(0);
+        else if (taps == 1) BY_STEP(1);
+        else if (taps == 2) BY_STEP(2);
+        else if (taps == 3) BY_STEP(3);
+        else BY_STEP(4);
+#undef BY_STEP
 #undef GO
     } else {
         const size_t smem = (size_t)C * sizeof(float);
@@ -429,7 +462,7 @@ SIB_EXPORT int sib_row_prepare(
         });
     }
     int rc = sib_check_launch("row_prepare");
-    if (rc || single || taps <= 1) return rc;
+    if (rc || single || fresh || taps <= 1) return rc;
     SIB_DISPATCH_DTYPE(dtype, sib_launch_chained(row_prepare_state_kernel<T>, dim3((C + 255) / 256, n_seqs), dim3(256), 0,
                                                  s, p));
     return sib_check_launch("row_prepare_state");

@@ -929,7 +929,7 @@ def row_prepare(proj: torch.Tensor, qkv: torch.Tensor, ctx, *, n_heads: int, n_k
         _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_end), _ptr(ctx.seq_row0), _ptr(k_pool), _ptr(v_pool),
         _ptr(page_table), c_int(max_pages), c_int(page_tokens), c_int(ring_tokens), c_int(fixed_tokens), c_int(rows),
         c_int(ctx.n_seqs), c_int(n_heads), c_int(n_kv), c_int(key_dim), c_int(value_dim), c_int(pad),
-        c_int(1 if values_from_keys else 0), c_int(1 if single else 0), _stream()))
+        c_int(1 if values_from_keys else 0), c_int(1 if single else 0), c_int(1 if ctx.all_from_start else 0), _stream()))
     return qkv
 
 

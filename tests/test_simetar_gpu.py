@@ -512,6 +512,7 @@ class _Step:
         rows = [n for _, _, n in seqs]
         self.seq_row0 = i32([sum(rows[:b]) for b in range(len(rows))])
         self.n_rows, self.n_seqs, self.max_count = sum(rows), len(seqs), max(rows)
+        self.all_from_start = all(st == 0 for _, st, _ in seqs)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
